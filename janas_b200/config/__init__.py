@@ -132,6 +132,8 @@ class RunEntry:
     cache_of: Optional[int] = None
     # before this entry the embedding output is added to the residual stream once more
     add_embedding: bool = False
+    # before this entry the residual stream becomes the model's join matrix over it and the embedding output
+    join_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -154,6 +156,7 @@ class ModelSpec:
     embedding_norm_name: str = "model.embed_norm"
     token_table_name: str = ""         # a second table of vectors per token that the layers' blocks read; "": none
     token_table_width: int = 0
+    join_name: str = ""                # the matrix of the entries with join_embedding; "": none
 
     def to_json(self) -> Dict[str, Any]:
         d = {
@@ -161,7 +164,8 @@ class ModelSpec:
             "vocab_size": self.vocab_size, "max_positions": self.max_positions,
             "layers": [l.to_json() for l in self.layers],
             "run_order": [dict({"layer": e.layer, "cache_of": e.cache_of},
-                               **({"add_embedding": True} if e.add_embedding else {}))
+                               **({"add_embedding": True} if e.add_embedding else {}),
+                               **({"join_embedding": True} if e.join_embedding else {}))
                           for e in self.run_order],
             "final_norm": self.final_norm.to_json(), "tie_embeddings": self.tie_embeddings,
             "embedding_name": self.embedding_name, "final_norm_name": self.final_norm_name,
@@ -175,6 +179,8 @@ class ModelSpec:
         if self.token_table_name:
             d["token_table_name"] = self.token_table_name
             d["token_table_width"] = self.token_table_width
+        if self.join_name:
+            d["join_name"] = self.join_name
         if self.embedding_norm:
             d["embedding_norm"] = self.embedding_norm.to_json()
             d["embedding_norm_name"] = self.embedding_norm_name
@@ -189,11 +195,13 @@ class ModelSpec:
             embedding_scale=d.get("embedding_scale", 1.0),
             token_table_name=d.get("token_table_name", ""),
             token_table_width=d.get("token_table_width", 0),
+            join_name=d.get("join_name", ""),
             embedding_norm=PartSpec.from_json(d["embedding_norm"]) if d.get("embedding_norm") else None,
             embedding_norm_name=d.get("embedding_norm_name", "model.embed_norm"),
             architecture=d["architecture"], hidden_size=d["hidden_size"],
             vocab_size=d["vocab_size"], max_positions=d["max_positions"], layers=layers,
-            run_order=tuple(RunEntry(e["layer"], e["cache_of"], bool(e.get("add_embedding", False)))
+            run_order=tuple(RunEntry(e["layer"], e["cache_of"], bool(e.get("add_embedding", False)),
+                                     bool(e.get("join_embedding", False)))
                             for e in d["run_order"]),
             final_norm=PartSpec.from_json(d["final_norm"]), tie_embeddings=d["tie_embeddings"],
             embedding_name=d["embedding_name"], final_norm_name=d["final_norm_name"],
@@ -348,8 +356,40 @@ class MunisunConfig:
         return hash(json.dumps(self.to_dict(), sort_keys=True))
 
 
+@dataclass(frozen=True)
+class SalivikConfig:
+    """The Salivik decoder's ``config.json`` keys, as the library read them."""
+    vocab: int
+    width: int
+    norm_eps: float
+    loop: Optional[Mapping[str, int]]         # start, stop, times; None: every layer runs once
+    layers: Tuple[Mapping[str, Any], ...]     # each: type, mixer {...}, mlp {...} or None
+    eos_token_ids: Tuple[int, ...] = ()
+    architecture: str = "Salivik"
+    _json: Mapping[str, Any] = field(default_factory=dict, compare=False, repr=False)
+    _spec: Mapping[str, Any] = field(default_factory=dict, compare=False, repr=False)
+
+    @classmethod
+    def from_dict(cls, d: Mapping[str, Any]) -> "SalivikConfig":
+        return _wrap(_call("config.parse", config=dict(d)))
+
+    def to_dict(self) -> Dict[str, Any]:
+        return dict(self._json)
+
+    def to_model_spec(self) -> ModelSpec:
+        return ModelSpec.from_json(self._spec)
+
+    def __hash__(self) -> int:
+        return hash(json.dumps(self.to_dict(), sort_keys=True))
+
+
 def _wrap(r: Mapping[str, Any]):
     c = r["config"]
+    if r["architecture"] == "Salivik":
+        return SalivikConfig(
+            vocab=c["vocab"], width=c["width"], norm_eps=c["norm"]["eps"],
+            loop=dict(c["loop"]) if c["loop"] else None, layers=tuple(c["layers"]),
+            eos_token_ids=tuple(r["eos_token_ids"]), _json=c, _spec=r["spec"])
     if r["architecture"] == "Munisun":
         return MunisunConfig(
             vocab=c["vocab"], width=c["width"], norm_eps=c["norm"]["eps"],
@@ -400,4 +440,5 @@ def config_from_dir(model_dir: str):
 
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "Qwen3Config",
-           "ZuzelornConfig", "DunavikConfig", "KefesunConfig", "MunisunConfig", "config_from_dict", "config_from_dir", "known_architectures"]
+           "ZuzelornConfig", "DunavikConfig", "KefesunConfig", "MunisunConfig",
+           "SalivikConfig", "config_from_dict", "config_from_dir", "known_architectures"]

@@ -38,6 +38,7 @@ static Tables &ready() {
         register_dunavik();
         register_kefesun();
         register_munisun();
+        register_salivik();
     });
     return raw_tables();
 }

@@ -56,6 +56,10 @@ void ModelSpec::validate() const {
         if (e.layer < 0 || e.layer >= (int)layers.size())
             config_error(fmt("run order entry %zu names layer %d, the model has %zu", at, e.layer,
                              layers.size()));
+        if (e.join_embedding && join_name.empty())
+            config_error(fmt("run order entry %zu joins the embedding output and the model names no join matrix", at));
+        if (e.join_embedding && e.add_embedding)
+            config_error(fmt("run order entry %zu both adds and joins the embedding output", at));
         if (e.cache_of >= 0) {
             if (e.cache_of >= (int)at)
                 config_error(fmt("run order entry %zu reads the cache of entry %d, which has not run "
@@ -100,6 +104,7 @@ Json ModelSpec::to_json() const {
         o.set("layer", e.layer);
         o.set("cache_of", e.cache_of >= 0 ? Json(e.cache_of) : Json());
         if (e.add_embedding) o.set("add_embedding", true);
+        if (e.join_embedding) o.set("join_embedding", true);
         ro.push(o);
     }
     j.set("run_order", ro);
@@ -116,6 +121,7 @@ Json ModelSpec::to_json() const {
         j.set("token_table_name", token_table_name);
         j.set("token_table_width", token_table_width);
     }
+    if (!join_name.empty()) j.set("join_name", join_name);
     j.set("embedding_name", embedding_name);
     j.set("final_norm_name", final_norm_name);
     j.set("head_name", head_name);
@@ -163,6 +169,7 @@ ModelSpec ModelSpec::from_json(const Json &j) {
         e.layer = (int)o.get("layer").as_int();
         e.cache_of = o.get("cache_of").is_null() ? -1 : (int)o.get("cache_of").as_int();
         e.add_embedding = o.get("add_embedding").is_bool() && o.get("add_embedding").as_bool();
+        e.join_embedding = o.get("join_embedding").is_bool() && o.get("join_embedding").as_bool();
         s.run_order.push_back(e);
     }
     s.final_norm = PartSpec::from_json(j.get("final_norm"));
@@ -174,6 +181,7 @@ ModelSpec ModelSpec::from_json(const Json &j) {
     if (j.get("embedding_scale").is_number()) s.embedding_scale = j.get("embedding_scale").as_double();
     s.token_table_name = str_or(j, "token_table_name", "");
     if (j.get("token_table_width").is_number()) s.token_table_width = j.get("token_table_width").as_int();
+    s.join_name = str_or(j, "join_name", "");
     s.embedding_name = str_or(j, "embedding_name", s.embedding_name);
     s.final_norm_name = str_or(j, "final_norm_name", s.final_norm_name);
     s.head_name = str_or(j, "head_name", s.head_name);

@@ -77,10 +77,15 @@ struct LayerSpec {
 // add_embedding: before this entry runs, the embedding output (the residual stream
 // as it was before the first entry) is added to the residual stream once more: the
 // start of a repeated pass over layers that have run already.
+//
+// join_embedding: before this entry runs, the residual stream x becomes J [x; e], the
+// model's join matrix (ModelSpec::join_name, [hidden, 2 hidden]) over x and the embedding
+// output e side by side.
 struct RunEntry {
     int layer = 0;
     int cache_of = -1;
     bool add_embedding = false;
+    bool join_embedding = false;
 };
 
 struct ModelSpec {
@@ -104,6 +109,8 @@ struct ModelSpec {
     // the layers' blocks read by columns (a per-layer input of the token itself)
     std::string token_table_name;
     long long token_table_width = 0;
+    // the matrix of the run-order entries with join_embedding ("": the model has none)
+    std::string join_name;
     std::string embedding_name = "model.embed_tokens.weight";
     std::string final_norm_name = "model.norm";
     std::string head_name = "lm_head.weight";

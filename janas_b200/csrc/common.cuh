@@ -115,6 +115,20 @@ __device__ __forceinline__ float add_partials(float v, const float *__restrict__
 // writes are visible.  What a kernel does before pdl_wait() must not touch
 // anything an earlier kernel writes or reads-and-frees: only its own shared and
 // tensor memory and the (immutable) weights.
+// A gated unit of a feed-forward: g sigmoid(alpha g) (u + shift), with limit > 0 both sides cut
+// off first: g <- min(g, limit), u <- clamp(u, -limit, limit).  {1, 0, 0} is SiLU(g) u.
+struct GatedUnit {
+    float alpha, limit, shift;
+};
+__device__ __forceinline__ float gated_unit(float g, float u, const GatedUnit &p)
+{
+    if (p.limit > 0.0f) {
+        g = fminf(g, p.limit);
+        u = fminf(fmaxf(u, -p.limit), p.limit);
+    }
+    return g / (1.0f + expf(-p.alpha * g)) * (u + p.shift);
+}
+
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_trigger()
 {

@@ -147,14 +147,26 @@ __device__ __forceinline__ void store_partial(uint32_t taddr, int hgrp, float *_
     }
 }
 
-// SiLU(gate) * up in bfloat16: the gate's tokens are columns [0, BN), the up
-// projection's [BN, 2 BN).  SiLU(g) u = g u / (1 + 2^(-g log2 e)), with the
-// approximate exponential and reciprocal (a few units in the last place of a
-// float; the result is rounded to bfloat16).
+// The gated unit (common.cuh) with the approximate exponential and reciprocal: g sigmoid(alpha g)
+// u = g u / (1 + 2^(-alpha g log2 e)), a few units in the last place of a float; the result is
+// rounded to bfloat16.  k: -alpha log2 e.
+__device__ __forceinline__ bf16 unit_bf16(float g, float u, float k, const GatedUnit &p)
+{
+    if (p.limit > 0.0f) {
+        g = fminf(g, p.limit);
+        u = fminf(fmaxf(u, -p.limit), p.limit);
+    }
+    float e = fast_exp2(g * k);
+    return __float2bfloat16_rn(__fdividef(g * (u + p.shift), 1.0f + e));
+}
+
+// The gated unit of gate and up in bfloat16: the gate's tokens are columns [0, BN), the up
+// projection's [BN, 2 BN).
 template <int BN>
 __device__ __forceinline__ void store_swiglu(uint32_t taddr, int hgrp, bf16 *__restrict__ out_act,
-                                             int f, int ff, int n0, int n)
+                                             int f, int ff, int n0, int n, const GatedUnit &unit)
 {
+    const float k = unit.alpha * -1.4426950408889634f;
     uint32_t ga[32], ua[32], gb[32], ub[32];
     auto act32 = [&](const uint32_t *g, const uint32_t *u, int c0) {
         if (f >= ff)
@@ -164,9 +176,7 @@ __device__ __forceinline__ void store_swiglu(uint32_t taddr, int hgrp, bf16 *__r
 #pragma unroll
         for (int j = 0; j < 32; j++, p += ff) {
             if (whole || n0 + c0 + j < n) {
-                float gv = __uint_as_float(g[j]), uv = __uint_as_float(u[j]);
-                float e = fast_exp2(gv * -1.4426950408889634f);
-                *p = __float2bfloat16_rn(__fdividef(gv * uv, 1.0f + e));
+                *p = unit_bf16(__uint_as_float(g[j]), __uint_as_float(u[j]), k, unit);
             }
         }
     };
@@ -203,8 +213,9 @@ template <int BN>
 __device__ __forceinline__ void store_swiglu_half(uint32_t taddr, int q, int lane, int hgrp,
                                                   bool ok, float *xch,
                                                   bf16 *__restrict__ out_act, int m0, int ff,
-                                                  int n0, int n)
+                                                  int n0, int n, const GatedUnit &unit)
 {
+    const float k = unit.alpha * -1.4426950408889634f;
     constexpr int LD = BN + 1;
     float v[16];
     if (ok && q >= 2) {
@@ -226,11 +237,8 @@ __device__ __forceinline__ void store_swiglu_half(uint32_t taddr, int q, int lan
                 bf16 *p = out_act + (size_t)(n0 + c) * ff + f;
 #pragma unroll
                 for (int j = 0; j < 16; j++, p += ff)
-                    if (n0 + c + j < n) {
-                        float gv = v[j], uv = row[c + j];
-                        float e = fast_exp2(gv * -1.4426950408889634f);
-                        *p = __float2bfloat16_rn(__fdividef(gv * uv, 1.0f + e));
-                    }
+                    if (n0 + c + j < n)
+                        *p = unit_bf16(v[j], row[c + j], k, unit);
             }
         }
     }
@@ -240,7 +248,7 @@ template <int BN, int MT, int EPI>
 __global__ void __launch_bounds__(GEMM_THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
                float *__restrict__ out, bf16 *__restrict__ out_act, int n, int m, int k,
-               int second_off, int kb_per_split, int heads)
+               int second_off, int kb_per_split, int heads, const GatedUnit unit)
 {
     using Cfg = TileCfg<BN, MT, EPI == EPI_SWIGLU_HALF>;
     constexpr int STAGES = Cfg::STAGES;
@@ -383,13 +391,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         if (EPI == EPI_SWIGLU_HALF) {
             if constexpr (MT == 1 && BN <= 128)
                 store_swiglu_half<BN>(taddr, q, lane, hgrp, ok, (float *)smem, out_act, m0,
-                                      second_off, n0, n);
+                                      second_off, n0, n, unit);
         } else if (ok) {
             if (EPI == EPI_PARTIAL)
                 store_partial<BN, MT>(taddr, hgrp, out + (size_t)blockIdx.z * n * m, f, n0, n, m,
                                       second_off);
             else
-                store_swiglu<BN>(taddr, hgrp, out_act, f, second_off, n0, n);
+                store_swiglu<BN>(taddr, hgrp, out_act, f, second_off, n0, n, unit);
         }
     }
 
@@ -451,7 +459,8 @@ static bool tensor_map(const void *ptr, int rows, int k, int box_rows, CUtensorM
 
 template <int BN, int MT, int EPI>
 static int launch_tc(const void *A, const void *W, float *out, bf16 *out_act, int n, int m, int k,
-                     int w_rows, int second_off, int splits, cudaStream_t st, int heads = 1)
+                     int w_rows, int second_off, int splits, cudaStream_t st, int heads = 1,
+                     GatedUnit unit = GatedUnit{1.0f, 0.0f, 0.0f})
 {
     using Cfg = TileCfg<BN, MT, EPI == EPI_SWIGLU_HALF>;
     CUtensorMap map_w, map_a;
@@ -472,7 +481,7 @@ static int launch_tc(const void *A, const void *W, float *out, bf16 *out_act, in
     if (grid.y > 65535 || grid.z > 65535)
         return JB_EINVAL;
     launch(kern, grid, GEMM_THREADS, Cfg::SMEM_BYTES, st, map_w, map_a, out, out_act, n, m, k, second_off,
-           kbps, heads);
+           kbps, heads, unit);
     return launch_status();
 }
 
@@ -644,11 +653,19 @@ extern "C" int jb_gemm_tc_heads(const void *A, const void *W, float *out, int n,
 extern "C" int jb_gemm_tc_swiglu(const void *A, const void *W, void *out_act, int n, int ff, int k,
                                  cudaStream_t st)
 {
+    return jb_gemm_tc_gated(A, W, out_act, n, ff, k, 1.0f, 0.0f, 0.0f, st);
+}
+
+// The same with the gated unit's constants (see jb_gated_unit).
+extern "C" int jb_gemm_tc_gated(const void *A, const void *W, void *out_act, int n, int ff, int k, float alpha,
+                                float limit, float shift, cudaStream_t st)
+{
+    const GatedUnit unit{alpha, limit, shift};
     if (!jb_gemm_tc_ok(A, W, n, 2 * ff, k))
         return JB_EINVAL;
     if (n > 128) {
 #define JB_SWIGLU(B)                                                                           \
-    launch_tc<B, 2, EPI_SWIGLU>(A, W, nullptr, (bf16 *)out_act, n, 2 * ff, k, 2 * ff, ff, 1, st)
+    launch_tc<B, 2, EPI_SWIGLU>(A, W, nullptr, (bf16 *)out_act, n, 2 * ff, k, 2 * ff, ff, 1, st, 1, unit)
         switch (many_tokens_tile(n, 2 * ff, k, 1)) {
         case 128: return JB_SWIGLU(128);
         case 160: return JB_SWIGLU(160);
@@ -660,7 +677,7 @@ extern "C" int jb_gemm_tc_swiglu(const void *A, const void *W, void *out_act, in
     }
     // few tokens: as many CTAs as the plain product has (64 gate and 64 up features each)
 #define JB_SWIGLU_HALF(B)                                                                      \
-    launch_tc<B, 1, EPI_SWIGLU_HALF>(A, W, nullptr, (bf16 *)out_act, n, 2 * ff, k, 2 * ff, ff, 1, st)
+    launch_tc<B, 1, EPI_SWIGLU_HALF>(A, W, nullptr, (bf16 *)out_act, n, 2 * ff, k, 2 * ff, ff, 1, st, 1, unit)
     if (n <= 16)
         return JB_SWIGLU_HALF(16);
     if (n <= 32)

@@ -29,6 +29,12 @@
 // q and k heads are divided by their root mean square after the rotation
 #define JB_ROT_PAIRS 1
 #define JB_UNIT_NORM 2
+// a key's sums are its value too (before norm and rotation): the product holds q and k alone
+#define JB_VALUES_FROM_KEYS 4
+// what a router's scores are (jb_moe_route)
+#define JB_SCORE_SOFTMAX 0
+#define JB_SCORE_SIGMOID 1
+#define JB_SCORE_CHOSEN 2
 
 #ifdef __cplusplus
 extern "C" {
@@ -42,6 +48,12 @@ int jb_rmsnorm(float *x, const float *delta, int S, long long delta_stride,
                int dm, float eps, cudaStream_t st);
 int jb_swiglu(const float *gu, int S, long long stride, void *out, int out_dt, int n, int ff,
               cudaStream_t st);
+int jb_gated_unit(const float *gu, int S, long long stride, void *out, int out_dt, int n, int ff,
+                  float alpha, float limit, float shift, cudaStream_t st);
+int jb_join_rows(float *x, const float *delta, int S, long long stride, const float *e, void *out,
+                 int out_dt, int n, int dm, cudaStream_t st);
+int jb_rope_table_scaled(float *cs, float *sn, const float *inv_freq, int n_pos, int half,
+                         double amplitude, cudaStream_t st);
 int jb_rope_table(float *cs, float *sn, const float *inv_freq, int n_pos, int half,
                   cudaStream_t st);
 int jb_qk_norm_rope_append(const float *qkv, int S, long long split_stride, const void *q_w,
@@ -123,12 +135,12 @@ int jb_latent_down_rows(const float *P, int S, long long stride, int ld, int q_c
                         const float *cs, const float *sn, int rot_half, const int32_t *row_pos,
                         const int32_t *row_seq, const int32_t *block_table, int bt_stride,
                         void *cq_out, void *k_cache, void *rows_out, int cache_dt, int n, float eps,
-                        cudaStream_t st);
+                        int halves, cudaStream_t st);
 int jb_gate_rows(const void *a, const float *g, int Sg, long long g_stride, int g_ld, int g_col0,
                  void *out, int dt, int n, int width, cudaStream_t st);
 int jb_latent_q_split(const float *Q, int S, long long stride, int nh, int D, int R, int C,
                       const float *cs, const float *sn, int rot_half, const int32_t *row_pos,
-                      void *q_plain, void *q_lat, int dt, int n, cudaStream_t st);
+                      void *q_plain, void *q_lat, int dt, int n, int halves, int q_ld, cudaStream_t st);
 int jb_latent_q_join(const float *A, int S, int nh, int C, int R, void *q_lat, int dt, int n,
                      cudaStream_t st);
 int jb_heads_gate(const float *A, int S, int nh, int Dv, const float *g, int Sg, long long g_stride,
@@ -155,11 +167,16 @@ int jb_mingru(const float *P, int S, long long stride, int ld, int col0, const f
               float *state, const int32_t *row_seq, const int32_t *seq_slot, float *scratch,
               void *out, int out_dt, int n, int n_seqs, int W, int every_row_starts,
               cudaStream_t st);
-int jb_moe_route(const float *P, int S, long long stride, int ld, int col0, const float *correction,
-                 float *weights, float *skip_coef, int n, int E, int groups, int keep, int top,
-                 int first_identity, float scale, int sigmoid_scores, int group_best, cudaStream_t st);
+int jb_moe_route(const float *P, int S, long long stride, int ld, int col0, const float *bias,
+                 const float *correction, float *weights, float *skip_coef, int n, int E, int groups,
+                 int keep, int top, int first_identity, float scale, int score, int group_best,
+                 cudaStream_t st);
 int jb_gated_weighted(const float *z, int S, long long stride, int ld, const float *weights, int w_ld,
-                      int n_experts, int ff, int kind, void *out, int out_dt, int n, cudaStream_t st);
+                      int n_experts, int ff, int shared_ff, int kind, const float *unit, void *out,
+                      int out_dt, int n, cudaStream_t st);
+int jb_turn_heads(const float *src, int S, long long stride, int ld, int col0, int H, int D, int Dv,
+                  const float *cs, const float *sn, int rot_half, const int32_t *row_pos, float key_scale,
+                  float *out, int n, cudaStream_t st);
 int jb_causal_conv(const float *u, int S, long long stride, int ld, int col0, const float *w,
                    const float *bias, float *state, long long slot_stride, const int32_t *row_pos,
                    const int32_t *row_seq, const int32_t *seq_slot, void *out, int out_dt, int out_ld,
@@ -175,8 +192,8 @@ int jb_matrix_state_piece(void);
 long long jb_matrix_state_scratch(int n_seqs, int max_len, int H, int N, int P);
 int jb_gated_part_norm(const float *y, const float *pre, int pre_S, long long pre_stride, int pre_ld,
                        int pre_col0, const float *post, int post_S, long long post_stride, int post_ld,
-                       int post_col0, const float *w, float eps, void *out, int out_dt, int n, int width,
-                       int parts, int few_rows, cudaStream_t st);
+                       int post_col0, int post_silu, const float *w, float eps, void *out, int out_dt,
+                       int n, int width, int parts, int few_rows, cudaStream_t st);
 int jb_pair_combine(const float *L, int SL, long long strideL, const float *R, int SR, long long strideR,
                     const float *wl, const float *wr, float sl, float sr, float eps, float *out, int n,
                     int m, int few_rows, cudaStream_t st);
@@ -266,6 +283,8 @@ int jb_gemm_tc_heads(const void *A, const void *W, float *out, int n, int m, int
                      int heads, cudaStream_t st);
 int jb_gemm_tc_swiglu(const void *A, const void *W, void *out_act, int n, int ff, int k,
                       cudaStream_t st);
+int jb_gemm_tc_gated(const void *A, const void *W, void *out_act, int n, int ff, int k, float alpha,
+                     float limit, float shift, cudaStream_t st);
 int jb_gemm_tc_error(void);
 int jb_gemm_tc_force_tile(int tokens);
 int jb_gemm_tc_last_tile(void);

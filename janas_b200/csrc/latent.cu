@@ -19,9 +19,9 @@
 //                   [n, H Dv], times sigmoid of a gate's sums
 //   transpose_heads [H, D, C] -> [H, C, D] (a weight, once at load time)
 //
-// The rotation takes pairs (2i, 2i+1) of the first 2 * rot_half values by the
-// angle whose cos and sin the tables hold at [position, i]; what lies beyond
-// passes unchanged.  All sums, norms and angles are float32.
+// The rotation takes pairs of the first 2 * rot_half values, neighbours (2i, 2i+1) or (with
+// halves) value i and value i + rot_half, by the angle whose cos and sin the tables hold at
+// [position, i]; what lies beyond passes unchanged.  All sums, norms and angles are float32.
 #include "common.cuh"
 #include "kernels.h"
 
@@ -37,7 +37,7 @@ latent_down_kernel(const float *__restrict__ P, int S, size_t stride, int ld, in
                    const float *__restrict__ sn, int rot_half, const int32_t *__restrict__ row_pos,
                    const int32_t *__restrict__ row_seq, const int32_t *__restrict__ block_table,
                    int bt_stride, TC *__restrict__ cq_out, TC *__restrict__ k_cache,
-                   TC *__restrict__ rows_out, float eps)
+                   TC *__restrict__ rows_out, float eps, int halves)
 {
     extern __shared__ float buf[];      // q_rank + kv_rank + rot_dim sums of this row
     __shared__ float red[32];
@@ -82,9 +82,11 @@ latent_down_kernel(const float *__restrict__ P, int S, size_t stride, int ld, in
     for (int i = threadIdx.x; i < rot_dim; i += blockDim.x) {
         float v = zr[i];
         if (i < 2 * rot_half) {
-            float c = cs[(size_t)pos * rot_half + i / 2], s = sn[(size_t)pos * rot_half + i / 2];
-            float other = zr[i ^ 1];
-            v = (i & 1) ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
+            int f = halves ? (i < rot_half ? i : i - rot_half) : i / 2;
+            bool high = halves ? i >= rot_half : (i & 1) != 0;
+            float c = cs[(size_t)pos * rot_half + f], s = sn[(size_t)pos * rot_half + f];
+            float other = zr[halves ? (high ? i - rot_half : i + rot_half) : i ^ 1];
+            v = high ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
         }
         dst[kv_rank + i] = from_f<TC>(v);
         if (dst2 != nullptr)
@@ -97,7 +99,7 @@ __global__ void latent_q_split_kernel(const float *__restrict__ Q, int S, size_t
                                       int R, int C, const float *__restrict__ cs,
                                       const float *__restrict__ sn, int rot_half,
                                       const int32_t *__restrict__ row_pos, TC *__restrict__ q_plain,
-                                      TC *__restrict__ q_lat, int n, size_t total)
+                                      TC *__restrict__ q_lat, int n, size_t total, int halves, int q_ld)
 {
     pdl_trigger();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -112,21 +114,27 @@ __global__ void latent_q_split_kernel(const float *__restrict__ Q, int S, size_t
     float v = add_partials(0.0f, Q + i, S, stride);
     if (e < D) {
         // one head's rows together, or (no q_plain) the value's own place in q_lat, whose
-        // rows are then [plain | rotated] and C is D
+        // rows are then [plain | rotated | zeros] and C is D; the plain values' threads write the zeros
         if (q_plain != nullptr)
             q_plain[((size_t)h * n + row) * D + e] = from_f<TC>(v);
         else
-            q_lat[(row * nh + h) * (size_t)(C + R) + e] = from_f<TC>(v);
+            q_lat[(row * nh + h) * (size_t)q_ld + e] = from_f<TC>(v);
+        if (q_plain == nullptr)
+            for (int z = per + e; z < q_ld; z += D)
+                q_lat[(row * nh + h) * (size_t)q_ld + z] = from_f<TC>(0.0f);
         return;
     }
     int r = e - D;
     if (r < 2 * rot_half) {
         // the pair's other value, by its column within the head
-        float other = add_partials(0.0f, Q + (i - e) + D + (r ^ 1), S, stride);
-        float c = cs[(size_t)pos * rot_half + r / 2], s = sn[(size_t)pos * rot_half + r / 2];
-        v = (r & 1) ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
+        int f = halves ? (r < rot_half ? r : r - rot_half) : r / 2;
+        bool high = halves ? r >= rot_half : (r & 1) != 0;
+        int ro = halves ? (high ? r - rot_half : r + rot_half) : r ^ 1;
+        float other = add_partials(0.0f, Q + (i - e) + D + ro, S, stride);
+        float c = cs[(size_t)pos * rot_half + f], s = sn[(size_t)pos * rot_half + f];
+        v = high ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
     }
-    q_lat[(row * nh + h) * (size_t)(C + R) + C + r] = from_f<TC>(v);
+    q_lat[(row * nh + h) * (size_t)q_ld + C + r] = from_f<TC>(v);
 }
 
 // p[0] + p[stride] + ... for four neighbouring values at once
@@ -141,13 +149,14 @@ __device__ __forceinline__ float4 sum4(const float *__restrict__ p, int S, size_
 }
 
 // latent_q_split with four neighbouring values of a head per thread (D, R and C multiples
-// of four: the four lie in the plain or in the rotated part, and hold whole pairs)
+// of four: the four lie in the plain or in the rotated part, and hold whole pairs; with
+// halves rot_half is a multiple of four too, so that a thread's partners are four neighbours)
 template <typename TC>
 __global__ void latent_q_split_vec_kernel(const float *__restrict__ Q, int S, size_t stride, int nh, int D,
                                           int R, int C, const float *__restrict__ cs,
                                           const float *__restrict__ sn, int rot_half,
                                           const int32_t *__restrict__ row_pos, TC *__restrict__ q_plain,
-                                          TC *__restrict__ q_lat, int n, size_t total4)
+                                          TC *__restrict__ q_lat, int n, size_t total4, int halves, int q_ld)
 {
     pdl_trigger();
     size_t i4 = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -165,21 +174,36 @@ __global__ void latent_q_split_vec_kernel(const float *__restrict__ Q, int S, si
         if (q_plain != nullptr)
             store4(q_plain + ((size_t)h * n + row) * D + e, v);
         else
-            store4(q_lat + (row * nh + h) * (size_t)(C + R) + e, v);
+            store4(q_lat + (row * nh + h) * (size_t)q_ld + e, v);
+        if (q_plain == nullptr)
+            for (int z = per + e; z < q_ld; z += D)
+                store4(q_lat + (row * nh + h) * (size_t)q_ld + z, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
         return;
     }
     int r = e - D;
     float o[4] = {v.x, v.y, v.z, v.w};
+    if (halves && r < 2 * rot_half) {
+        bool high = r >= rot_half;
+        int f = high ? r - rot_half : r;
+        float4 w = high ? sum4(Q + i - rot_half, S, stride) : sum4(Q + i + rot_half, S, stride);
+        float4 c = load4(cs + (size_t)pos * rot_half + f), s = load4(sn + (size_t)pos * rot_half + f);
+        if (!high)
+            s = make_float4(-s.x, -s.y, -s.z, -s.w);
+        o[0] = fmaf(v.x, c.x, w.x * s.x);
+        o[1] = fmaf(v.y, c.y, w.y * s.y);
+        o[2] = fmaf(v.z, c.z, w.z * s.z);
+        o[3] = fmaf(v.w, c.w, w.w * s.w);
+    }
 #pragma unroll
     for (int u = 0; u < 4; u += 2) {
-        if (r + u < 2 * rot_half) {
+        if (!halves && r + u < 2 * rot_half) {
             float c = cs[(size_t)pos * rot_half + (r + u) / 2], s = sn[(size_t)pos * rot_half + (r + u) / 2];
             float a = o[u], b = o[u + 1];
             o[u] = fmaf(a, c, -b * s);
             o[u + 1] = fmaf(b, c, a * s);
         }
     }
-    store4(q_lat + (row * nh + h) * (size_t)(C + R) + C + r, make_float4(o[0], o[1], o[2], o[3]));
+    store4(q_lat + (row * nh + h) * (size_t)q_ld + C + r, make_float4(o[0], o[1], o[2], o[3]));
 }
 
 template <typename TC>
@@ -349,18 +373,18 @@ extern "C" int jb_latent_down(const float *P, int S, long long stride, int ld, i
 {
     return jb_latent_down_rows(P, S, stride, ld, q_col0, q_rank, wq, kv_col0, kv_rank, wkv, rot_dim, cs, sn,
                                rot_half, row_pos, row_seq, block_table, bt_stride, cq_out, k_cache,
-                               nullptr, cache_dt, n, eps, st);
+                               nullptr, cache_dt, n, eps, 0, st);
 }
 
 // The same; rows_out (or null): [n, kv_rank + rot_dim], the rows that go to the cache
-// once more, one after the other.
+// once more, one after the other.  halves: the rotation's pairs are (i, i + rot_half).
 extern "C" int jb_latent_down_rows(const float *P, int S, long long stride, int ld, int q_col0,
                                    int q_rank, const float *wq, int kv_col0, int kv_rank,
                                    const float *wkv, int rot_dim, const float *cs, const float *sn,
                                    int rot_half, const int32_t *row_pos, const int32_t *row_seq,
                                    const int32_t *block_table, int bt_stride, void *cq_out,
                                    void *k_cache, void *rows_out, int cache_dt, int n, float eps,
-                                   cudaStream_t st)
+                                   int halves, cudaStream_t st)
 {
     if (n <= 0)
         return JB_OK;
@@ -375,7 +399,7 @@ extern "C" int jb_latent_down_rows(const float *P, int S, long long stride, int 
 #define JB_LD(TC, ONE)                                                                          \
     launch(latent_down_kernel<TC, ONE>, n, 256, smem, st, P, S, (size_t)stride, ld, q_col0, q_rank, wq, \
            kv_col0, kv_rank, wkv, rot_dim, cs, sn, rot_half, row_pos, row_seq, block_table,      \
-           bt_stride, (TC *)cq_out, (TC *)k_cache, (TC *)rows_out, eps)
+           bt_stride, (TC *)cq_out, (TC *)k_cache, (TC *)rows_out, eps, halves)
     if (cache_dt == JB_F32 && S == 1)
         JB_LD(float, true);
     else if (cache_dt == JB_F32)
@@ -391,38 +415,41 @@ extern "C" int jb_latent_down_rows(const float *P, int S, long long stride, int 
 }
 
 // Q: the query product's sums [S, n, nh (D + R)].  q_plain: [nh, n, D]; q_lat:
-// [n, nh, C + R], of which columns C.. are written here.
+// [n, nh, C + R], of which columns C.. are written here.  Without q_plain whole queries [plain |
+// rotated] go to q_lat (C = D), its rows q_ld >= D + R long and zero past D + R.  halves: as above.
 extern "C" int jb_latent_q_split(const float *Q, int S, long long stride, int nh, int D, int R, int C,
                                  const float *cs, const float *sn, int rot_half,
                                  const int32_t *row_pos, void *q_plain, void *q_lat, int dt, int n,
-                                 cudaStream_t st)
+                                 int halves, int q_ld, cudaStream_t st)
 {
     size_t total = (size_t)n * nh * (D + R);
     if (total == 0)
         return JB_OK;
-    if (S <= 0 || D <= 0 || R < 0 || C <= 0 || 2 * rot_half > R ||
+    if (S <= 0 || D <= 0 || R < 0 || C <= 0 || 2 * rot_half > R || q_ld < C + R ||
+        (q_plain != nullptr && q_ld != C + R) ||
         (rot_half > 0 && (cs == nullptr || sn == nullptr)))
         return JB_EINVAL;
     size_t esz = dt == JB_F32 ? 4 : 2;
-    if (D % 4 == 0 && R % 4 == 0 && C % 4 == 0 && stride % 4 == 0 && (uintptr_t)Q % 16 == 0 &&
+    if (D % 4 == 0 && R % 4 == 0 && C % 4 == 0 && q_ld % 4 == 0 && stride % 4 == 0 && (uintptr_t)Q % 16 == 0 &&
+        (!halves || (rot_half % 4 == 0 && (uintptr_t)cs % 16 == 0 && (uintptr_t)sn % 16 == 0)) &&
         (uintptr_t)q_plain % (4 * esz) == 0 && (uintptr_t)q_lat % (4 * esz) == 0 && (dt == JB_F32 || dt == JB_BF16)) {
         size_t total4 = total / 4;
         unsigned vb = (unsigned)((total4 + 255) / 256);
         if (dt == JB_F32)
             launch(latent_q_split_vec_kernel<float>, vb, 256, 0, st, Q, S, (size_t)stride, nh, D, R, C, cs, sn,
-                   rot_half, row_pos, (float *)q_plain, (float *)q_lat, n, total4);
+                   rot_half, row_pos, (float *)q_plain, (float *)q_lat, n, total4, halves, q_ld);
         else
             launch(latent_q_split_vec_kernel<bf16>, vb, 256, 0, st, Q, S, (size_t)stride, nh, D, R, C, cs, sn,
-                   rot_half, row_pos, (bf16 *)q_plain, (bf16 *)q_lat, n, total4);
+                   rot_half, row_pos, (bf16 *)q_plain, (bf16 *)q_lat, n, total4, halves, q_ld);
         return launch_status();
     }
     unsigned blocks = (unsigned)((total + 255) / 256);
     if (dt == JB_F32)
         launch(latent_q_split_kernel<float>, blocks, 256, 0, st, Q, S, (size_t)stride, nh, D, R, C, cs, sn,
-               rot_half, row_pos, (float *)q_plain, (float *)q_lat, n, total);
+               rot_half, row_pos, (float *)q_plain, (float *)q_lat, n, total, halves, q_ld);
     else if (dt == JB_BF16)
         launch(latent_q_split_kernel<bf16>, blocks, 256, 0, st, Q, S, (size_t)stride, nh, D, R, C, cs, sn,
-               rot_half, row_pos, (bf16 *)q_plain, (bf16 *)q_lat, n, total);
+               rot_half, row_pos, (bf16 *)q_plain, (bf16 *)q_lat, n, total, halves, q_ld);
     else
         return JB_EINVAL;
     return launch_status();

@@ -208,21 +208,23 @@ Buf moe_route(Device &d, const Stack &P, long long col0, const RouteParams &r, B
     if (P.m < col0 + r.experts) fail(JB_LLM_EINVAL, "moe_route: the product is narrower than the router's rows");
     Buf weights = d.pool.get(std::max<size_t>((size_t)P.n * (size_t)r.experts * 4, 16));
     if (skip_coef) *skip_coef = d.pool.get(std::max<size_t>((size_t)P.n * 4, 16));
-    check(jb_moe_route(P.data(), P.S, P.stride(), as_int(P.m, "width"), (int)col0, r.correction,
+    check(jb_moe_route(P.data(), P.S, P.stride(), as_int(P.m, "width"), (int)col0, r.bias, r.correction,
                        weights.as<float>(), skip_coef ? skip_coef->as<float>() : nullptr, as_int(P.n, "rows"),
-                       r.experts, r.groups, r.keep, r.top, r.first_identity, r.scale, r.sigmoid_scores ? 1 : 0,
+                       r.experts, r.groups, r.keep, r.top, r.first_identity, r.scale, r.score,
                        r.group_best, d.stream), "moe_route");
     return weights;
 }
 
 Buf gated_weighted(Device &d, const Stack &z, const float *weights, int w_ld, int n_experts, long long ff,
-                   int kind, DType out_dt) {
+                   int kind, DType out_dt, long long shared_ff, UnitParams unit, UnitParams shared_unit) {
     need_float(out_dt, "activation output");
-    long long width = (long long)n_experts * ff;
+    long long width = (long long)n_experts * ff + shared_ff;
     if (width <= 0 || 2 * width > z.m) fail(JB_LLM_EINVAL, "gated_weighted: the product is narrower than the experts");
     Buf out = d.pool.get((size_t)z.n * (size_t)width * dtype_size(out_dt));
+    const float u[6] = {unit.alpha, unit.limit, unit.shift, shared_unit.alpha, shared_unit.limit, shared_unit.shift};
     check(jb_gated_weighted(z.data(), z.S, z.stride(), as_int(z.m, "width"), weights, w_ld, n_experts,
-                            as_int(ff, "width"), kind, out.ptr, out_dt, as_int(z.n, "rows"), d.stream),
+                            as_int(ff, "width"), as_int(shared_ff, "width"), kind, kind == JB_ACT_SILU ? u : nullptr,
+                            out.ptr, out_dt, as_int(z.n, "rows"), d.stream),
           "gated_weighted");
     return out;
 }
@@ -265,15 +267,29 @@ Buf matrix_state_scan(Device &d, const Stack &src, const MatrixScan &m, float *s
 
 Buf gated_part_norm(Device &d, const float *y, long long n, long long width, int parts, const Stack *pre,
                     long long pre_col0, const Stack *post, long long post_col0, const float *w, float eps,
-                    DType out_dt, bool few_rows) {
+                    DType out_dt, bool few_rows, bool post_silu) {
     need_float(out_dt, "gated_part_norm output");
     if ((pre && pre->n != n) || (post && post->n != n)) fail(JB_LLM_EINVAL, "gated_part_norm: a gate of other rows");
     Buf out = d.pool.get(std::max<size_t>((size_t)n * (size_t)width * dtype_size(out_dt), 16));
     check(jb_gated_part_norm(y, pre ? pre->data() : nullptr, pre ? pre->S : 0, pre ? pre->stride() : 0,
                              pre ? as_int(pre->m, "width") : 0, (int)pre_col0, post ? post->data() : nullptr,
                              post ? post->S : 0, post ? post->stride() : 0, post ? as_int(post->m, "width") : 0,
-                             (int)post_col0, w, eps, out.ptr, out_dt, as_int(n, "rows"), as_int(width, "width"),
-                             parts, few_rows ? 1 : 0, d.stream), "gated_part_norm");
+                             (int)post_col0, post_silu ? 1 : 0, w, eps, out.ptr, out_dt, as_int(n, "rows"),
+                             as_int(width, "width"), parts, few_rows ? 1 : 0, d.stream), "gated_part_norm");
+    return out;
+}
+
+Stack turn_heads(Device &d, const Stack &src, long long col0, int H, long long D, long long Dv, const float *cs,
+                 const float *sn, int rot_half, const int32_t *row_pos, float key_scale) {
+    Stack out;
+    out.S = 1;
+    out.n = src.n;
+    out.m = (long long)H * (2 * D + Dv);
+    if (!src || col0 < 0 || col0 + out.m > src.m) fail(JB_LLM_EINVAL, "turn_heads: the columns lie outside the product");
+    out.buf = d.pool.get(std::max<size_t>((size_t)out.n * (size_t)out.m * 4, 16));
+    check(jb_turn_heads(src.data(), src.S, src.stride(), as_int(src.m, "width"), (int)col0, H, as_int(D, "width"),
+                        as_int(Dv, "width"), cs, sn, rot_half, row_pos, key_scale, out.data(), as_int(src.n, "rows"),
+                        d.stream), "turn_heads");
     return out;
 }
 
@@ -317,9 +333,12 @@ Buf activation_weighted(Device &d, const Stack &z, long long width, const float 
 Buf qkv_prepare_append(Device &d, const Stack &qkv, const float *bias, const float *q_w, const float *k_w,
                        float eps, const float *cos, const float *sin, int rot_half, const int32_t *row_pos,
                        const int32_t *row_seq, const AttnCache &c, const AttnGeometry &g, DType out_dt,
-                       bool pairs, bool unit_norm) {
+                       bool pairs, bool unit_norm, bool values_from_keys) {
     bool append = c.writes;
-    long long width = (long long)g.nh * g.hd + (append ? (long long)g.nkv * (g.hd + g.value_dim()) : 0);
+    if (values_from_keys && (!append || g.value_dim() != g.hd))
+        fail(JB_LLM_EINVAL, "qkv_prepare_append: values that are the keys need a cache of their own and the keys' size");
+    long long width = (long long)g.nh * g.hd +
+                      (append ? (long long)g.nkv * (g.hd + (values_from_keys ? 0 : g.value_dim())) : 0);
     if (qkv.m < width) fail(JB_LLM_EINVAL, "qkv_prepare_append: the product is narrower than q, k and v");
     if (append && (!c.k || !c.v)) fail(JB_LLM_EINVAL, "qkv_prepare_append: no cache to append to");
     if (append && c.dt != out_dt) fail(JB_LLM_EINVAL, "qkv_prepare_append: the cache is of another type");
@@ -328,7 +347,8 @@ Buf qkv_prepare_append(Device &d, const Stack &qkv, const float *bias, const flo
                                 sin, rot_half, row_pos, row_seq, c.block_table, c.bt_stride, q.ptr,
                                 append ? c.k : nullptr, append ? c.v : nullptr, out_dt, as_int(qkv.n, "rows"),
                                 g.nh, g.nkv, g.hd, g.value_dim(),
-                                (pairs ? JB_ROT_PAIRS : 0) | (unit_norm ? JB_UNIT_NORM : 0), d.stream),
+                                (pairs ? JB_ROT_PAIRS : 0) | (unit_norm ? JB_UNIT_NORM : 0) |
+                                    (values_from_keys ? JB_VALUES_FROM_KEYS : 0), d.stream),
           "qkv_prepare_append");
     return q;
 }
@@ -356,7 +376,7 @@ Buf activation(Device &d, const Stack &z, long long ff, int kind, DType out_dt, 
 Buf latent_down(Device &d, const Stack &P, long long q_col0, long long q_rank, const float *wq,
                 long long kv_col0, long long kv_rank, const float *wkv, long long rot_dim, const float *cs,
                 const float *sn, int rot_half, const int32_t *row_pos, const int32_t *row_seq,
-                const AttnCache &c, float eps, DType out_dt, Buf *rows_out) {
+                const AttnCache &c, float eps, DType out_dt, Buf *rows_out, bool halves) {
     if (!c.k || !c.writes) fail(JB_LLM_EINVAL, "latent_down: no cache to write the latent to");
     if (c.dt != out_dt) fail(JB_LLM_EINVAL, "latent_down: the cache is of another type");
     Buf cq = d.pool.get(std::max<size_t>((size_t)P.n * (size_t)q_rank * dtype_size(out_dt), 16));
@@ -365,20 +385,22 @@ Buf latent_down(Device &d, const Stack &P, long long q_col0, long long q_rank, c
                               (int)kv_col0, (int)kv_rank, wkv, (int)rot_dim, cs, sn, rot_half, row_pos,
                               row_seq, c.block_table, c.bt_stride, cq.ptr, c.k,
                               rows_out ? rows_out->ptr : nullptr, out_dt, as_int(P.n, "rows"), eps,
-                              d.stream), "latent_down");
+                              halves ? 1 : 0, d.stream), "latent_down");
     return cq;
 }
 
 Buf latent_q_split(Device &d, const Stack &Q, int nh, long long D, long long R, long long C, const float *cs,
                    const float *sn, int rot_half, const int32_t *row_pos, void *q_lat, DType dt,
-                   bool plain_head_major) {
+                   bool plain_head_major, bool halves, int row_len) {
     if (Q.m != (long long)nh * (D + R)) fail(JB_LLM_EINVAL, "latent_q_split: the product is not heads x (plain + rotated) wide");
     if (!plain_head_major && C != D) fail(JB_LLM_EINVAL, "latent_q_split: whole queries have their plain part first");
+    if (row_len == 0 || plain_head_major) row_len = (int)(C + R);
+    if (row_len < C + R) fail(JB_LLM_EINVAL, "latent_q_split: a query does not fit its row");
     resolve_bias(d, const_cast<Stack &>(Q));
     Buf qp;
     if (plain_head_major) qp = d.pool.get((size_t)nh * (size_t)Q.n * (size_t)D * dtype_size(dt));
     check(jb_latent_q_split(Q.data(), Q.S, Q.stride(), nh, (int)D, (int)R, (int)C, cs, sn, rot_half, row_pos,
-                            qp.ptr, q_lat, dt, as_int(Q.n, "rows"), d.stream), "latent_q_split");
+                            qp.ptr, q_lat, dt, as_int(Q.n, "rows"), halves ? 1 : 0, row_len, d.stream), "latent_q_split");
     return qp;
 }
 
@@ -477,17 +499,28 @@ void add_(Device &d, float *x, long long n, long long dm, const Stack &delta) {
                      as_int(n, "rows"), as_int(dm, "width"), 0.0f, d.stream), "add");
 }
 
-Buf swiglu(Device &d, const Stack &gu, DType out_dt) {
-    if (gu.m % 2) fail(JB_LLM_EINVAL, "swiglu: the gate_up width must be even");
-    long long ff = gu.m / 2;
-    Buf out = d.pool.get((size_t)gu.n * (size_t)ff * dtype_size(out_dt));
-    check(jb_swiglu(gu.data(), gu.S, gu.stride(), out.ptr, out_dt, as_int(gu.n, "rows"), as_int(ff, "width"),
-                    d.stream), "swiglu");
+Buf join_rows(Device &d, float *x, long long n, long long dm, const Stack *delta, const float *e, DType out_dt) {
+    need_float(out_dt, "join_rows output");
+    if (delta && (delta->n != n || delta->m != dm)) fail(JB_LLM_EINVAL, "join_rows: delta's shape is not x's");
+    if (delta) resolve_bias(d, const_cast<Stack &>(*delta));
+    Buf out = d.pool.get(std::max<size_t>((size_t)n * (size_t)(2 * dm) * dtype_size(out_dt), 16));
+    check(jb_join_rows(x, delta ? delta->data() : nullptr, delta ? delta->S : 0, delta ? delta->stride() : 0, e,
+                       out.ptr, out_dt, as_int(n, "rows"), as_int(dm, "width"), d.stream), "join_rows");
     return out;
 }
 
-void rope_table(Device &d, const float *inv, int half, long long n_pos, float *cs, float *sn) {
-    check(jb_rope_table(cs, sn, inv, as_int(n_pos, "positions"), half, d.stream), "rope_table");
+Buf swiglu(Device &d, const Stack &gu, DType out_dt, UnitParams unit) {
+    if (gu.m % 2) fail(JB_LLM_EINVAL, "swiglu: the gate_up width must be even");
+    long long ff = gu.m / 2;
+    Buf out = d.pool.get((size_t)gu.n * (size_t)ff * dtype_size(out_dt));
+    check(jb_gated_unit(gu.data(), gu.S, gu.stride(), out.ptr, out_dt, as_int(gu.n, "rows"), as_int(ff, "width"),
+                        unit.alpha, unit.limit, unit.shift, d.stream), "swiglu");
+    return out;
+}
+
+void rope_table(Device &d, const float *inv, int half, long long n_pos, float *cs, float *sn,
+                double amplitude) {
+    check(jb_rope_table_scaled(cs, sn, inv, as_int(n_pos, "positions"), half, amplitude, d.stream), "rope_table");
 }
 
 // ------------------------------------------------------------------ products
@@ -556,7 +589,8 @@ HeadStack linear_heads(Device &d, const void *a, DType a_dt, int H, long long n,
     return out;
 }
 
-Buf linear_swiglu(Device &d, const void *a, DType a_dt, long long n, long long k, const DevTensor &gu) {
+Buf linear_swiglu(Device &d, const void *a, DType a_dt, long long n, long long k, const DevTensor &gu,
+                  UnitParams unit) {
     if (gu.shape.size() != 2 || gu.shape[1] != k)
         fail(JB_LLM_EINVAL, "linear_swiglu: the weight's rows are not as long as the activations'");
     if (gu.shape[0] % 2 || n == 0 || a_dt != BF16 || gu.dt != BF16 ||
@@ -564,8 +598,8 @@ Buf linear_swiglu(Device &d, const void *a, DType a_dt, long long n, long long k
         return Buf();
     long long ff = gu.shape[0] / 2;
     Buf out = d.pool.get((size_t)n * (size_t)ff * 2);
-    check(jb_gemm_tc_swiglu(a, gu.ptr, out.ptr, as_int(n, "rows"), as_int(ff, "features"), as_int(k, "width"),
-                            d.stream), "linear_swiglu (tcgen05)");
+    check(jb_gemm_tc_gated(a, gu.ptr, out.ptr, as_int(n, "rows"), as_int(ff, "features"), as_int(k, "width"),
+                           unit.alpha, unit.limit, unit.shift, d.stream), "linear_swiglu (tcgen05)");
     return out;
 }
 

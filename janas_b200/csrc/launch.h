@@ -114,6 +114,12 @@ Buf short_conv(Device &d, const float *x, long long n, long long dm, const float
 Buf mingru(Device &d, const Stack &P, long long col0, long long W, const float *bias, float *state,
            const int32_t *row_seq, const int32_t *seq_slot, int n_seqs, bool every_row_starts, DType out_dt);
 
+// A gated unit's constants: gate sigmoid(alpha gate) (up + shift), with limit > 0 the gate cut off
+// above limit and the up side on both sides first; the default is SiLU(gate) * up.
+struct UnitParams {
+    float alpha = 1.0f, limit = 0.0f, shift = 0.0f;
+};
+
 // The router of a routed feed-forward (csrc/moe.cu): weights [n, E] float32 (0 for experts
 // not chosen) and, with skip_coef, the summed weight of the chosen experts from
 // first_identity on.
@@ -121,7 +127,10 @@ struct RouteParams {
     int experts = 0, groups = 1, keep = 1, top = 1, first_identity = 0;
     float scale = 1.0f;
     const float *correction = nullptr;
-    bool sigmoid_scores = false;      // each score the sigmoid of its logit, instead of a softmax over all
+    // what the scores are: JB_SCORE_SOFTMAX, a softmax over all; JB_SCORE_SIGMOID, each the sigmoid of
+    // its logit; JB_SCORE_CHOSEN, the logits, with a softmax over the chosen ones as their weights
+    int score = 0;
+    const float *bias = nullptr;      // float32 [experts], added to the logits
     int group_best = 1;               // a group's score: the sum of this many of its largest choices
 };
 Buf moe_route(Device &d, const Stack &P, long long col0, const RouteParams &r, Buf *skip_coef);
@@ -131,9 +140,11 @@ Buf activation_weighted(Device &d, const Stack &z, long long width, const float 
                         long long ff, int kind, DType out_dt);
 
 // The same for experts with a gate: per expert [gate (ff) | up (ff)] in z's columns;
-// act(gate) * up * weights[row, expert] as [n, n_experts ff] in out_dt.
+// act(gate) * up * weights[row, expert] (silu: the gated unit), then the shared expert's shared_ff
+// values from the columns after the experts', without a weight: [n, n_experts ff + shared_ff] in out_dt.
 Buf gated_weighted(Device &d, const Stack &z, const float *weights, int w_ld, int n_experts, long long ff,
-                   int kind, DType out_dt);
+                   int kind, DType out_dt, long long shared_ff = 0, UnitParams unit = UnitParams(),
+                   UnitParams shared_unit = UnitParams());
 
 // A causal convolution over time on C columns (from col0) of a product's sums u, without
 // the input added: act(bias + sum_j w[:, j] u_{t - taps + 1 + j}) as [n, C] in out_dt (act:
@@ -161,12 +172,17 @@ struct MatrixScan {
 Buf matrix_state_scan(Device &d, const Stack &src, const MatrixScan &m, float *state, long long slot_stride,
                       const int32_t *row_seq, const int32_t *seq_slot, int n_seqs, bool every_row_starts,
                       long long max_len = 0);
-// rms(y * silu(pre)) in `parts` equal parts of the row, times w, times sigmoid(post): y float32
-// [n, width]; pre / post: sums whose columns from pre_col0 / post_col0 are read (null: none).
+// A linear attention's q, k and v ahead of its recurrence: [q | k | v] (H D, H D and H Dv columns from
+// col0 of the sums) as one float32 stack, the first 2 rot_half values of every q and k head turned
+// (value i with value i + rot_half), k times key_scale.
+Stack turn_heads(Device &d, const Stack &src, long long col0, int H, long long D, long long Dv, const float *cos,
+                 const float *sin, int rot_half, const int32_t *row_pos, float key_scale);
+// rms(y * silu(pre)) in `parts` equal parts of the row, times w (null: 1), times sigmoid(post)
+// (post_silu: silu(post)): y float32 [n, width]; pre / post: sums whose columns from pre_col0 / post_col0 are read (null: none).
 // few_rows: the bfloat16 path's kernel for a decode step's rows (a cluster of CTAs per row and part).
 Buf gated_part_norm(Device &d, const float *y, long long n, long long width, int parts, const Stack *pre,
                     long long pre_col0, const Stack *post, long long post_col0, const float *w, float eps,
-                    DType out_dt, bool few_rows = false);
+                    DType out_dt, bool few_rows = false, bool post_silu = false);
 // Two results as one stack of one sum: sl * sum(L) + sr * sum(R), or with weights (float32
 // [m] each) sl * rms(sum L) wl + sr * rms(sum R) wr.
 // few_rows: the bfloat16 path's kernel for a decode step's rows (a cluster of CTAs per row).
@@ -186,12 +202,16 @@ void add_(Device &d, float *x, long long n, long long dm, const Stack &delta);
 // y[r, :] += bias for every row of y (float32 [n, m])
 void add_bias_(Device &d, float *y, long long n, long long m, const float *bias);
 
-// SiLU(gate) * up for a stack [S, n, 2 ff] whose columns are [gate | up]
-Buf swiglu(Device &d, const Stack &gate_up, DType out_dt);
+// x becomes [x + sum(delta) | e] (delta: what is still to be added, or null) as [n, 2 dm] in out_dt;
+// x itself is left at zero
+Buf join_rows(Device &d, float *x, long long n, long long dm, const Stack *delta, const float *e, DType out_dt);
 
-// cos and sin of (float)p * inv_freq[i] for p < n_pos: two float32 [n_pos, half]
+// SiLU(gate) * up, or another gated unit, for a stack [S, n, 2 ff] whose columns are [gate | up]
+Buf swiglu(Device &d, const Stack &gate_up, DType out_dt, UnitParams unit = UnitParams());
+
+// cos and sin of (float)p * inv_freq[i] for p < n_pos, times amplitude: two float32 [n_pos, half]
 void rope_table(Device &d, const float *inv_freq_dev, int half, long long n_pos, float *cos_out,
-                float *sin_out);
+                float *sin_out, double amplitude = 1.0);
 
 // a [n, k] . weight[m, k]^T as a stack of float32 partial sums.  bfloat16 operands
 // whose rows are a multiple of 8 long go to the tensor-core kernel (which may cut
@@ -214,7 +234,7 @@ int linear_parts(long long n, long long m, long long k);
 // SiLU(a . gate^T) * (a . up^T) in one tensor-core kernel; an empty Buf when the
 // kernel does not take the operands.  Output bfloat16 [n, ff].
 Buf linear_swiglu(Device &d, const void *a, DType a_dt, long long n, long long k,
-                  const DevTensor &gate_up);
+                  const DevTensor &gate_up, UnitParams unit = UnitParams());
 
 struct AttnGeometry {
     int nh = 0, nkv = 0, hd = 0, window = 0;
@@ -261,15 +281,18 @@ Buf qkv_bias_append(Device &d, const Stack &qkv, const float *bias, const int32_
 // The element-wise steps of latent attention (csrc/latent.cu).  P: the down products'
 // sums; the RMS-normed query latent [n, q_rank] comes back in out_dt, the row
 // [RMS-normed latent | rotated shared key part] goes to the cache at each row's position.
+// halves: the rotation's pairs are (i, i + rot_half) instead of neighbours.
 Buf latent_down(Device &d, const Stack &P, long long q_col0, long long q_rank, const float *wq,
                 long long kv_col0, long long kv_rank, const float *wkv, long long rot_dim,
                 const float *cos, const float *sin, int rot_half, const int32_t *row_pos,
-                const int32_t *row_seq, const AttnCache &c, float eps, DType out_dt, Buf *rows_out = nullptr);
+                const int32_t *row_seq, const AttnCache &c, float eps, DType out_dt, Buf *rows_out = nullptr,
+                bool halves = false);
 // Q: the query product's sums [S, n, nh (D + R)] -> the plain parts [nh, n, D] (returned)
-// and the rotated parts in columns C.. of q_lat [n, nh, C + R]
+// and the rotated parts in columns C.. of q_lat [n, nh, C + R].  Without plain_head_major whole queries
+// [plain | rotated] go to q_lat, whose rows are row_len long (0: D + R) and are zeros past D + R.
 Buf latent_q_split(Device &d, const Stack &Q, int nh, long long D, long long R, long long C,
                    const float *cos, const float *sin, int rot_half, const int32_t *row_pos,
-                   void *q_lat, DType dt, bool plain_head_major = true);
+                   void *q_lat, DType dt, bool plain_head_major = true, bool halves = false, int row_len = 0);
 // A product that holds keys and values alone, [k | v] per row: into the cache pages at
 // the rows' positions (c.k, c.v, c.block_table; kv_heads heads of hd and vd values).
 void kv_append(Device &d, const Stack &kv, const int32_t *row_pos, const int32_t *row_seq,
@@ -289,11 +312,12 @@ DevTensor transpose_heads(Device &d, const DevTensor &w, int H);
 // values of a head, K and V (of their own head size) into the cache.  Returns q [n, heads, hd].
 // pairs: the rotation turns neighbours (2i, 2i + 1) by angle i instead of (i, i + rot_half);
 // unit_norm: q and k heads are divided by their root mean square (eps inside the root)
-// after the rotation, without a weight.
+// after the rotation, without a weight; values_from_keys: the product holds q and k alone, and a
+// key's sums, before any norm and rotation, are its value.
 Buf qkv_prepare_append(Device &d, const Stack &qkv, const float *bias, const float *q_w, const float *k_w,
                        float eps, const float *cos, const float *sin, int rot_half, const int32_t *row_pos,
                        const int32_t *row_seq, const AttnCache &c, const AttnGeometry &g, DType out_dt,
-                       bool pairs = false, bool unit_norm = false);
+                       bool pairs = false, bool unit_norm = false, bool values_from_keys = false);
 // chunks that the kept first tokens of a windowed mixer add to a row's range
 int attention_kept_chunks(int window, int keep_first);
 

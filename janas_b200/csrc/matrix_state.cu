@@ -360,15 +360,15 @@ matrix_state_carry_kernel(float *__restrict__ state, size_t slot_stride, const i
 }
 
 // out[r, c] = rms_part(y[r, :] * pre)[c] * w[c] * post, where pre = silu of the sums in
-// columns pre_col0.. of `pre` (null: 1), post = sigmoid of the sums in columns post_col0..
-// of `post` (null: 1), and the row is normed in `parts` equal parts, each by its own root
+// columns pre_col0.. of `pre` (null: 1), post = sigmoid (post_silu: silu) of the sums in columns
+// post_col0.. of `post` (null: 1), w null is a weight of 1, and the row is normed in `parts` equal parts, each by its own root
 // mean square.  A block per (row, part).
 template <typename TO>
 __global__ void __launch_bounds__(256)
 gated_part_norm_kernel(const float *__restrict__ y, const float *__restrict__ pre, int pre_S, size_t pre_stride,
                        int pre_ld, int pre_col0, const float *__restrict__ post, int post_S, size_t post_stride,
                        int post_ld, int post_col0, const float *__restrict__ w, float eps, TO *__restrict__ out,
-                       int width, int parts, int keep)
+                       int width, int parts, int keep, int post_silu)
 {
     extern __shared__ float held[];          // the part's gated values, where they fit (keep != 0)
     __shared__ float red[32];
@@ -395,11 +395,139 @@ gated_part_norm_kernel(const float *__restrict__ y, const float *__restrict__ pr
             if (pre != nullptr)
                 v *= silu_f(add_partials(0.0f, pre + (size_t)r * pre_ld + pre_col0 + c, pre_S, pre_stride));
         }
-        v = (v * scale) * w[c];
-        if (post != nullptr)
-            v *= sigmoid_f(add_partials(0.0f, post + (size_t)r * post_ld + post_col0 + c, post_S, post_stride));
+        v *= scale;
+        if (w != nullptr)
+            v *= w[c];
+        if (post != nullptr) {
+            float g = add_partials(0.0f, post + (size_t)r * post_ld + post_col0 + c, post_S, post_stride);
+            v *= post_silu ? silu_f(g) : sigmoid_f(g);
+        }
         out[(size_t)r * width + c] = from_f<TO>(v);
     }
+}
+
+// The same for short parts (a head's values each): a warp per (row, part), four neighbouring values
+// a lane and up to U of those; lengths, columns and rows are multiples of four.
+template <typename TO, int U>
+__global__ void __launch_bounds__(256)
+gated_part_norm_warp_kernel(const float *__restrict__ y, const float *__restrict__ pre, int pre_S, size_t pre_stride,
+                            int pre_ld, int pre_col0, const float *__restrict__ post, int post_S, size_t post_stride,
+                            int post_ld, int post_col0, const float *__restrict__ w, float eps, TO *__restrict__ out,
+                            int width, int parts, int post_silu, unsigned tasks)
+{
+    pdl_trigger();
+    unsigned task = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (task >= tasks)
+        return;
+    int lane = threadIdx.x & 31;
+    unsigned r = task / parts;
+    int len = width / parts, c0 = (int)(task - r * parts) * len;
+    auto sums4 = [](const float *p, int S, size_t stride) {
+        float4 v = load4(p);
+        for (int k = 1; k < S; k++) {
+            float4 t = load4(p + (size_t)k * stride);
+            v = make_float4(v.x + t.x, v.y + t.y, v.z + t.z, v.w + t.w);
+        }
+        return v;
+    };
+    pdl_wait();
+    float4 v[U], g[U];
+    float ss = 0.0f;
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+        int c = c0 + 4 * (lane + 32 * u);
+        v[u] = g[u] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (c >= c0 + len)
+            continue;
+        v[u] = load4(y + (size_t)r * width + c);
+        if (post != nullptr)
+            g[u] = sums4(post + (size_t)r * post_ld + post_col0 + c, post_S, post_stride);
+        if (pre != nullptr) {
+            float4 t = sums4(pre + (size_t)r * pre_ld + pre_col0 + c, pre_S, pre_stride);
+            v[u] = make_float4(v[u].x * silu_f(t.x), v[u].y * silu_f(t.y), v[u].z * silu_f(t.z), v[u].w * silu_f(t.w));
+        }
+        ss = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, fmaf(v[u].z, v[u].z, fmaf(v[u].w, v[u].w, ss))));
+    }
+    ss = warp_sum(ss);
+    float scale = 1.0f / sqrtf(ss / (float)len + eps);
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+        int c = c0 + 4 * (lane + 32 * u);
+        if (c >= c0 + len)
+            continue;
+        float4 o = make_float4(v[u].x * scale, v[u].y * scale, v[u].z * scale, v[u].w * scale);
+        if (w != nullptr) {
+            float4 t = load4(w + c);
+            o = make_float4(o.x * t.x, o.y * t.y, o.z * t.z, o.w * t.w);
+        }
+        if (post != nullptr) {
+            if (post_silu)
+                o = make_float4(o.x * silu_f(g[u].x), o.y * silu_f(g[u].y), o.z * silu_f(g[u].z), o.w * silu_f(g[u].w));
+            else
+                o = make_float4(o.x * sigmoid_f(g[u].x), o.y * sigmoid_f(g[u].y), o.z * sigmoid_f(g[u].z),
+                                o.w * sigmoid_f(g[u].w));
+        }
+        store4(out + (size_t)r * width + c, o);
+    }
+}
+
+// q, k and v of a linear attention ahead of its recurrence, float32: out[r] = [q | k | v] from the
+// sums' columns col0 .. (H D, H D and H Dv values), with the first 2 rot_half values of every q and
+// k head turned (value i with value i + rot_half, angle tables [position, i]) and k times key_scale
+// after that.  VEC values per thread: 4 where D, Dv and rot_half are multiples of four and
+// everything lies on 16-byte boundaries.
+template <int VEC>
+__global__ void __launch_bounds__(256)
+turn_heads_kernel(const float *__restrict__ src, int S, size_t stride, int ld, int col0, int H, int D, int Dv,
+                  const float *__restrict__ cs, const float *__restrict__ sn, int rot_half,
+                  const int32_t *__restrict__ row_pos, float key_scale, float *__restrict__ out, int width)
+{
+    pdl_trigger();
+    int r = blockIdx.x, c = (int)(blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    if (c >= width)
+        return;
+    int d = c < 2 * H * D ? c % D : 2 * rot_half;          // v is not turned
+    bool turned = d < 2 * rot_half, high = d >= rot_half;
+    float f = c >= H * D && c < 2 * H * D ? key_scale : 1.0f;
+    float co[VEC], si[VEC];
+    if (turned) {
+        size_t at = (size_t)row_pos[r] * rot_half + (high ? d - rot_half : d);
+#pragma unroll
+        for (int u = 0; u < VEC; u++) {
+            co[u] = cs[at + u];
+            si[u] = high ? sn[at + u] : -sn[at + u];
+        }
+    }
+    pdl_wait();
+    const float *p = src + (size_t)r * ld + col0 + c, *o = p + (high ? -rot_half : rot_half);
+    float v[VEC], w[VEC];
+    if (VEC == 4) {
+        float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f), b = a;
+        for (int k = 0; k < S; k++) {
+            float4 t = load4(p + (size_t)k * stride);
+            a = make_float4(a.x + t.x, a.y + t.y, a.z + t.z, a.w + t.w);
+            if (turned) {
+                t = load4(o + (size_t)k * stride);
+                b = make_float4(b.x + t.x, b.y + t.y, b.z + t.z, b.w + t.w);
+            }
+        }
+        v[0] = a.x; v[1 % VEC] = a.y; v[2 % VEC] = a.z; v[3 % VEC] = a.w;
+        w[0] = b.x; w[1 % VEC] = b.y; w[2 % VEC] = b.z; w[3 % VEC] = b.w;
+    } else {
+        v[0] = add_partials(0.0f, p, S, stride);
+        w[0] = turned ? add_partials(0.0f, o, S, stride) : 0.0f;
+    }
+#pragma unroll
+    for (int u = 0; u < VEC; u++) {
+        if (turned)
+            v[u] = fmaf(v[u], co[u], w[u] * si[u]);
+        v[u] *= f;
+    }
+    float *dst = out + (size_t)r * width + c;
+    if (VEC == 4)
+        store4(dst, make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]));
+    else
+        dst[0] = v[0];
 }
 
 // The same for few rows: a cluster of C CTAs per (row, part), each with `cols` columns of the part
@@ -410,7 +538,7 @@ gated_part_norm_cluster_kernel(const float *__restrict__ y, const float *__restr
                                size_t pre_stride, int pre_ld, int pre_col0, const float *__restrict__ post,
                                int post_S, size_t post_stride, int post_ld, int post_col0,
                                const float *__restrict__ w, float eps, TO *__restrict__ out, int width, int parts,
-                               int cols)
+                               int cols, int post_silu)
 {
     extern __shared__ float held[];
     __shared__ float red[32];
@@ -439,9 +567,13 @@ gated_part_norm_cluster_kernel(const float *__restrict__ y, const float *__restr
         tot += part_sq[k];
     float scale = 1.0f / sqrtf(tot / (float)len + eps);
     for (int c = c0 + threadIdx.x; c < c1; c += blockDim.x) {
-        float v = (held[c - c0] * scale) * w[c];
-        if (post != nullptr)
-            v *= sigmoid_f(add_partials(0.0f, post + (size_t)r * post_ld + post_col0 + c, post_S, post_stride));
+        float v = held[c - c0] * scale;
+        if (w != nullptr)
+            v *= w[c];
+        if (post != nullptr) {
+            float g = add_partials(0.0f, post + (size_t)r * post_ld + post_col0 + c, post_S, post_stride);
+            v *= post_silu ? silu_f(g) : sigmoid_f(g);
+        }
         out[(size_t)r * width + c] = from_f<TO>(v);
     }
 }
@@ -666,12 +798,12 @@ extern "C" int jb_matrix_state_scan(const float *src, int S, long long stride, i
 
 extern "C" int jb_gated_part_norm(const float *y, const float *pre, int pre_S, long long pre_stride, int pre_ld,
                                   int pre_col0, const float *post, int post_S, long long post_stride, int post_ld,
-                                  int post_col0, const float *w, float eps, void *out, int out_dt, int n, int width,
-                                  int parts, int few_rows, cudaStream_t st)
+                                  int post_col0, int post_silu, const float *w, float eps, void *out, int out_dt,
+                                  int n, int width, int parts, int few_rows, cudaStream_t st)
 {
     if (n <= 0)
         return JB_OK;
-    if (width <= 0 || parts <= 0 || width % parts || parts > 65535 || y == nullptr || w == nullptr ||
+    if (width <= 0 || parts <= 0 || width % parts || parts > 65535 || y == nullptr ||
         (pre != nullptr && (pre_S <= 0 || pre_ld < pre_col0 + width)) ||
         (post != nullptr && (post_S <= 0 || post_ld < post_col0 + width)))
         return JB_EINVAL;
@@ -682,23 +814,71 @@ extern "C" int jb_gated_part_norm(const float *y, const float *pre, int pre_S, l
         if ((size_t)cols * 4 <= 40 * 1024) {
             launch_cluster(gated_part_norm_cluster_kernel<bf16, C>, dim3((unsigned)(n * parts * C)), 256, (size_t)cols * 4,
                            st, C, y, pre, pre_S, (size_t)pre_stride, pre_ld, pre_col0, post, post_S, (size_t)post_stride,
-                           post_ld, post_col0, w, eps, (bf16 *)out, width, parts, cols);
+                           post_ld, post_col0, w, eps, (bf16 *)out, width, parts, cols, post_silu);
             return launch_status();
         }
     }
     dim3 grid((unsigned)n, (unsigned)parts);
     size_t len = (size_t)(width / parts);
+    // short parts of which a row has several: a warp each
+    auto four = [](const float *p, int ld, long long stride, int col0) {
+        return p == nullptr || ((uintptr_t)p % 16 == 0 && ld % 4 == 0 && stride % 4 == 0 && col0 % 4 == 0);
+    };
+    if (parts > 1 && len % 4 == 0 && len <= 256 && (long long)n * parts <= 0x7fffffffll && four(y, width, 0, 0) &&
+        four(w, 4, 0, 0) && four(pre, pre_ld, pre_stride, pre_col0) && four(post, post_ld, post_stride, post_col0) &&
+        (uintptr_t)out % 16 == 0 && (out_dt == JB_F32 || out_dt == JB_BF16)) {
+        unsigned tasks = (unsigned)n * (unsigned)parts;
+        const int warps = n <= 64 ? 2 : 8;          // few rows: more blocks
+        unsigned g = (tasks + warps - 1) / warps;
+#define JB_GPN(TO, U)                                                                                          \
+    launch(gated_part_norm_warp_kernel<TO, U>, g, 32 * warps, 0, st, y, pre, pre_S, (size_t)pre_stride, pre_ld,  \
+           pre_col0, post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (TO *)out, width, parts,     \
+           post_silu, tasks)
+        if (out_dt == JB_F32) {
+            if (len <= 128) JB_GPN(float, 1); else JB_GPN(float, 2);
+        } else {
+            if (len <= 128) JB_GPN(bf16, 1); else JB_GPN(bf16, 2);
+        }
+#undef JB_GPN
+        return launch_status();
+    }
     int keep = len * 4 <= 40 * 1024 ? 1 : 0;
     size_t smem = keep ? len * 4 : 0;
     int threads = len >= 1024 ? 256 : 128;
     if (out_dt == JB_F32)
         launch(gated_part_norm_kernel<float>, grid, threads, smem, st, y, pre, pre_S, (size_t)pre_stride, pre_ld, pre_col0,
-               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (float *)out, width, parts, keep);
+               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (float *)out, width, parts, keep, post_silu);
     else if (out_dt == JB_BF16)
         launch(gated_part_norm_kernel<bf16>, grid, threads, smem, st, y, pre, pre_S, (size_t)pre_stride, pre_ld, pre_col0,
-               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (bf16 *)out, width, parts, keep);
+               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (bf16 *)out, width, parts, keep, post_silu);
     else
         return JB_EINVAL;
+    return launch_status();
+}
+
+// src: sums [S, n, ld]; out: float32 [n, 2 H D + H Dv].  See turn_heads_kernel.
+extern "C" int jb_turn_heads(const float *src, int S, long long stride, int ld, int col0, int H, int D, int Dv,
+                             const float *cs, const float *sn, int rot_half, const int32_t *row_pos, float key_scale,
+                             float *out, int n, cudaStream_t st)
+{
+    if (n <= 0)
+        return JB_OK;
+    long long width = (long long)H * (2 * D + Dv);
+    if (src == nullptr || out == nullptr || S <= 0 || H <= 0 || D <= 0 || Dv <= 0 || rot_half < 0 || 2 * rot_half > D ||
+        col0 < 0 || col0 + width > ld || (rot_half > 0 && (cs == nullptr || sn == nullptr || row_pos == nullptr)))
+        return JB_EINVAL;
+    bool vec = D % 4 == 0 && Dv % 4 == 0 && rot_half % 4 == 0 && ld % 4 == 0 && stride % 4 == 0 && col0 % 4 == 0 &&
+               (uintptr_t)src % 16 == 0 && (uintptr_t)out % 16 == 0;
+    long long per_row = vec ? width / 4 : width;
+    if ((per_row + 255) / 256 > 65535)
+        return JB_EINVAL;
+    dim3 grid((unsigned)n, (unsigned)((per_row + 255) / 256));
+    if (vec)
+        launch(turn_heads_kernel<4>, grid, 256, 0, st, src, S, (size_t)stride, ld, col0, H, D, Dv, cs, sn, rot_half,
+               row_pos, key_scale, out, (int)width);
+    else
+        launch(turn_heads_kernel<1>, grid, 256, 0, st, src, S, (size_t)stride, ld, col0, H, D, Dv, cs, sn, rot_half,
+               row_pos, key_scale, out, (int)width);
     return launch_status();
 }
 

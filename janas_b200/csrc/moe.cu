@@ -33,16 +33,18 @@ __device__ __forceinline__ void warp_argmax(float &v, int &i)
 //   the E experts form `groups` equal groups of neighbours; a group's score is its largest
 //   choice; only the `keep` best groups' experts can be chosen; the `top` largest choices
 //   among them are chosen (the lower index wins a tie); weight_e = s_e * scale.
-// With sigmoid_scores, s = sigmoid(logits), each on its own, instead of the softmax; with
-// group_best = b > 1 a group's score is the sum of its b largest choices.
+// bias (null: none) is added to the logits.  score JB_SCORE_SIGMOID: s = sigmoid(logits), each on
+// its own, instead of the softmax; JB_SCORE_CHOSEN: s = the logits themselves (the choice falls on
+// the largest), and the chosen ones' weights are the softmax over the chosen logits alone, times
+// scale.  With group_best = b > 1 a group's score is the sum of its b largest choices.
 // weights: [n, E], the weight of every chosen expert and 0 for the others.  skip_coef
 // [n]: the sum of the weights of the chosen experts from first_identity on (experts whose
 // output is their input).  Shared memory: 2 E + groups floats per warp.
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float *__restrict__ P, int S, size_t stride, int ld, int col0,
-                 const float *__restrict__ correction, float *__restrict__ weights,
-                 float *__restrict__ skip_coef, int n, int E, int groups, int keep, int top,
-                 int first_identity, float scale, int sigmoid_scores, int group_best)
+                 const float *__restrict__ bias, const float *__restrict__ correction,
+                 float *__restrict__ weights, float *__restrict__ skip_coef, int n, int E, int groups,
+                 int keep, int top, int first_identity, float scale, int score, int group_best)
 {
     extern __shared__ float sm[];
     pdl_trigger();
@@ -54,16 +56,17 @@ moe_route_kernel(const float *__restrict__ P, int S, size_t stride, int ld, int 
     pdl_wait();
     float mx = -INFINITY;
     for (int e = lane; e < E; e += 32) {
-        s[e] = add_partials(0.0f, P + (size_t)r * ld + col0 + e, S, stride);
+        s[e] = add_partials(0.0f, P + (size_t)r * ld + col0 + e, S, stride) + (bias != nullptr ? bias[e] : 0.0f);
         mx = fmaxf(mx, s[e]);
     }
     mx = warp_max(mx);
     float sum = 0.0f;
     for (int e = lane; e < E; e += 32) {
-        s[e] = sigmoid_scores ? 1.0f / (1.0f + expf(-s[e])) : expf(s[e] - mx);
+        if (score != JB_SCORE_CHOSEN)
+            s[e] = score == JB_SCORE_SIGMOID ? 1.0f / (1.0f + expf(-s[e])) : expf(s[e] - mx);
         sum += s[e];
     }
-    sum = sigmoid_scores ? 1.0f : warp_sum(sum);
+    sum = score == JB_SCORE_SOFTMAX ? warp_sum(sum) : 1.0f;
     for (int e = lane; e < E; e += 32) {
         s[e] = s[e] / sum;
         choice[e] = s[e] + (correction != nullptr ? correction[e] : 0.0f);
@@ -112,7 +115,9 @@ moe_route_kernel(const float *__restrict__ P, int S, size_t stride, int ld, int 
                 choice[e] = -INFINITY;
         __syncwarp();
     }
-    float skip = 0.0f;
+    // JB_SCORE_CHOSEN: the first choice's logit, and the sum of the chosen logits' exponentials
+    // relative to it
+    float skip = 0.0f, first = 0.0f, total = 0.0f;
     for (int k = 0; k < top; k++) {
         float v = -INFINITY;
         int i = 0x7fffffff;
@@ -124,7 +129,18 @@ moe_route_kernel(const float *__restrict__ P, int S, size_t stride, int ld, int 
         warp_argmax(v, i);
         if (i == 0x7fffffff)
             break;          // fewer experts may be chosen than top asks for
-        if (lane == 0) {
+        if (score == JB_SCORE_CHOSEN) {
+            float logit = s[i];
+            if (k == 0)
+                first = logit;
+            float ex = expf(logit - first);
+            total += ex;
+            __syncwarp();
+            if (lane == 0) {
+                s[i] = ex;
+                choice[i] = NAN;         // chosen: no comparison finds it again
+            }
+        } else if (lane == 0) {
             float wgt = s[i] * scale;
             weights[(size_t)r * E + i] = wgt;
             if (i >= first_identity)
@@ -132,6 +148,16 @@ moe_route_kernel(const float *__restrict__ P, int S, size_t stride, int ld, int 
             choice[i] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (score == JB_SCORE_CHOSEN) {
+        for (int e = lane; e < E; e += 32)
+            if (isnan(choice[e])) {
+                float wgt = s[e] / total * scale;
+                weights[(size_t)r * E + e] = wgt;
+                if (e >= first_identity)
+                    skip += wgt;
+            }
+        skip = warp_sum(skip);
     }
     if (lane == 0 && skip_coef != nullptr)
         skip_coef[r] = skip;
@@ -193,41 +219,58 @@ activation_weighted_kernel(const float *__restrict__ z, int S, size_t stride, in
     }
 }
 
+// act(g) * u, for silu with the gated unit's constants
+__device__ __forceinline__ float gated_value(float g, float u, int kind, const GatedUnit &unit)
+{
+    return kind == JB_ACT_SILU ? gated_unit(g, u, unit) : act_value(g, kind) * u;
+}
+
 // The same for experts with a gate: expert e's sums are [gate (ff) | up (ff)] in columns
-// 2 e ff .. of z, and out[r, e ff + j] = act(gate_j) * up_j * weights[r, e]; out: [n, n_experts ff].
-// V values per thread (V = 4: ff a multiple of four and everything on 16-byte boundaries).
+// 2 e ff .. of z, and out[r, e ff + j] = act(gate_j) * up_j * weights[r, e]; then a shared expert's
+// shared_ff values without a weight, its sums [gate | up] after the experts'; out: [n, width].
+// V values per thread (V = 4: ff and shared_ff multiples of four and everything on 16-byte
+// boundaries).
 template <typename TO, int V>
 __global__ void __launch_bounds__(256)
 gated_weighted_kernel(const float *__restrict__ z, int S, size_t stride, int ld,
-                      const float *__restrict__ weights, int w_ld, int ff, int kind,
-                      TO *__restrict__ out, int width)
+                      const float *__restrict__ weights, int w_ld, int n_experts, int ff, int shared_ff,
+                      int kind, GatedUnit unit, GatedUnit shared_unit, TO *__restrict__ out, int width)
 {
     pdl_trigger();
     int r = blockIdx.x, c = (int)(blockIdx.y * blockDim.x + threadIdx.x) * V;
     if (c >= width)
         return;
     pdl_wait();
-    int e = c / ff, j = c - e * ff;
-    float wgt = weights[(size_t)r * w_ld + e];
-    const float *src = z + (size_t)r * ld + (size_t)2 * e * ff + j;
+    int e = c / ff, j = c - e * ff, up = ff;
+    float wgt;
+    const float *src = z + (size_t)r * ld;
+    if (e < n_experts) {
+        wgt = weights[(size_t)r * w_ld + e];
+        src += (size_t)2 * e * ff + j;
+    } else {
+        wgt = 1.0f;
+        unit = shared_unit;
+        up = shared_ff;
+        src += (size_t)n_experts * ff + c;       // 2 n_experts ff + (c - n_experts ff)
+    }
     if (V == 4) {
         float4 g = make_float4(0.0f, 0.0f, 0.0f, 0.0f), u = g;
         if (wgt != 0.0f)
             for (int sp = 0; sp < S; sp++) {
-                float4 a = load4(src + (size_t)sp * stride), b = load4(src + ff + (size_t)sp * stride);
+                float4 a = load4(src + (size_t)sp * stride), b = load4(src + up + (size_t)sp * stride);
                 g.x += a.x; g.y += a.y; g.z += a.z; g.w += a.w;
                 u.x += b.x; u.y += b.y; u.z += b.z; u.w += b.w;
             }
         float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (wgt != 0.0f)
-            v = make_float4(act_value(g.x, kind) * u.x * wgt, act_value(g.y, kind) * u.y * wgt,
-                            act_value(g.z, kind) * u.z * wgt, act_value(g.w, kind) * u.w * wgt);
+            v = make_float4(gated_value(g.x, u.x, kind, unit) * wgt, gated_value(g.y, u.y, kind, unit) * wgt,
+                            gated_value(g.z, u.z, kind, unit) * wgt, gated_value(g.w, u.w, kind, unit) * wgt);
         store4<TO>(out + (size_t)r * width + c, v);
     } else {
         float v = 0.0f;
         if (wgt != 0.0f) {
-            float g = add_partials(0.0f, src, S, stride), u = add_partials(0.0f, src + ff, S, stride);
-            v = act_value(g, kind) * u * wgt;
+            float g = add_partials(0.0f, src, S, stride), u = add_partials(0.0f, src + up, S, stride);
+            v = gated_value(g, u, kind, unit) * wgt;
         }
         out[(size_t)r * width + c] = from_f<TO>(v);
     }
@@ -271,18 +314,19 @@ extern "C" int jb_add_row_scaled(float *y, const void *skip, int skip_dt, const 
 }
 
 extern "C" int jb_moe_route(const float *P, int S, long long stride, int ld, int col0,
-                            const float *correction, float *weights, float *skip_coef, int n, int E,
-                            int groups, int keep, int top, int first_identity, float scale,
-                            int sigmoid_scores, int group_best, cudaStream_t st)
+                            const float *bias, const float *correction, float *weights, float *skip_coef,
+                            int n, int E, int groups, int keep, int top, int first_identity, float scale,
+                            int score, int group_best, cudaStream_t st)
 {
     if (n <= 0)
         return JB_OK;
     if (E <= 0 || E > 2048 || groups <= 0 || E % groups || keep <= 0 || keep > groups || top <= 0 || top > E ||
-        ld < col0 + E || S <= 0 || first_identity < 0 || group_best < 1)
+        ld < col0 + E || S <= 0 || first_identity < 0 || group_best < 1 ||
+        score < JB_SCORE_SOFTMAX || score > JB_SCORE_CHOSEN)
         return JB_EINVAL;
     size_t smem = (size_t)4 * (2 * E + groups) * 4;
-    launch(moe_route_kernel, (unsigned)((n + 3) / 4), 128, smem, st, P, S, (size_t)stride, ld, col0, correction,
-           weights, skip_coef, n, E, groups, keep, top, first_identity, scale, sigmoid_scores, group_best);
+    launch(moe_route_kernel, (unsigned)((n + 3) / 4), 128, smem, st, P, S, (size_t)stride, ld, col0, bias,
+           correction, weights, skip_coef, n, E, groups, keep, top, first_identity, scale, score, group_best);
     return launch_status();
 }
 
@@ -321,23 +365,34 @@ extern "C" int jb_activation_weighted(const float *z, int S, long long stride, i
 }
 
 // z: float32 [S, n, ld] whose first 2 n_experts ff columns are, per expert, ff gate values and
-// then ff up values; weights: float32 [n, w_ld].  out: [n, n_experts ff] in out_dt.
+// then ff up values, and then a shared expert's 2 shared_ff columns (shared_ff 0: none); weights:
+// float32 [n, w_ld].  out: [n, n_experts ff + shared_ff] in out_dt.  unit: the three constants
+// {alpha, limit, shift} of the experts' gated unit and after them the shared expert's three, on
+// the host (null: SiLU(gate) * up); they are for JB_ACT_SILU alone.
 extern "C" int jb_gated_weighted(const float *z, int S, long long stride, int ld, const float *weights, int w_ld,
-                                 int n_experts, int ff, int kind, void *out, int out_dt, int n, cudaStream_t st)
+                                 int n_experts, int ff, int shared_ff, int kind, const float *unit, void *out,
+                                 int out_dt, int n, cudaStream_t st)
 {
     if (n <= 0)
         return JB_OK;
-    long long width = (long long)n_experts * ff;
-    if (n_experts <= 0 || ff <= 0 || ld < 2 * width || width > 0x7fffffffll || weights == nullptr || w_ld < n_experts ||
-        S <= 0 || (kind != JB_ACT_RELU2 && kind != JB_ACT_RELU && kind != JB_ACT_GELU_TANH && kind != JB_ACT_SILU) ||
-        (width + 255) / 256 > 65535)
+    long long width = (long long)n_experts * ff + shared_ff;
+    if (n_experts <= 0 || ff <= 0 || shared_ff < 0 || ld < 2 * width || width > 0x7fffffffll || weights == nullptr ||
+        w_ld < n_experts || S <= 0 ||
+        (kind != JB_ACT_RELU2 && kind != JB_ACT_RELU && kind != JB_ACT_GELU_TANH && kind != JB_ACT_SILU) ||
+        (width + 255) / 256 > 65535 || (unit != nullptr && kind != JB_ACT_SILU))
         return JB_EINVAL;
-    bool vec = ff % 4 == 0 && ld % 4 == 0 && stride % 4 == 0 && (uintptr_t)z % 16 == 0 && (uintptr_t)out % 16 == 0;
+    GatedUnit u{1.0f, 0.0f, 0.0f}, us = u;
+    if (unit != nullptr) {
+        u = GatedUnit{unit[0], unit[1], unit[2]};
+        us = GatedUnit{unit[3], unit[4], unit[5]};
+    }
+    bool vec = ff % 4 == 0 && shared_ff % 4 == 0 && ld % 4 == 0 && stride % 4 == 0 && (uintptr_t)z % 16 == 0 &&
+               (uintptr_t)out % 16 == 0;
     long long per_row = vec ? width / 4 : width;
     dim3 grid((unsigned)n, (unsigned)((per_row + 255) / 256));
-#define JB_GW(TO, V)                                                                                        \
-    launch(gated_weighted_kernel<TO, V>, grid, 256, 0, st, z, S, (size_t)stride, ld, weights, w_ld, ff, kind, \
-           (TO *)out, (int)width)
+#define JB_GW(TO, V)                                                                                         \
+    launch(gated_weighted_kernel<TO, V>, grid, 256, 0, st, z, S, (size_t)stride, ld, weights, w_ld, n_experts, ff, \
+           shared_ff, kind, u, us, (TO *)out, (int)width)
     if (out_dt == JB_F32) {
         if (vec) JB_GW(float, 4); else JB_GW(float, 1);
     } else if (out_dt == JB_BF16) {

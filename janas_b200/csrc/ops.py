@@ -209,8 +209,10 @@ def add_(x: torch.Tensor, delta: torch.Tensor) -> torch.Tensor:
     return x
 
 
-def swiglu(gate_up: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
-    """SiLU(gate) * up for a stack [S, n, 2 ff] whose columns are [gate | up]."""
+def swiglu(gate_up: torch.Tensor, out_dtype: torch.dtype, alpha: float = 1.0, limit: float = 0.0,
+           shift: float = 0.0) -> torch.Tensor:
+    """gate sigmoid(alpha gate) (up + shift) for a stack [S, n, 2 ff] whose columns are [gate | up]; with
+    limit > 0 the gate is cut off above it and up on both sides first.  The defaults are SiLU(gate) * up."""
     gate_up = stack(gate_up)
     _need(gate_up, "gate_up", torch.float32, (None, None, None))
     S, n, two_ff = gate_up.shape
@@ -218,19 +220,19 @@ def swiglu(gate_up: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
         raise KernelError("swiglu: the gate_up width must be even")
     ff = two_ff // 2
     out = torch.empty((n, ff), dtype=out_dtype, device=gate_up.device)
-    _check(lib().jb_swiglu(_p(gate_up), S, int(n * two_ff), _p(out),
-                           _DT[out_dtype], n, ff, _stream()), "swiglu")
+    _check(lib().jb_gated_unit(_p(gate_up), S, int(n * two_ff), _p(out), _DT[out_dtype], n, ff,
+                               float(alpha), float(limit), float(shift), _stream()), "swiglu")
     return out
 
 
 # ------------------------------------------------------------------ position
-def rope_table(inv_freq: torch.Tensor, n_pos: int) -> Tuple[torch.Tensor, torch.Tensor]:
-    """cos and sin of (float)p * inv_freq[i] for p < n_pos: two [n_pos, half]."""
+def rope_table(inv_freq: torch.Tensor, n_pos: int, amplitude: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """cos and sin of (float)p * inv_freq[i] for p < n_pos, times amplitude: two [n_pos, half]."""
     _need(inv_freq, "inv_freq", torch.float32)
     half = inv_freq.numel()
     cs = torch.empty((n_pos, half), dtype=torch.float32, device=inv_freq.device)
     sn = torch.empty_like(cs)
-    _check(lib().jb_rope_table(_p(cs), _p(sn), _p(inv_freq), n_pos, half, _stream()),
+    _check(lib().jb_rope_table_scaled(_p(cs), _p(sn), _p(inv_freq), n_pos, half, float(amplitude), _stream()),
            "rope_table")
     return cs, sn
 
@@ -510,12 +512,14 @@ def mingru(P: torch.Tensor, width: int, bias: Optional[torch.Tensor], state: tor
 
 def moe_route(P: torch.Tensor, col0: int, outputs: int, correction: Optional[torch.Tensor], groups: int,
               keep: int, top: int, first_identity: int, scale: float, sigmoid_scores: bool = False,
-              group_best: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
+              group_best: int = 1, chosen_softmax: bool = False,
+              bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """The router of a routed feed-forward over the logits in columns col0 .. col0 + outputs - 1
     of the sums P [S, n, ld]: (weights [n, outputs], 0 for outputs not chosen; the summed
     weight of the chosen outputs from first_identity on, [n]).  sigmoid_scores: each score is
     the sigmoid of its logit instead of a softmax over all; group_best: a group's score is the
-    sum of that many of its largest choice scores."""
+    sum of that many of its largest choice scores; chosen_softmax: the scores are the logits, and the
+    chosen ones' weights are a softmax over them alone; bias: added to the logits."""
     P = stack(P)
     _need(P, "P", torch.float32, (None, None, None))
     S, n, ld = P.shape
@@ -523,24 +527,31 @@ def moe_route(P: torch.Tensor, col0: int, outputs: int, correction: Optional[tor
         _need(correction, "correction", torch.float32, (outputs,))
     weights = torch.empty((n, outputs), dtype=torch.float32, device=P.device)
     skip = torch.empty((n,), dtype=torch.float32, device=P.device)
-    _check(lib().jb_moe_route(_p(P), S, n * ld, ld, col0, _p(correction), _p(weights), _p(skip), n, outputs,
-                              groups, keep, top, first_identity, float(scale), 1 if sigmoid_scores else 0,
-                              group_best, _stream()), "moe_route")
+    if bias is not None:
+        _need(bias, "bias", torch.float32, (outputs,))
+    _check(lib().jb_moe_route(_p(P), S, n * ld, ld, col0, _p(bias), _p(correction), _p(weights), _p(skip), n,
+                              outputs, groups, keep, top, first_identity, float(scale),
+                              2 if chosen_softmax else 1 if sigmoid_scores else 0, group_best, _stream()),
+           "moe_route")
     return weights, skip
 
 
 def gated_weighted(z: torch.Tensor, weights: torch.Tensor, n_experts: int, ff: int, kind: str,
-                   out_dtype: torch.dtype) -> torch.Tensor:
+                   out_dtype: torch.dtype, shared_ff: int = 0,
+                   units: Optional[Tuple[float, ...]] = None) -> torch.Tensor:
     """act(gate) * up * weights[row, expert] for experts whose sums lie [gate (ff) | up (ff)] one
-    after the other in z [S, n, ld]: [n, n_experts * ff]."""
+    after the other in z [S, n, ld], then a shared expert's shared_ff values without a weight:
+    [n, n_experts * ff + shared_ff].  units (silu alone): alpha, limit, shift of the experts' gated
+    unit and then of the shared expert's."""
     z = stack(z)
     _need(z, "z", torch.float32, (None, None, None))
     S, n, ld = z.shape
     _need(weights, "weights", torch.float32, (n, None))
-    out = torch.empty((n, n_experts * ff), dtype=out_dtype, device=z.device)
+    out = torch.empty((n, n_experts * ff + shared_ff), dtype=out_dtype, device=z.device)
+    u = None if units is None else (ctypes.c_float * 6)(*units)
     kinds = {"relu2": 0, "relu": 1, "gelu_tanh": 2, "silu": 3}
     _check(lib().jb_gated_weighted(_p(z), S, n * ld, ld, _p(weights), weights.shape[1], n_experts, ff,
-                                   kinds[kind], _p(out), _DT[out_dtype], n, _stream()), "gated_weighted")
+                                   shared_ff, kinds[kind], u, _p(out), _DT[out_dtype], n, _stream()), "gated_weighted")
     return out
 
 
@@ -598,20 +609,52 @@ def matrix_state_scan(src: torch.Tensor, H: int, G: int, N: int, P: int, val_col
     return y
 
 
-def gated_part_norm(y: torch.Tensor, parts: int, w: torch.Tensor, eps: float, out_dtype: torch.dtype,
+def turn_heads(src: torch.Tensor, col0: int, H: int, D: int, Dv: int, cos: Optional[torch.Tensor],
+               sin: Optional[torch.Tensor], row_pos: torch.Tensor, key_scale: float) -> torch.Tensor:
+    """[q | k | v] float32 [n, H (2 D + Dv)] out of the sums src [S, n, ld] from column col0 on: the
+    first 2 * cos.shape[1] values of every q and k head turned by the row's position (value i with value
+    i + cos.shape[1]), k times key_scale."""
+    src = stack(src)
+    _need(src, "src", torch.float32, (None, None, None))
+    S, n, ld = src.shape
+    out = torch.empty((n, H * (2 * D + Dv)), dtype=torch.float32, device=src.device)
+    _check(lib().jb_turn_heads(_p(src), S, n * ld, ld, col0, H, D, Dv, _p(cos), _p(sin),
+                               0 if cos is None else cos.shape[1], _p(row_pos), float(key_scale), _p(out), n,
+                               _stream()), "turn_heads")
+    return out
+
+
+def join_rows(x: torch.Tensor, delta: Optional[torch.Tensor], e: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """[x + sum(delta) | e] as [n, 2 dm]; x (float32 [n, dm]) is left at zero."""
+    _need(x, "x", torch.float32, (None, None))
+    n, dm = x.shape
+    _need(e, "e", torch.float32, (n, dm))
+    if delta is not None:
+        delta = stack(delta)
+        _need(delta, "delta", torch.float32, (None, n, dm))
+    out = torch.empty((n, 2 * dm), dtype=out_dtype, device=x.device)
+    _check(lib().jb_join_rows(_p(x), _p(delta), 0 if delta is None else delta.shape[0], n * dm, _p(e), _p(out),
+                              _DT[out_dtype], n, dm, _stream()), "join_rows")
+    return out
+
+
+def gated_part_norm(y: torch.Tensor, parts: int, w: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype,
                     pre: Optional[torch.Tensor] = None, pre_col0: int = 0,
-                    post: Optional[torch.Tensor] = None, post_col0: int = 0, few_rows: bool = False) -> torch.Tensor:
-    """rms(y * silu(pre)) in ``parts`` equal parts of each row, times w, times sigmoid(post)."""
+                    post: Optional[torch.Tensor] = None, post_col0: int = 0, few_rows: bool = False,
+                    post_silu: bool = False) -> torch.Tensor:
+    """rms(y * silu(pre)) in ``parts`` equal parts of each row, times w (None: 1), times sigmoid(post) or,
+    with post_silu, silu(post)."""
     _need(y, "y", torch.float32, (None, None))
     n, width = y.shape
-    _need(w, "w", torch.float32, (width,))
+    if w is not None:
+        _need(w, "w", torch.float32, (width,))
     pre = None if pre is None else stack(pre)
     post = None if post is None else stack(post)
     out = torch.empty((n, width), dtype=out_dtype, device=y.device)
     a = (0, 0, 0) if pre is None else (pre.shape[0], n * pre.shape[2], pre.shape[2])
     b = (0, 0, 0) if post is None else (post.shape[0], n * post.shape[2], post.shape[2])
     _check(lib().jb_gated_part_norm(_p(y), _p(pre), a[0], a[1], a[2], pre_col0, _p(post), b[0], b[1], b[2],
-                                    post_col0, _p(w), float(eps), _p(out), _DT[out_dtype], n, width, parts,
+                                    post_col0, 1 if post_silu else 0, _p(w), float(eps), _p(out), _DT[out_dtype], n, width, parts,
                                     1 if few_rows else 0, _stream()), "gated_part_norm")
     return out
 
@@ -662,9 +705,11 @@ def qkv_prepare_append(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight
                        k_weight: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor],
                        sin: Optional[torch.Tensor], row_pos: torch.Tensor, row_seq: torch.Tensor,
                        block_table: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
-                       num_heads: int, pairs: bool = False, unit_norm: bool = False) -> torch.Tensor:
+                       num_heads: int, pairs: bool = False, unit_norm: bool = False,
+                       values_from_keys: bool = False) -> torch.Tensor:
     """pairs: the rotation turns neighbours (2i, 2i + 1); unit_norm: q and k heads are divided by
-    their root mean square after the rotation.
+    their root mean square after the rotation; values_from_keys: the product holds q and k alone, and
+    a key's sums are its value too.
     q, k, v out of the sums of one product [S, n, ld] = [q | k | v | ...]: the bias, an RMS
     norm per head on q and k (weights float32 [hd] or None), a rotation of the first
     2 * cos.shape[1] values of each head (value i with value i + cos.shape[1]), K and V
@@ -685,7 +730,8 @@ def qkv_prepare_append(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight
                                        float(eps), _p(cos), _p(sin), rot_half, _p(row_pos), _p(row_seq),
                                        _p(block_table), block_table.shape[1], _p(q), _p(k_cache),
                                        _p(v_cache), _DT[k_cache.dtype], n, num_heads, nkv, hd, vd,
-                                       (1 if pairs else 0) | (2 if unit_norm else 0), _stream()),
+                                       (1 if pairs else 0) | (2 if unit_norm else 0) | (4 if values_from_keys else 0),
+                                       _stream()),
            "qkv_prepare_append")
     return q
 
@@ -693,27 +739,29 @@ def qkv_prepare_append(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight
 def latent_down(P: torch.Tensor, q_rank: int, wq: Optional[torch.Tensor], kv_rank: int,
                 wkv: torch.Tensor, rot_dim: int, cos: Optional[torch.Tensor],
                 sin: Optional[torch.Tensor], row_pos: torch.Tensor, row_seq: torch.Tensor,
-                block_table: torch.Tensor, k_cache: torch.Tensor, eps: float) -> torch.Tensor:
+                block_table: torch.Tensor, k_cache: torch.Tensor, eps: float, halves: bool = False) -> torch.Tensor:
     """P: sums [S, n, >= q_rank + kv_rank + rot_dim], columns [query latent | latent |
     shared key part].  Returns the RMS-normed query latent [n, q_rank] in the cache's
     dtype and writes [RMS-normed latent | rotated key part] to the cache rows
-    (k_cache [pages, 1, PAGE, kv_rank + rot_dim]) at the rows' positions."""
+    (k_cache [pages, 1, PAGE, kv_rank + rot_dim]) at the rows' positions.  halves: the rotation's
+    pairs are (i, i + rot_half) instead of neighbours."""
     P = stack(P)
     _need(P, "P", torch.float32, (None, None, None))
     S, n, ld = P.shape
     _need(k_cache, "k_cache", _FLOATS, (None, 1, PAGE, kv_rank + rot_dim))
     rot_half = 0 if cos is None else cos.shape[1]
     cq = torch.empty((n, q_rank), dtype=k_cache.dtype, device=P.device)
-    _check(lib().jb_latent_down(_p(P), S, n * ld, ld, 0, q_rank, _p(wq), q_rank, kv_rank, _p(wkv),
-                                rot_dim, _p(cos), _p(sin), rot_half, _p(row_pos), _p(row_seq),
-                                _p(block_table), block_table.shape[1], _p(cq), _p(k_cache),
-                                _DT[k_cache.dtype], n, float(eps), _stream()), "latent_down")
+    _check(lib().jb_latent_down_rows(_p(P), S, n * ld, ld, 0, q_rank, _p(wq), q_rank, kv_rank, _p(wkv),
+                                     rot_dim, _p(cos), _p(sin), rot_half, _p(row_pos), _p(row_seq),
+                                     _p(block_table), block_table.shape[1], _p(cq), _p(k_cache), None,
+                                     _DT[k_cache.dtype], n, float(eps), 1 if halves else 0, _stream()),
+           "latent_down")
     return cq
 
 
 def latent_queries(Q: torch.Tensor, w_ukT: torch.Tensor, num_heads: int, D: int, R: int, C: int,
                    cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], row_pos: torch.Tensor,
-                   dtype: torch.dtype) -> torch.Tensor:
+                   dtype: torch.dtype, halves: bool = False) -> torch.Tensor:
     """Q: the query product's sums [S, n, heads (D + R)]; w_ukT [heads C, D]: per head
     the key matrix, transposed.  Returns the latent queries [n, heads, C + R]: per head
     [Wuk_head^T q_plain | rotated q_rot]."""
@@ -725,7 +773,8 @@ def latent_queries(Q: torch.Tensor, w_ukT: torch.Tensor, num_heads: int, D: int,
     q_lat = torch.empty((n, num_heads, C + R), dtype=dtype, device=Q.device)
     L = lib()
     _check(L.jb_latent_q_split(_p(Q), S, Q.shape[1] * Q.shape[2], num_heads, D, R, C, _p(cos), _p(sin),
-                               rot_half, _p(row_pos), _p(q_plain), _p(q_lat), _DT[dtype], n, _stream()),
+                               rot_half, _p(row_pos), _p(q_plain), _p(q_lat), _DT[dtype], n,
+                               1 if halves else 0, C + R, _stream()),
            "latent_q_split")
     A = torch.stack([stack(linear(q_plain[h], w_ukT[h * C:(h + 1) * C], force_simt=True))
                      for h in range(num_heads)])
@@ -1086,8 +1135,9 @@ def linear_heads(a: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def linear_swiglu(a: torch.Tensor, gate_up: torch.Tensor) -> Optional[torch.Tensor]:
-    """SiLU(a . gate^T) * (a . up^T) in one tensor-core kernel, for bfloat16
+def linear_swiglu(a: torch.Tensor, gate_up: torch.Tensor, alpha: float = 1.0, limit: float = 0.0,
+                  shift: float = 0.0) -> Optional[torch.Tensor]:
+    """SiLU(a . gate^T) * (a . up^T), or swiglu's other units, in one tensor-core kernel, for bfloat16
     a [n, k] and gate_up [2 ff, k] (rows [gate | up]); returns bfloat16 [n, ff],
     or None when the kernel does not take the operands."""
     _need(a, "activations", _FLOATS, (None, None))
@@ -1097,7 +1147,8 @@ def linear_swiglu(a: torch.Tensor, gate_up: torch.Tensor) -> Optional[torch.Tens
     n, k = a.shape
     ff = gate_up.shape[0] // 2
     out = torch.empty((n, ff), dtype=torch.bfloat16, device=a.device)
-    _check(lib().jb_gemm_tc_swiglu(_p(a), _p(gate_up), _p(out), n, ff, k, _stream()),
+    _check(lib().jb_gemm_tc_gated(_p(a), _p(gate_up), _p(out), n, ff, k, float(alpha), float(limit),
+                                  float(shift), _stream()),
            "linear_swiglu (tcgen05)")
     return out
 

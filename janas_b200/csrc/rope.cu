@@ -18,7 +18,7 @@
 namespace jb {
 
 __global__ void rope_table_kernel(float *__restrict__ cs, float *__restrict__ sn,
-                                  const float *__restrict__ inv_freq, int n_pos, int half)
+                                  const float *__restrict__ inv_freq, int n_pos, int half, double amplitude)
 {
     pdl_trigger();
     pdl_wait();
@@ -29,8 +29,8 @@ __global__ void rope_table_kernel(float *__restrict__ cs, float *__restrict__ sn
     float theta = __fmul_rn((float)p, inv_freq[f]);
     double s, c;
     sincos((double)theta, &s, &c);
-    cs[i] = (float)c;
-    sn[i] = (float)s;
+    cs[i] = (float)(c * amplitude);
+    sn[i] = (float)(s * amplitude);
 }
 
 // One warp per (row, head slot); head slots are the q heads, then the k heads,
@@ -387,11 +387,12 @@ qkv_prepare_append_kernel(const float *__restrict__ qkv, int S, size_t split_str
                           int n, int nh, int nkv, int hd, int vd, int mode)
 {
     pdl_trigger();
-    unsigned slots = nh + 2 * nkv;
+    // with JB_VALUES_FROM_KEYS a key's slot stores its sums as the value too, before norm and rotation
+    const bool pairs = mode & JB_ROT_PAIRS, unit = mode & JB_UNIT_NORM, both = mode & JB_VALUES_FROM_KEYS;
+    unsigned slots = nh + (both ? 1 : 2) * nkv;
     unsigned task = blockIdx.x * blockDim.y + threadIdx.y;
     if (task >= (unsigned)n * slots)
         return;
-    const bool pairs = mode & JB_ROT_PAIRS, unit = mode & JB_UNIT_NORM;
     unsigned row = task / slots, hs = task - row * slots;
     int lane = threadIdx.x;
     bool is_q = hs < (unsigned)nh;
@@ -417,6 +418,11 @@ qkv_prepare_append_kernel(const float *__restrict__ qkv, int S, size_t split_str
     }
     const float *src = qkv + (size_t)row * ld + col0;
     const float *b = bias != nullptr ? bias + col0 : nullptr;
+    if (both && !is_q) {
+        TC *vdst = v_cache + (((size_t)page * nkv + (hs - nh)) * PAGE + (pos % PAGE)) * vd;
+        for (int i = lane; i < len; i += 32)
+            vdst[i] = from_f<TC>(add_partials(b != nullptr ? b[i] : 0.0f, src + i, S, split_stride));
+    }
     float ss = 0.0f;
     if (w != nullptr) {
         for (int i = lane; i < len; i += 32) {
@@ -472,9 +478,9 @@ qkv_prepare_append_vec_kernel(const float *__restrict__ qkv, int S, size_t split
                               int n, int nh, int nkv, int hd, int vd, int mode)
 {
     constexpr int PER_WARP = 32 / L;
-    const bool pairs = mode & JB_ROT_PAIRS, unit = mode & JB_UNIT_NORM;
+    const bool pairs = mode & JB_ROT_PAIRS, unit = mode & JB_UNIT_NORM, both = mode & JB_VALUES_FROM_KEYS;
     pdl_trigger();
-    unsigned slots = nh + 2 * nkv;
+    unsigned slots = nh + (both ? 1 : 2) * nkv;
     unsigned total = (unsigned)n * slots;
     unsigned task = (blockIdx.x * blockDim.y + threadIdx.y) * PER_WARP + threadIdx.x / L;
     bool live = task < total;
@@ -526,6 +532,8 @@ qkv_prepare_append_vec_kernel(const float *__restrict__ qkv, int S, size_t split
             float4 u = load4(src + (size_t)sp * split_stride);
             v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
         }
+        if (both && !is_q && live && dst != nullptr)
+            store4(v_cache + (dst - k_cache) + 4 * l, v);      // vd = hd: the same place in the value pages
     }
     float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
 #pragma unroll
@@ -588,10 +596,11 @@ extern "C" int jb_qkv_prepare_append(const float *qkv, int S, long long split_st
         return JB_OK;
     if (hd <= 0 || hd > 512 || vd <= 0 || vd > 512 || rot_half < 0 || 2 * rot_half > hd || nh < 0 || nkv < 0 ||
         (q_w == nullptr) != (k_w == nullptr) || (rot_half > 0 && (cs == nullptr || sn == nullptr)) ||
-        (mode & ~(JB_ROT_PAIRS | JB_UNIT_NORM)) ||
-        ld < nh * hd + (k_cache != nullptr ? nkv * (hd + vd) : 0) || (k_cache != nullptr && v_cache == nullptr))
+        (mode & ~(JB_ROT_PAIRS | JB_UNIT_NORM | JB_VALUES_FROM_KEYS)) ||
+        ((mode & JB_VALUES_FROM_KEYS) && (vd != hd || k_cache == nullptr)) ||
+        ld < nh * hd + (k_cache == nullptr ? 0 : (mode & JB_VALUES_FROM_KEYS) ? nkv * hd : nkv * (hd + vd)) || (k_cache != nullptr && v_cache == nullptr))
         return JB_EINVAL;
-    size_t tasks = (size_t)n * (nh + 2 * nkv);
+    size_t tasks = (size_t)n * (nh + ((mode & JB_VALUES_FROM_KEYS) ? 1 : 2) * nkv);
     if (tasks > 0xffffffffu)
         return JB_EINVAL;
     dim3 block(32, 4);
@@ -640,11 +649,18 @@ extern "C" int jb_qkv_prepare_append(const float *qkv, int S, long long split_st
 extern "C" int jb_rope_table(float *cs, float *sn, const float *inv_freq, int n_pos, int half,
                              cudaStream_t st)
 {
+    return jb_rope_table_scaled(cs, sn, inv_freq, n_pos, half, 1.0, st);
+}
+
+// The same with cos and sin times a factor.
+extern "C" int jb_rope_table_scaled(float *cs, float *sn, const float *inv_freq, int n_pos, int half,
+                                    double amplitude, cudaStream_t st)
+{
     size_t total = (size_t)n_pos * half;
     if (total == 0)
         return JB_OK;
     launch(rope_table_kernel, (unsigned)((total + 255) / 256), 256, 0, st, cs, sn, inv_freq, n_pos,
-           half);
+           half, amplitude);
     return launch_status();
 }
 

@@ -316,11 +316,11 @@ rmsnorm_vec_kernel(float *__restrict__ x, const float *__restrict__ delta, int S
 }
 
 // gu: S stacked [n, 2 ff] float partial sums; columns [0, ff) are the gate,
-// [ff, 2 ff) the up projection.  out[n, ff] = SiLU(gate) * up.  VEC values per
+// [ff, 2 ff) the up projection.  out[n, ff] = gated_unit(gate, up).  VEC values per
 // thread (4 when ff is a multiple of 4 and nothing is split, else 1).
 template <typename TO, int VEC>
 __global__ void swiglu_kernel(const float *__restrict__ gu, int S, size_t stride,
-                              TO *__restrict__ out, int ff, size_t total)
+                              TO *__restrict__ out, int ff, size_t total, GatedUnit unit)
 {
     pdl_trigger();
     pdl_wait();
@@ -336,11 +336,47 @@ __global__ void swiglu_kernel(const float *__restrict__ gu, int S, size_t stride
         float gv[4] = {g.x, g.y, g.z, g.w}, uv[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
         for (int e = 0; e < 4; e++)
-            out[i + e] = from_f<TO>(gv[e] / (1.0f + expf(-gv[e])) * uv[e]);
+            out[i + e] = from_f<TO>(gated_unit(gv[e], uv[e], unit));
     } else {
         float g = add_partials(0.0f, p + c, S, stride);
         float u = add_partials(0.0f, p + ff + c, S, stride);
-        out[i] = from_f<TO>(g / (1.0f + expf(-g)) * u);
+        out[i] = from_f<TO>(gated_unit(g, u, unit));
+    }
+}
+
+// [x + delta | e] in the compute type, rows [n, 2 dm], from the residual stream x (delta: S
+// stacked partial sums still to be added, or none) and the embedding output e; x is left at
+// zero, ready for the product over these rows to be added to it.  VEC values per thread.
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(256)
+join_rows_kernel(float *__restrict__ x, const float *__restrict__ delta, int S, size_t stride,
+                 const float *__restrict__ e, TO *__restrict__ out, int dm, size_t total)
+{
+    pdl_trigger();
+    pdl_wait();
+    size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (i >= total)
+        return;
+    size_t row = i / dm;
+    TO *o = out + row * 2 * dm + (i - row * dm);
+    if (VEC == 4) {
+        float4 v = load4(x + i);
+        for (int s = 0; s < S; s++) {
+            float4 d = load4(delta + (size_t)s * stride + i);
+            v = make_float4(v.x + d.x, v.y + d.y, v.z + d.z, v.w + d.w);
+        }
+        float4 ev = load4(e + i);
+        store4(o, v);
+        store4(o + dm, ev);
+        store4(x + i, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+    } else {
+        float v = x[i];
+        if (S > 0)
+            v = add_partials(v, delta + i, S, stride);
+        float ev = e[i];
+        o[0] = from_f<TO>(v);
+        o[dm] = from_f<TO>(ev);
+        x[i] = 0.0f;
     }
 }
 
@@ -500,6 +536,14 @@ extern "C" int jb_rmsnorm(float *x, const float *delta, int S, long long delta_s
 extern "C" int jb_swiglu(const float *gu, int S, long long stride, void *out, int out_dt, int n,
                          int ff, cudaStream_t st)
 {
+    return jb_gated_unit(gu, S, stride, out, out_dt, n, ff, 1.0f, 0.0f, 0.0f, st);
+}
+
+// The same with the unit's constants: gate sigmoid(alpha gate) (up + shift), cut off at limit (0: not).
+extern "C" int jb_gated_unit(const float *gu, int S, long long stride, void *out, int out_dt, int n,
+                             int ff, float alpha, float limit, float shift, cudaStream_t st)
+{
+    const GatedUnit unit{alpha, limit, shift};
     size_t total = (size_t)n * ff;
     if (total == 0)
         return JB_OK;
@@ -507,14 +551,39 @@ extern "C" int jb_swiglu(const float *gu, int S, long long stride, void *out, in
     size_t threads = vec ? total / 4 : total;
     unsigned blocks = (unsigned)((threads + 255) / 256);
     if (out_dt == JB_F32 && vec)
-        launch(swiglu_kernel<float, 4>, blocks, 256, 0, st, gu, S, (size_t)stride, (float *)out, ff, total);
+        launch(swiglu_kernel<float, 4>, blocks, 256, 0, st, gu, S, (size_t)stride, (float *)out, ff, total, unit);
     else if (out_dt == JB_F32)
-        launch(swiglu_kernel<float, 1>, blocks, 256, 0, st, gu, S, (size_t)stride, (float *)out, ff, total);
+        launch(swiglu_kernel<float, 1>, blocks, 256, 0, st, gu, S, (size_t)stride, (float *)out, ff, total, unit);
     else if (out_dt == JB_BF16 && vec)
-        launch(swiglu_kernel<bf16, 4>, blocks, 256, 0, st, gu, S, (size_t)stride, (bf16 *)out, ff, total);
+        launch(swiglu_kernel<bf16, 4>, blocks, 256, 0, st, gu, S, (size_t)stride, (bf16 *)out, ff, total, unit);
     else if (out_dt == JB_BF16)
-        launch(swiglu_kernel<bf16, 1>, blocks, 256, 0, st, gu, S, (size_t)stride, (bf16 *)out, ff, total);
+        launch(swiglu_kernel<bf16, 1>, blocks, 256, 0, st, gu, S, (size_t)stride, (bf16 *)out, ff, total, unit);
     else
         return JB_EINVAL;
+    return launch_status();
+}
+
+// See join_rows_kernel.  x, e: float32 [n, dm]; delta: S stacked [n, dm], or null with S = 0.
+extern "C" int jb_join_rows(float *x, const float *delta, int S, long long stride, const float *e, void *out,
+                            int out_dt, int n, int dm, cudaStream_t st)
+{
+    size_t total = (size_t)n * dm;
+    if (total == 0)
+        return JB_OK;
+    if (x == nullptr || e == nullptr || out == nullptr || S < 0 || (S > 0 && delta == nullptr))
+        return JB_EINVAL;
+    bool vec = dm % 4 == 0 && stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)delta % 16 == 0 &&
+               (uintptr_t)e % 16 == 0 && (uintptr_t)out % 16 == 0;
+    unsigned blocks = (unsigned)(((vec ? total / 4 : total) + 255) / 256);
+#define JB_JOIN(TO, V)                                                                              \
+    launch(join_rows_kernel<TO, V>, blocks, 256, 0, st, x, delta, S, (size_t)stride, e, (TO *)out, dm, total)
+    if (out_dt == JB_F32) {
+        if (vec) JB_JOIN(float, 4); else JB_JOIN(float, 1);
+    } else if (out_dt == JB_BF16) {
+        if (vec) JB_JOIN(bf16, 4); else JB_JOIN(bf16, 1);
+    } else {
+        return JB_EINVAL;
+    }
+#undef JB_JOIN
     return launch_status();
 }

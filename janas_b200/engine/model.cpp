@@ -53,6 +53,8 @@ TensorList DecoderModel::top_tensors() const {
         t.emplace_back(spec.token_table_name,
                        TensorSpec{{spec.vocab_size, spec.token_table_width}, EMBEDDING, false});
     if (embedding_norm) embedding_norm->tensors(spec.embedding_norm_name, t);
+    if (!spec.join_name.empty())
+        t.emplace_back(spec.join_name, TensorSpec{{spec.hidden_size, 2 * spec.hidden_size}, MATRIX, false});
     final_norm->tensors(spec.final_norm_name, t);
     t.emplace_back(spec.head_name, TensorSpec{{spec.vocab_size, spec.hidden_size}, MATRIX, spec.tie_embeddings});
     return t;
@@ -68,6 +70,7 @@ TensorList DecoderModel::tensors() const {
         embedding_norm->tensors(spec.embedding_norm_name, en);
         first += en.size();                                      // and the norm of their rows
     }
+    if (!spec.join_name.empty()) first++;
     t.insert(t.end(), top.begin(), top.begin() + first);
     for (size_t i = 0; i < blocks.size(); i++) {
         TensorList l = layer_tensors((int)i);
@@ -94,6 +97,7 @@ void DecoderModel::load_top(TensorMap &t) {
         fail(JB_LLM_EOPEN, "tensor " + spec.head_name + " is missing");
     }
     if (embedding_norm) embedding_norm->load(spec.embedding_norm_name, t);
+    if (!spec.join_name.empty()) join = Part::take(t, spec.join_name);
     final_norm->load(spec.final_norm_name, t);
 }
 
@@ -154,7 +158,7 @@ void DecoderModel::load_random(unsigned long long seed) {
 }
 
 size_t DecoderModel::weight_bytes() const {
-    size_t total = head.bytes() + token_table.bytes();
+    size_t total = head.bytes() + token_table.bytes() + join.bytes();
     std::set<int> used;
     for (auto &e : spec.run_order) used.insert(e.layer);
     for (int layer : used) {
@@ -220,10 +224,10 @@ Buf DecoderModel::forward(StepContext &ctx, const int32_t *tokens, std::vector<L
     ctx.normed.reset();
     ctx.normed_by = nullptr;
     if (embedding_norm) x = embedding_norm->apply(ctx, x.as<float>(), n, F32, nullptr, nullptr, 0);
-    // the embedding output, kept for the entries that add it once more
+    // the embedding output, kept for the entries that add it once more or join it
     Stack again;
     for (auto &e : spec.run_order)
-        if (e.add_embedding && !again) {
+        if ((e.add_embedding || e.join_embedding) && !again) {
             again.buf = d.pool.get((size_t)n * (size_t)spec.hidden_size * 4);
             again.S = 1;
             again.n = n;
@@ -240,10 +244,18 @@ Buf DecoderModel::forward(StepContext &ctx, const int32_t *tokens, std::vector<L
             }
             ops::add_(d, x.as<float>(), n, spec.hidden_size, again);
         }
+        if (spec.run_order[e].join_embedding) {
+            // x (with what is still to be added) and the embedding output side by side; the
+            // product is then all there is of the residual stream: x itself is left at zero
+            Buf both = ops::join_rows(d, x.as<float>(), n, spec.hidden_size, pending ? &pending : nullptr,
+                                      again.data(), ctx.dtype);
+            pending = ops::linear(d, both.ptr, ctx.dtype, n, 2 * spec.hidden_size, join);
+        }
         // the norm that meets the residual stream next: the next entry's first one (the
         // model's last norm runs on the wanted rows alone and is not computed ahead, and
         // neither is a norm that something is added in front of)
-        b.next_norm = e + 1 < spec.run_order.size() && !spec.run_order[e + 1].add_embedding
+        b.next_norm = e + 1 < spec.run_order.size() && !spec.run_order[e + 1].add_embedding &&
+                              !spec.run_order[e + 1].join_embedding
                           ? blocks[(size_t)spec.run_order[e + 1].layer]->mixer_norm.get() : nullptr;
         b.forward(ctx, x.as<float>(), pending, caches[e]);
         if (ctx.trace) {

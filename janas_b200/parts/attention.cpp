@@ -195,10 +195,15 @@ private:
 // head AFTER the rotation, without a weight; gate: the joined heads are multiplied by
 // sigmoid(Wg h) before the output product (Wg's rows go into the q, k, v product).
 //
+// values_are_keys: there is no Wv; a position's values are its keys as they come out of the
+// product, before norm and rotation.  sink_score (instead of sink): every head's sink is this
+// number (0: a one added to each denominator), not learned.
+//
 // params: hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim (default: head_dim),
 // scale (default 1/sqrt(head_dim)), window (0: none), keep_first (0: none), qk_norm_eps
 // (absent: no q/k norm), qk_unit_norm_eps (absent: none), conv_taps (0: none), gate (boolean),
-// position (a part; absent: none), score_bias (boolean),
+// position (a part; absent: none), score_bias (boolean), values_are_keys (boolean), sink_score
+// (a number; absent: none),
 // softcap (0 or absent: none),
 // distance_slope_exponent (absent: no bias), q_temp_coef and q_temp_every (absent or
 // every = 0: none), bias (on q, k, v), out_bias (on o; default: as bias), head_scale, sink, own_kv
@@ -237,7 +242,11 @@ public:
         qk_norm_ = s.has("qk_norm_eps");
         qk_eps_ = qk_norm_ ? (float)s.get_double("qk_norm_eps") : 0.0f;
         score_bias_ = flag(s, "score_bias", false);
-        if (score_bias_ && (sink_ || g_.softcap > 0.0f || has_slopes_ || head_scale_))
+        values_are_keys_ = flag(s, "values_are_keys", false);
+        has_sink_score_ = s.has("sink_score");
+        sink_score_ = has_sink_score_ ? (float)s.get_double("sink_score") : 0.0f;
+        if (has_sink_score_ && sink_) config_error("sink_attention: a learned sink and a given one exclude each other");
+        if (score_bias_ && (sink_ || has_sink_score_ || g_.softcap > 0.0f || has_slopes_ || head_scale_))
             config_error("sink_attention: weights that are sigmoids take no sink, cap, slopes or head factors");
         if (s.has("position")) {
             position_ = build_position(s.get_part("position"), dt, d);
@@ -255,7 +264,11 @@ public:
         }
         if (conv_taps_ > 0 && (bias_ || !own_kv_))
             config_error("sink_attention: the convolutions over q, k and v take no bias and need keys and values of the layer's own");
-        prepared_ = qk_norm_ || unit_norm_ || conv_taps_ > 0 || (position_ && position_->rotary_dim() > 0);
+        prepared_ = qk_norm_ || unit_norm_ || conv_taps_ > 0 || values_are_keys_ ||
+                    (position_ && position_->rotary_dim() > 0);
+        if (values_are_keys_ && (g_.vd != g_.hd || !own_kv_ || conv_taps_ > 0))
+            config_error("sink_attention: values that are the keys have the keys' size, a cache of their own and no "
+                         "convolutions");
         if (prepared_ && q_every_ > 0)
             config_error("sink_attention: a query temperature together with a q/k norm or a rotation is not built");
         if (prepared_ && !own_kv_)
@@ -288,7 +301,7 @@ public:
         mat(n_q_, qw, hidden_, bias_);
         if (own_kv_) {
             mat(n_k_, kw, hidden_, bias_);
-            mat(n_v_, vw, hidden_, bias_);
+            if (!values_are_keys_) mat(n_v_, vw, hidden_, bias_);
         }
         if (head_scale_) out.emplace_back(name(p, n_hs_), TensorSpec{{g_.nh}, PARAM, false, 1.0f, 0.1f});
         if (sink_) out.emplace_back(name(p, n_sink_), TensorSpec{{g_.nh}, PARAM, false, 0.0f, 0.5f});
@@ -314,8 +327,10 @@ public:
         if (own_kv_) {
             in.push_back(take(t, name(p, n_k_)));
             if (bias_) bs.push_back(take(t, name(p, n_k_ + n_bias_)));
-            in.push_back(take(t, name(p, n_v_)));
-            if (bias_) bs.push_back(take(t, name(p, n_v_ + n_bias_)));
+            if (!values_are_keys_) {
+                in.push_back(take(t, name(p, n_v_)));
+                if (bias_) bs.push_back(take(t, name(p, n_v_ + n_bias_)));
+            }
         }
         if (gate_) {
             gate_col0_ = 0;
@@ -356,7 +371,13 @@ public:
             g_.slopes = (const float *)slopes_.ptr;
         }
         g_.head_scale = head_scale_ ? (const float *)temp_.ptr : nullptr;
-        g_.sink = sink_ ? (const float *)sinks_.ptr : nullptr;
+        if (has_sink_score_) {
+            std::vector<float> sc((size_t)g_.nh, sink_score_);
+            sinks_ = dev->tensor(F32, {g_.nh});
+            cuda_check(cudaMemcpy(sinks_.ptr, sc.data(), sc.size() * 4, cudaMemcpyHostToDevice),
+                       "copying the heads' sinks");
+        }
+        g_.sink = sink_ || has_sink_score_ ? (const float *)sinks_.ptr : nullptr;
         if (head_scale_) {
             // one kernel takes the largest raw score before the factor: it needs factors > 0
             std::vector<float> host((size_t)g_.nh);
@@ -437,7 +458,7 @@ public:
                                             qk_norm_ ? (const float *)k_norm_.ptr : nullptr, qk_eps_,
                                             rot ? position_->cos() : nullptr, rot ? position_->sin() : nullptr,
                                             rot / 2, ctx.row_pos, ctx.row_seq, cache.kv, g_, ctx.dtype,
-                                            rot && position_->pairs(), unit_norm_);
+                                            rot && position_->pairs(), unit_norm_, values_are_keys_);
             conv = Stack();
             const int32_t *blocks = prefill_blocks(ctx, decode);
             Buf a = ops::attention(d, q.ptr, n, cache.kv, g_, ctx.row_pos, ctx.row_seq, max_chunks, blocks,
@@ -550,6 +571,8 @@ private:
     bool qk_norm_ = false, score_bias_ = false;
     bool prepared_ = false;      // q and k are normed or rotated: qkv_prepare_append makes them
     bool gate_ = false, unit_norm_ = false;
+    bool values_are_keys_ = false, has_sink_score_ = false;
+    float sink_score_ = 0.0f;
     bool shared_ = false;        // the first product's rows went into a pair's shared first product
     int conv_taps_ = 0;
     long long gate_col0_ = 0;
@@ -579,7 +602,9 @@ private:
 //   z = Wdkv h;  c = rms(z[0:C]) wc;  kr = z[C:C+R]
 //   the first rotary_dim values of q's rotated part and of kr turn pair by pair
 //   (2i, 2i+1) with the position
-//   s_ij = (q_plain_i . (Wuk c_j)_head + q_rot_i . kr_j) * scale,  j <= i;  softmax
+//   (or, with a position part of kind rope_neox, value i with value i + rotary_dim / 2)
+//   s_ij = (q_plain_i . (Wuk c_j)_head + q_rot_i . kr_j) * scale,  j <= i and i - j < window;
+//   softmax, with a learned sink per head in the denominator (optional)
 //   out = Wo (concat_heads(sum_j p_ij (Wuv c_j)_head) * sigmoid(Wg h))     (the gate optional)
 //
 // The cache holds [c | kr] per position, once for all heads, and the values are read
@@ -590,16 +615,18 @@ private:
 // over rows gathered head by head (ops::linear_heads).
 //
 // A step of whole prompts in bfloat16 whose per-head sizes the tensor-core attention
-// kernel takes (D + R = Dv = 64 or 128) forms keys and values per head after all,
-// for that step alone, in pages of its own: [Wuk_head c | kr] and Wuv_head c are one
+// kernel takes (D + R and Dv up to 64 or up to 128, padded with zeros to that where they
+// are not; padded values want a mixer without a gate) forms keys and values per head after
+// all, for that step alone, in pages of its own: [Wuk_head c | kr] and Wuv_head c are one
 // product of the rows [c | kr] with a matrix made at load time (the heads' key and
 // value matrices with an identity for the shared part).  The cache gets the latents
 // as always, and decoding goes on from them.
 //
 // params: hidden_size, num_heads, head_dim (D), rot_dim (R), v_head_dim (Dv), kv_rank
 // (C), q_rank (Cq), scale, eps, gate (default true), per_head_prompts (default true:
-// false keeps prompts on the latents too), position (a part, kind rope_pairs), names
-// (optional): dq, dq_norm, uq, dkv, dkv_norm, uk, uv, gate, o
+// false keeps prompts on the latents too), window (0: none), sink (default false), position (a
+// part, kind rope_pairs or rope_neox), names (optional): dq, dq_norm, uq, dkv, dkv_norm, uk, uv,
+// gate, o, sink
 class LatentAttention : public Mixer {
 public:
     LatentAttention(const PartSpec &s, DType dt, Device *d) : Mixer(s, dt, d) {
@@ -641,9 +668,18 @@ public:
         g_.hd = (int)(C_ + R_);
         g_.vd = (int)C_;
         g_.scale = scale_;
+        g_.window = (int)s.get_int("window", 0);
+        if (g_.window < 0) config_error("latent_attention: window must not be negative");
+        sink_ = s.has("sink") && s.params.get("sink").as_bool();
+        n_sink_ = leaf("sink", "sink");
+        // the head size that prompts per head run with: the next one that the kernel takes
+        long long need = std::max(D_ + R_, Dv_);
+        P_ = need <= 64 ? 64 : need <= 128 ? 128 : 0;
+        if (gate_ && P_ != Dv_) P_ = 0;
     }
 
     void tensors(const std::string &p, TensorList &out) const override {
+        if (sink_) out.emplace_back(name(p, n_sink_), TensorSpec{{H_}, PARAM, false, 0.0f, 0.5f});
         out.emplace_back(name(p, n_dq_), TensorSpec{{Cq_, hidden_}, MATRIX, false});
         out.emplace_back(name(p, n_dqn_), TensorSpec{{Cq_}, PARAM, false, 1.0f, 0.1f});
         out.emplace_back(name(p, n_uq_), TensorSpec{{H_ * (D_ + R_), Cq_}, MATRIX, false});
@@ -672,9 +708,22 @@ public:
         w_uv_ = take(t, name(p, n_uv_));
         w_o_ = take(t, name(p, n_o_));
         position_->load(name(p, "position"), t);
-        if (per_head_prompts_ && dtype == BF16 && D_ + R_ == Dv_ && ops::attention_tc_ok(H_, H_, (int)Dv_) &&
-            w_uv_.dt == BF16 && w_ukT_.dt == BF16)
+        if (sink_) {
+            sinks_ = take(t, name(p, n_sink_));
+            g_.sink = (const float *)sinks_.ptr;
+        }
+        if (per_head_prompts_ && dtype == BF16 && P_ > 0 && ops::attention_tc_ok(H_, H_, (int)P_) &&
+            w_uv_.dt == BF16 && w_ukT_.dt == BF16 && w_o_.dt == BF16) {
             make_expander(take_back_uk());
+            if (P_ != Dv_) {
+                // the output matrix with every head's columns at its padded place
+                w_o_pad_ = dev->tensor(BF16, {hidden_, (long long)H_ * P_}, true);
+                cuda_check(cudaMemcpy2D(w_o_pad_.ptr, (size_t)P_ * 2, w_o_.ptr, (size_t)Dv_ * 2, (size_t)Dv_ * 2,
+                                        (size_t)(hidden_ * H_), cudaMemcpyDeviceToDevice),
+                           "placing the output matrix's columns");
+                dev->sync();
+            }
+        }
     }
 
     // [H D, C] once more out of its transposed form (load() has given the original back)
@@ -685,11 +734,12 @@ public:
     }
 
     // Rows [c | kr] times this matrix are, head by head, [Wuk_head c | kr], and after
-    // all heads' keys the values Wuv c: [H (D + R) + H Dv, C + R].
+    // all heads' keys the values Wuv c: [H P + H P, C + R], P the padded head size (the rows past
+    // D + R and past Dv are zeros).
     void make_expander(const DevTensor &uk) {
         size_t es = dtype_size(uk.dt);
-        long long W = C_ + R_, hd = D_ + R_;
-        w_expand_ = dev->tensor(uk.dt, {H_ * hd + H_ * Dv_, W}, true);
+        long long W = C_ + R_, hd = P_;
+        w_expand_ = dev->tensor(uk.dt, {2 * H_ * hd, W}, true);
         std::vector<uint16_t> eye((size_t)(R_ * R_), 0);
         for (long long i = 0; i < R_; i++) eye[(size_t)(i * R_ + i)] = 0x3f80;      // 1.0 in bfloat16
         char *dst = (char *)w_expand_.ptr;
@@ -700,18 +750,20 @@ public:
                 cuda_check(cudaMemcpy2D(dst + ((size_t)(h * hd + D_) * W + C_) * es, W * es, eye.data(), R_ * es,
                                         R_ * es, R_, cudaMemcpyHostToDevice), "placing the shared part's identity");
         }
-        cuda_check(cudaMemcpy2D(dst + (size_t)(H_ * hd) * W * es, W * es, w_uv_.ptr, C_ * es, C_ * es, H_ * Dv_,
-                                cudaMemcpyDeviceToDevice), "placing the value matrices");
+        for (int h = 0; h < H_; h++)
+            cuda_check(cudaMemcpy2D(dst + (size_t)((H_ + h) * hd) * W * es, W * es,
+                                    (const char *)w_uv_.ptr + (size_t)h * Dv_ * C_ * es, C_ * es, C_ * es, Dv_,
+                                    cudaMemcpyDeviceToDevice), "placing a head's value matrix");
         dev->sync();
     }
 
     size_t weight_bytes() const override {
         // (the matrix a prompt step uses instead of uk and uv is not read by a decode step)
         return w_in_.bytes() + w_uq_.bytes() + w_ukT_.bytes() + w_uv_.bytes() + w_o_.bytes() +
-               wq_norm_.bytes() + wc_norm_.bytes();
+               wq_norm_.bytes() + wc_norm_.bytes() + sinks_.bytes();
     }
 
-    KVSpec kv_spec() const override { return KVSpec{1, (int)(C_ + R_), 0, (int)C_, true}; }
+    KVSpec kv_spec() const override { return KVSpec{1, (int)(C_ + R_), g_.window, (int)C_, true}; }
 
     void prepare(long long n_positions) override {
         position_->prepare(n_positions);
@@ -737,16 +789,17 @@ public:
             return forward_per_head(ctx, P, cache, rot_half);
         Buf cq = ops::latent_down(d, P, 0, Cq_, (const float *)wq_norm_.ptr, Cq_, C_,
                                   (const float *)wc_norm_.ptr, R_, position_->cos(), position_->sin(), rot_half,
-                                  ctx.row_pos, ctx.row_seq, cache.kv, eps_, ctx.dtype);
+                                  ctx.row_pos, ctx.row_seq, cache.kv, eps_, ctx.dtype, nullptr, halves());
         Buf q_lat = d.pool.get((size_t)n * (size_t)H_ * (size_t)(C_ + R_) * esz);
         {
             Stack Q = ops::linear(d, cq.ptr, ctx.dtype, n, Cq_, w_uq_);
             Buf q_plain = ops::latent_q_split(d, Q, H_, D_, R_, C_, position_->cos(), position_->sin(), rot_half,
-                                              ctx.row_pos, q_lat.ptr, ctx.dtype);
+                                              ctx.row_pos, q_lat.ptr, ctx.dtype, true, halves());
             ops::HeadStack A = ops::linear_heads(d, q_plain.ptr, ctx.dtype, H_, n, D_, w_ukT_);
             ops::latent_q_join(d, A, R_, q_lat.ptr, ctx.dtype);
         }
         int max_chunks = (int)(ctx.max_pos / chunk_ + 1);
+        if (g_.window) max_chunks = std::min(max_chunks, (g_.window - 1) / chunk_ + 2);
         // the weighted sums of the latents, one head's rows together
         Buf o = ops::attention(d, q_lat.ptr, n, cache.kv, g_, ctx.row_pos, ctx.row_seq, max_chunks, nullptr, 0,
                                ctx.kind == DECODE, false, true);
@@ -761,17 +814,17 @@ public:
     Stack forward_per_head(StepContext &ctx, Stack &P, LayerCache &cache, int rot_half) {
         Device &d = *ctx.dev;
         long long n = ctx.n_rows;
-        int hd = (int)(D_ + R_);
+        int hd = (int)P_;
         Buf rows;
         Buf cq = ops::latent_down(d, P, 0, Cq_, (const float *)wq_norm_.ptr, Cq_, C_,
                                   (const float *)wc_norm_.ptr, R_, position_->cos(), position_->sin(), rot_half,
-                                  ctx.row_pos, ctx.row_seq, cache.kv, eps_, ctx.dtype, &rows);
-        // whole queries [n, H, D + R], the rotated part turned
+                                  ctx.row_pos, ctx.row_seq, cache.kv, eps_, ctx.dtype, &rows, halves());
+        // whole queries [n, H, P], the rotated part turned
         Buf q = d.pool.get((size_t)n * (size_t)H_ * (size_t)hd * 2);
         {
             Stack Q = ops::linear(d, cq.ptr, ctx.dtype, n, Cq_, w_uq_);
             ops::latent_q_split(d, Q, H_, D_, R_, D_, position_->cos(), position_->sin(), rot_half, ctx.row_pos,
-                                q.ptr, ctx.dtype, false);
+                                q.ptr, ctx.dtype, false, halves(), hd);
         }
         // pages of this step's own: every sequence starts at position 0 and gets the pages
         // it needs one after the other
@@ -805,6 +858,8 @@ public:
         g.nh = g.nkv = H_;
         g.hd = g.vd = hd;
         g.scale = scale_;
+        g.window = g_.window;
+        g.sink = g_.sink;
         int per = ops::attention_block_positions(g.nh, g.nkv);
         std::string key = "attention_blocks/" + std::to_string(per);
         auto it = ctx.extras.find(key);
@@ -815,10 +870,11 @@ public:
             it = ctx.extras.emplace(key, std::move(e)).first;
         }
         int max_chunks = (int)(ctx.max_pos / chunk_ + 1);
+        if (g.window) max_chunks = std::min(max_chunks, (g.window - 1) / chunk_ + 2);
         Buf o = ops::attention(d, q.ptr, n, own, g, ctx.row_pos, ctx.row_seq, max_chunks,
                                it->second.buf.as<int32_t>(), it->second.n, false);
         Buf a = gate_ ? ops::gate_rows(d, o.ptr, ctx.dtype, n, (long long)H_ * Dv_, P, Cq_ + C_ + R_) : std::move(o);
-        return ops::linear(d, a.ptr, ctx.dtype, n, (long long)H_ * Dv_, w_o_);
+        return ops::linear(d, a.ptr, ctx.dtype, n, (long long)H_ * P_, w_o_pad_ ? w_o_pad_ : w_o_);
     }
 
     Json info() const override {
@@ -831,7 +887,13 @@ public:
     }
 
 private:
-    long long hidden_, D_, R_, Dv_, C_, Cq_;
+    // the rotation's pairs are (i, i + rotary_dim / 2)
+    bool halves() const { return !position_->pairs(); }
+
+    long long hidden_, D_, R_, Dv_, C_, Cq_, P_ = 0;     // P: the head size of prompts per head (0: none)
+    bool sink_ = false;
+    std::string n_sink_;
+    DevTensor sinks_, w_o_pad_;
     int H_;
     float scale_, eps_;
     bool gate_;

@@ -1,6 +1,7 @@
 // Block arrangements.
 //
-// prenorm: x += mixer(norm(x)); x += ffn(norm(x))  (src/llm/model.c:743-796).
+// prenorm: x += mixer(norm(x)); x += ffn(norm(x))  (src/llm/model.c:743-796); a layer may have
+// no feed-forward.
 //
 // parallel: one norm, both sublayers read its output, and their results join the
 // residual stream together, times a factor:
@@ -27,7 +28,7 @@ class PreNormBlock : public Block {
 public:
     explicit PreNormBlock(BlockParts p) : Block(std::move(p)) {
         if (!mixer_norm) config_error("prenorm: the layer needs a norm in front of its mixer");
-        if (!feed_forward || !ffn_norm) config_error("prenorm: the layer needs a feed-forward and its norm");
+        if (feed_forward && !ffn_norm) config_error("prenorm: the feed-forward needs its norm");
         if (post_mixer_norm || post_ffn_norm) config_error("prenorm: the arrangement has no norms on results");
     }
     void forward(StepContext &ctx, float *x, Stack &pending, LayerCache &cache) override {
@@ -35,6 +36,10 @@ public:
         // the add of what the previous part produced is fused into the norm
         Buf h = mixer_norm->apply(ctx, x, n, ctx.dtype, pending ? &pending : nullptr, nullptr, 0);
         Stack d = mixer->forward(ctx, h.ptr, cache);
+        if (!feed_forward) {
+            pending = std::move(d);
+            return;
+        }
         h = ffn_norm->apply(ctx, x, n, ctx.dtype, &d, nullptr, 0);
         pending = feed_forward->forward(ctx, h.ptr);
     }

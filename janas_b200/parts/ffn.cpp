@@ -6,9 +6,22 @@
 
 namespace jb {
 
+// a gated unit's constants out of a part's parameter `key` (absent: SiLU(gate) * up)
+ops::UnitParams read_unit(const PartSpec &s, const std::string &key) {
+    ops::UnitParams u;
+    if (!s.has(key)) return u;
+    PartSpec p{s.kind + ": " + key, s.params.get(key)};
+    if (p.has("alpha")) u.alpha = (float)p.get_double("alpha");
+    if (p.has("limit")) u.limit = (float)p.get_double("limit");
+    if (p.has("shift")) u.shift = (float)p.get_double("shift");
+    if (u.limit < 0.0f) config_error(s.kind + ": a gated unit's limit must not be negative");
+    return u;
+}
+
 namespace {
 
-// params: hidden_size, intermediate_size, names (optional): gate, up, down
+// params: hidden_size, intermediate_size, unit (optional): {alpha, limit, shift}, another gated unit
+// than SiLU(gate) * up (see ops::UnitParams), names (optional): gate, up, down
 class SwiGLU : public FeedForward {
 public:
     // Rows from which gate, up and the activation run as one kernel.  Measured on
@@ -26,6 +39,7 @@ public:
         hidden_ = s.get_int("hidden_size");
         inter_ = s.get_int("intermediate_size");
         if (hidden_ <= 0 || inter_ <= 0) config_error("swiglu: sizes must be positive");
+        unit_ = read_unit(s, "unit");
         const Json &nm = s.params.get("names");
         auto leaf = [&](const char *key, const char *dflt) {
             return nm.is_object() && nm.get(key).is_string() ? nm.get(key).as_string() : std::string(dflt);
@@ -58,12 +72,12 @@ public:
             (n >= FUSED_FROM || (n <= FUSED_UP_TO && ops::linear_parts(n, 2 * inter_, hidden_) == 1))) {
             // enough rows, or enough features, to fill the SMs without cutting k:
             // gate, up and the activation in one kernel
-            act = ops::linear_swiglu(d, h, ctx.dtype, n, hidden_, w_gate_up_);
+            act = ops::linear_swiglu(d, h, ctx.dtype, n, hidden_, w_gate_up_, unit_);
             fused_last_ = (bool)act;
         }
         if (!act) {
             Stack gu = ops::linear(d, h, ctx.dtype, n, hidden_, w_gate_up_);
-            act = ops::swiglu(d, gu, ctx.dtype);
+            act = ops::swiglu(d, gu, ctx.dtype, unit_);
         }
         return ops::linear(d, act.ptr, ctx.dtype, n, inter_, w_down_);
     }
@@ -79,6 +93,7 @@ public:
 private:
     long long hidden_, inter_;
     std::string n_gate_, n_up_, n_down_;
+    ops::UnitParams unit_;
     DevTensor w_gate_up_, w_down_;
     bool fused_last_ = false;      // whether the last forward took the one-kernel way
 };

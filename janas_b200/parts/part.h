@@ -275,6 +275,9 @@ DevTensor fuse_rows(Device &dev, std::vector<DevTensor> &mats);
 // The same along the columns: matrices with equally many rows side by side.
 DevTensor fuse_cols(Device &dev, std::vector<DevTensor> &mats);
 
+// A gated feed-forward unit's constants, {alpha, limit, shift}, out of the parameter `key`.
+ops::UnitParams read_unit(const PartSpec &s, const std::string &key);
+
 // the built-in kinds (each file registers its own)
 void register_builtin_norms();
 void register_builtin_positions();

@@ -257,8 +257,17 @@ private:
 // q, k, v and the gate are one product over h; the recurrence, the state and the norm are
 // float32 in both compute types.
 //
+// Retention's form of it ("Retentive Network: A Successor to Transformer for Large Language
+// Models"), by the parameters activation, position, key_scale, head_norm and gate:
+//   q = turn(Wq h), k = turn(Wk h) key_scale, v = Wv h
+//   out = Wo (rms(each head of o) * silu(Wg h))           no weight in the norm
+//
 // params: hidden_size, heads, head_dim (D), v_head_dim (Dv, default D), decay (a list of one
-// number per head), eps, names (optional): q, k, v, g, o, norm
+// number per head), eps, activation ("silu", the default, or "none": of q, k and v), position (a
+// part, rope_neox or none; absent: none; goes with activation none), key_scale (default 1; on k
+// after the rotation; goes with activation none), head_norm (default false: one norm with a weight
+// over all heads; true: each head by its own root mean square, no weight), gate ("sigmoid", the
+// default, or "silu"), names (optional): q, k, v, g, o, norm
 class DecayAttention : public Mixer {
 public:
     DecayAttention(const PartSpec &s, DType dt, Device *d) : Mixer(s, dt, d) {
@@ -276,6 +285,22 @@ public:
             if (!dc[i].is_number()) config_error("decay_attention: decay must list numbers");
             decay_host_.push_back((float)dc[i].as_double());
         }
+        auto word = [&](const char *key, const char *dflt) {
+            return s.params.get(key).is_string() ? s.params.get(key).as_string() : std::string(dflt);
+        };
+        std::string act = word("activation", "silu"), gate = word("gate", "sigmoid");
+        if (act != "silu" && act != "none") config_error("decay_attention: activation is silu or none");
+        if (gate != "sigmoid" && gate != "silu") config_error("decay_attention: gate is sigmoid or silu");
+        silu_ = act == "silu";
+        gate_silu_ = gate == "silu";
+        head_norm_ = s.has("head_norm") && s.params.get("head_norm").as_bool();
+        key_scale_ = s.has("key_scale") ? (float)s.get_double("key_scale") : 1.0f;
+        if (s.has("position")) position_ = build_position(s.get_part("position"), dt, d);
+        bool turned = position_ && position_->rotary_dim() > 0;
+        if (silu_ && (turned || key_scale_ != 1.0f))
+            config_error("decay_attention: a rotation or a factor on the keys goes with activation none");
+        if (turned && (position_->rotary_dim() > D_ || position_->pairs()))
+            config_error("decay_attention: the rotation turns value i with value i + dims / 2, within a head");
         const Json &nm = s.params.get("names");
         auto leaf = [&](const char *key, const char *dflt) {
             return nm.is_object() && nm.get(key).is_string() ? nm.get(key).as_string() : std::string(dflt);
@@ -294,7 +319,8 @@ public:
         out.emplace_back(name(p, n_v_), TensorSpec{{H_ * Dv_, hidden_}, MATRIX, false});
         out.emplace_back(name(p, n_g_), TensorSpec{{H_ * Dv_, hidden_}, MATRIX, false});
         out.emplace_back(name(p, n_o_), TensorSpec{{hidden_, H_ * Dv_}, MATRIX, false});
-        out.emplace_back(name(p, n_norm_), TensorSpec{{H_ * Dv_}, PARAM, false, 1.0f, 0.1f});
+        if (!head_norm_) out.emplace_back(name(p, n_norm_), TensorSpec{{H_ * Dv_}, PARAM, false, 1.0f, 0.1f});
+        if (position_) position_->tensors(name(p, "position"), out);
     }
 
     void load(const std::string &p, TensorMap &t) override {
@@ -302,7 +328,8 @@ public:
                                      take(t, name(p, n_g_))};
         w_in_ = fuse_rows(*dev, in);
         w_o_ = take(t, name(p, n_o_));
-        norm_ = take(t, name(p, n_norm_));
+        if (!head_norm_) norm_ = take(t, name(p, n_norm_));
+        if (position_) position_->load(name(p, "position"), t);
         decay_ = dev->tensor(F32, {H_});
         cuda_check(cudaMemcpy(decay_.ptr, decay_host_.data(), decay_host_.size() * 4, cudaMemcpyHostToDevice),
                    "copying the heads' decays");
@@ -316,6 +343,9 @@ public:
         col0_ = col0;
     }
 
+    void prepare(long long n_positions) override {
+        if (position_) position_->prepare(n_positions);
+    }
     StateSpec state_spec() const override { return StateSpec{{H_ * D_ * Dv_}, F32}; }
     bool strided_state() const override { return true; }
     bool graph_safe() const override { return true; }
@@ -331,6 +361,10 @@ public:
         else if (!ctx.shared) fail(JB_LLM_EFAIL, "decay_attention: the shared first product is missing");
         const Stack &P = shared_ ? *ctx.shared : own;
         const long long c0 = shared_ ? col0_ : 0;
+        int rot = position_ ? position_->rotary_dim() : 0;
+        if (rot > 0 && ctx.max_pos >= position_->n_positions())
+            fail(JB_LLM_EINVAL, fmt("position %lld is beyond the %lld positions the encoding was prepared "
+                                    "for", ctx.max_pos, position_->n_positions()));
         ops::MatrixScan m;
         m.H = (int)H_;
         m.G = (int)H_;
@@ -339,17 +373,23 @@ public:
         m.qry_col0 = c0;
         m.key_col0 = c0 + H_ * D_;
         m.val_col0 = c0 + 2 * H_ * D_;
-        m.silu = true;
+        m.silu = silu_;
         m.decay = (const float *)decay_.ptr;
         // Many rows: q, k and v are activated once, ahead of the recurrence, whose blocks would
         // otherwise each activate the rows they read (several blocks read the same k and q).
         Stack act;
-        if (ctx.kind != DECODE && n >= 64) {
+        if (rot > 0 || key_scale_ != 1.0f) {
+            // the turned and scaled q and k (and v) in float32
+            act = ops::turn_heads(d, P, c0, (int)H_, D_, Dv_, rot ? position_->cos() : nullptr,
+                                  rot ? position_->sin() : nullptr, rot / 2, ctx.row_pos, key_scale_);
+        } else if (silu_ && ctx.kind != DECODE && n >= 64) {
             act.buf = ops::activation(d, P, 2 * H_ * D_ + H_ * Dv_, ops::activation_kind("silu"), F32, c0);
             act.S = 1;
             act.n = n;
             act.m = 2 * H_ * D_ + H_ * Dv_;
             m.silu = false;
+        }
+        if (act) {
             m.qry_col0 = 0;
             m.key_col0 = H_ * D_;
             m.val_col0 = 2 * H_ * D_;
@@ -357,8 +397,9 @@ public:
         Buf y = ops::matrix_state_scan(d, act ? act : P, m, (float *)cache.state, stride, ctx.row_seq, ctx.seq_slot,
                                        ctx.n_seqs, ctx.kind == DECODE, longest(ctx));
         act = Stack();
-        Buf a = ops::gated_part_norm(d, y.as<float>(), n, H_ * Dv_, 1, nullptr, 0, &P, c0 + 2 * H_ * D_ + H_ * Dv_,
-                                     (const float *)norm_.ptr, eps_, ctx.dtype, ctx.kind == DECODE && ctx.dtype == BF16);
+        Buf a = ops::gated_part_norm(d, y.as<float>(), n, H_ * Dv_, head_norm_ ? (int)H_ : 1, nullptr, 0, &P,
+                                     c0 + 2 * H_ * D_ + H_ * Dv_, head_norm_ ? nullptr : (const float *)norm_.ptr, eps_,
+                                     ctx.dtype, ctx.kind == DECODE && ctx.dtype == BF16, gate_silu_);
         own = Stack();
         return ops::linear(d, a.ptr, ctx.dtype, n, H_ * Dv_, w_o_);
     }
@@ -375,6 +416,9 @@ private:
     std::vector<float> decay_host_;
     std::string n_q_, n_k_, n_v_, n_g_, n_o_, n_norm_;
     DevTensor w_in_, w_o_, norm_, decay_;
+    bool silu_ = true, gate_silu_ = false, head_norm_ = false;
+    float key_scale_ = 1.0f;
+    std::unique_ptr<PositionEncoding> position_;
     bool shared_ = false;        // the [q | k | v | g] rows went into a pair's shared first product
     long long col0_ = 0;
 };

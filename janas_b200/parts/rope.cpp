@@ -16,6 +16,7 @@
 // heads and appends K and V (csrc/rope.cu); this part owns the constants and the
 // table.  Only the whole head can be rotated (rotary_dim == head size); the
 // reference's partial rotation (n_rot < head size) is not built.
+#include <algorithm>
 #include <cmath>
 
 #include "part.h"
@@ -24,7 +25,8 @@ namespace jb {
 
 namespace {
 
-// params: rotary_dim, theta, max_positions, scaling (optional): {factor, low, high, original}
+// params: rotary_dim, theta, max_positions, scaling (optional): {factor, low, high, original}, or
+// yarn (optional): {factor, original, fast, slow}
 class RopeNeox : public PositionEncoding {
 public:
     RopeNeox(const PartSpec &s, DType dt, Device *d, bool pairs = false) : PositionEncoding(s, dt, d), pairs_(pairs) {
@@ -62,6 +64,31 @@ public:
                 inv_freq_[(size_t)i] = (float)f;
             }
         }
+        if (s.has("yarn")) {
+            // YaRN ("YaRN: Efficient Context Window Extension of Large Language Models", Peng, Quesnelle,
+            // Fan, Shippole): the frequency at index i turns `original` positions into t(i) full turns;
+            // from the index of `fast` turns to the index of `slow` turns (both made whole) the
+            // frequencies go over from f to f / factor along a straight ramp, and cos and sin are
+            // multiplied by 0.1 ln(factor) + 1.
+            if (s.has("scaling")) config_error("rope: scaling and yarn exclude each other");
+            PartSpec yn{"", s.params.get("yarn")};
+            double factor = yn.get_double("factor"), original = yn.get_double("original");
+            double fast = yn.get_double("fast"), slow = yn.get_double("slow");
+            if (factor <= 0 || original <= 0 || fast <= 0 || slow <= 0 || theta_ <= 0 || theta_ == 1.0)
+                config_error("rope: yarn needs factor, original, fast, slow and theta above 0 and theta other than 1");
+            const double two_pi = 6.283185307179586476925286766559;
+            auto index_of = [&](double turns) {
+                return (double)rotary_dim_ * std::log(original / (two_pi * turns)) / (2.0 * std::log(theta_));
+            };
+            double lo = std::max(std::floor(index_of(fast)), 0.0);
+            double hi = std::min(std::ceil(index_of(slow)), (double)(rotary_dim_ - 1));
+            for (int i = 0; i < half; i++) {
+                double f = std::pow(theta_, -2.0 * (double)i / (double)rotary_dim_);
+                double ramp = std::min(std::max(((double)i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+                inv_freq_[(size_t)i] = (float)(f / factor * ramp + f * (1.0 - ramp));
+            }
+            amplitude_ = 0.1 * std::log(factor) + 1.0;
+        }
     }
 
     void prepare(long long n_positions) override {
@@ -74,7 +101,7 @@ public:
         cuda_check(cudaMemcpy(inv.ptr, inv_freq_.data(), (size_t)half * 4, cudaMemcpyHostToDevice),
                    "copying the rotation's frequencies");
         DevTensor c = dev->tensor(F32, {n, half}), s = dev->tensor(F32, {n, half});
-        ops::rope_table(*dev, (const float *)inv.ptr, half, n, (float *)c.ptr, (float *)s.ptr);
+        ops::rope_table(*dev, (const float *)inv.ptr, half, n, (float *)c.ptr, (float *)s.ptr, amplitude_);
         dev->sync();
         cos_ = c;
         sin_ = s;
@@ -99,7 +126,7 @@ public:
 private:
     int rotary_dim_;
     bool pairs_ = false;
-    double theta_;
+    double theta_, amplitude_ = 1.0;     // amplitude: a factor on cos and sin
     long long max_positions_;
     std::vector<float> inv_freq_;
     DevTensor cos_, sin_;

@@ -10,6 +10,11 @@
 //   out = sum_{chosen e < E} weight_e Wd_e act(Wu_e h) + (sum_{chosen e >= E} weight_e) h
 //         + Wd_shared act(Wu_shared h)
 //
+// score "chosen_softmax": the choice falls on the largest logits themselves (with router_bias, a
+// vector added to them), and the chosen experts' weights are the softmax over the chosen logits
+// alone, times scale.  With gated, an expert is Wd unit(Wg h, Wu h), the shared expert too (with
+// constants of its own).
+//
 // All experts' up matrices, the shared expert's and the router's rows are ONE matrix, so
 // one product over h gives every hidden value and the router's logits; the activation
 // kernel multiplies expert e's values by the token's weight for e (0 where e was not
@@ -21,6 +26,7 @@
 // The identity experts' term is not added here: it rides on the result as
 // Stack::skip (h with one coefficient per row) and is taken by the kernel that ends the
 // sublayer, or by ops::resolve_bias for any other consumer.
+#include "../csrc/kernels.h"
 #include "part.h"
 
 namespace jb {
@@ -31,10 +37,12 @@ namespace {
 // group_keep (default groups), scale (default 1), correction (default false: a vector
 // added to the scores for the choice alone), shared_ff (default 0: no shared expert),
 // activation ("relu2", "relu", "gelu_tanh", "silu"), gated (default false: an expert is
-// Wd (act(Wg h) * (Wu h)) with a gate matrix of its own), score ("softmax", the default, or
-// "sigmoid": each score the sigmoid of its own logit), group_best (default 1: a group's score
+// Wd (act(Wg h) * (Wu h)) with a gate matrix of its own; for silu, unit and shared_unit (optional):
+// {alpha, limit, shift}, the experts' and the shared expert's gated unit, see ops::UnitParams),
+// score ("softmax", the default, "sigmoid": each score the sigmoid of its own logit, or
+// "chosen_softmax"), router_bias (default false: a vector added to the logits), group_best (default 1: a group's score
 // is the sum of this many of its largest choice scores), names (optional): expert (a prefix,
-// the expert's index follows), gate, up, down, router, correction, shared
+// the expert's index follows), gate, up, down, router, router_bias, correction, shared
 class RoutedFFN : public FeedForward {
 public:
     RoutedFFN(const PartSpec &s, DType dt, Device *d) : FeedForward(s, dt, d) {
@@ -53,15 +61,21 @@ public:
         if (act_ < 0) config_error("routed: activation '" + act + "' is not one of relu2, relu, gelu_tanh, silu");
         gated_ = s.has("gated") && s.params.get("gated").as_bool();
         std::string score = s.params.get("score").is_string() ? s.params.get("score").as_string() : "softmax";
-        if (score != "softmax" && score != "sigmoid") config_error("routed: score '" + score + "' is not softmax or sigmoid");
-        sigmoid_ = score == "sigmoid";
+        if (score != "softmax" && score != "sigmoid" && score != "chosen_softmax")
+            config_error("routed: score '" + score + "' is not softmax, sigmoid or chosen_softmax");
+        score_ = score == "sigmoid" ? JB_SCORE_SIGMOID : score == "chosen_softmax" ? JB_SCORE_CHOSEN : JB_SCORE_SOFTMAX;
+        bias_ = s.has("router_bias") && s.params.get("router_bias").as_bool();
+        unit_ = read_unit(s, "unit");
+        shared_unit_ = read_unit(s, "shared_unit");
+        if ((s.has("unit") || s.has("shared_unit")) && (!gated_ || act != "silu"))
+            config_error("routed: a gated unit's constants are for gated experts with the activation silu");
         group_best_ = s.get_int("group_best", 1);
         if (group_best_ < 1) config_error("routed: group_best must be positive");
-        if (gated_ && s.get_int("shared_ff", 0) > 0) config_error("routed: experts with a gate and a shared expert together are not built");
         long long outs = experts_ + identity_;
         if (hidden_ <= 0 || experts_ < 0 || identity_ < 0 || outs <= 0 || (experts_ > 0 && ff_ <= 0) ||
             shared_ff_ < 0)
             config_error("routed: sizes must be positive");
+        if (gated_ && experts_ == 0) config_error("routed: gated needs experts with matrices");
         if (outs > 2048) config_error("routed: the router's kernel takes up to 2048 outputs");
         if (groups_ <= 0 || outs % groups_) config_error("routed: the router's outputs do not form equal groups");
         if (keep_ <= 0 || keep_ > groups_) config_error("routed: group_keep must be between 1 and groups");
@@ -75,13 +89,14 @@ public:
         n_up_ = leaf("up", "up_proj.weight");
         n_down_ = leaf("down", "down_proj.weight");
         n_router_ = leaf("router", "router.weight");
+        n_rbias_ = leaf("router_bias", "router.bias");
         n_corr_ = leaf("correction", "router.correction");
         n_shared_ = leaf("shared", "shared");
         n_gate_ = leaf("gate", "gate_proj.weight");
         // the columns of the first product: experts, shared expert, padding to a
         // multiple of 8 (so that every row of sums can be read four values at a time), router
         act_width_ = experts_ * ff_ + shared_ff_;
-        up_width_ = gated_ ? 2 * experts_ * ff_ : act_width_;
+        up_width_ = gated_ ? 2 * act_width_ : act_width_;
         router_col0_ = (up_width_ + 7) / 8 * 8;
     }
 
@@ -93,10 +108,13 @@ public:
             out.emplace_back(name(ep, n_down_), TensorSpec{{hidden_, ff_}, MATRIX, false});
         }
         out.emplace_back(name(p, n_router_), TensorSpec{{experts_ + identity_, hidden_}, MATRIX, false});
+        if (bias_)
+            out.emplace_back(name(p, n_rbias_), TensorSpec{{experts_ + identity_}, PARAM, false, 0.0f, 0.05f});
         if (correction_)
             out.emplace_back(name(p, n_corr_), TensorSpec{{experts_ + identity_}, PARAM, false, 0.0f, 0.05f});
         if (shared_ff_ > 0) {
             std::string sp = name(p, n_shared_);
+            if (gated_) out.emplace_back(name(sp, n_gate_), TensorSpec{{shared_ff_, hidden_}, MATRIX, false});
             out.emplace_back(name(sp, n_up_), TensorSpec{{shared_ff_, hidden_}, MATRIX, false});
             out.emplace_back(name(sp, n_down_), TensorSpec{{hidden_, shared_ff_}, MATRIX, false});
         }
@@ -112,6 +130,7 @@ public:
         }
         if (shared_ff_ > 0) {
             std::string sp = name(p, n_shared_);
+            if (gated_) ups.push_back(take(t, name(sp, n_gate_)));
             ups.push_back(take(t, name(sp, n_up_)));
             downs.push_back(take(t, name(sp, n_down_)));
         }
@@ -120,10 +139,11 @@ public:
         ups.push_back(router);
         w_up_ = fuse_rows(*dev, ups);
         if (!downs.empty()) w_down_ = fuse_cols(*dev, downs);
+        if (bias_) rbias_ = take(t, name(p, n_rbias_));
         if (correction_) corr_ = take(t, name(p, n_corr_));
     }
 
-    size_t weight_bytes() const override { return w_up_.bytes() + w_down_.bytes() + corr_.bytes(); }
+    size_t weight_bytes() const override { return w_up_.bytes() + w_down_.bytes() + corr_.bytes() + rbias_.bytes(); }
 
     Stack forward(StepContext &ctx, const void *h) override {
         Device &d = *ctx.dev;
@@ -137,14 +157,15 @@ public:
         r.first_identity = (int)experts_;
         r.scale = scale_;
         r.correction = correction_ ? (const float *)corr_.ptr : nullptr;
-        r.sigmoid_scores = sigmoid_;
+        r.score = score_;
+        r.bias = bias_ ? (const float *)rbias_.ptr : nullptr;
         r.group_best = (int)group_best_;
         Buf skip_coef;
         Buf weights = ops::moe_route(d, z, router_col0_, r, identity_ > 0 ? &skip_coef : nullptr);
         Stack out;
         if (act_width_ > 0) {
             Buf act = gated_ ? ops::gated_weighted(d, z, weights.as<float>(), (int)(experts_ + identity_),
-                                                   (int)experts_, ff_, act_, ctx.dtype)
+                                                   (int)experts_, ff_, act_, ctx.dtype, shared_ff_, unit_, shared_unit_)
                              : ops::activation_weighted(d, z, act_width_, weights.as<float>(),
                                                         (int)(experts_ + identity_), (int)experts_, ff_, act_,
                                                         ctx.dtype);
@@ -179,13 +200,15 @@ public:
 private:
     long long hidden_, experts_, ff_, identity_, top_, groups_, keep_, shared_ff_;
     long long act_width_ = 0, up_width_ = 0, router_col0_ = 0, group_best_ = 1;
-    bool gated_ = false, sigmoid_ = false;
+    bool gated_ = false, bias_ = false;
+    int score_ = JB_SCORE_SOFTMAX;
+    ops::UnitParams unit_, shared_unit_;
     std::string n_gate_;
     float scale_;
     bool correction_;
     int act_;
-    std::string n_expert_, n_up_, n_down_, n_router_, n_corr_, n_shared_;
-    DevTensor w_up_, w_down_, corr_;
+    std::string n_expert_, n_up_, n_down_, n_router_, n_rbias_, n_corr_, n_shared_;
+    DevTensor w_up_, w_down_, corr_, rbias_;
 };
 
 }  // namespace

@@ -11,6 +11,7 @@
     python bench.py --only dunavik [--design-size 4b]      (the Dunavik design beside Zuzelorn at equal sizes)
     python bench.py --only kefesun [--design-size 4b]      (the Kefesun design beside Dunavik's attention layers)
     python bench.py --only munisun [--design-size 4b]      (the Munisun design beside Kefesun's mixed layers)
+    python bench.py --only salivik [--design-size 4b]      (the Salivik design beside Munisun and Dunavik layers)
 
 The default run has the layer sizes of Qwen3-4B (36 layers, hidden 2560, 32
 heads, 8 KV heads, head size 128, feed-forward 9728, vocabulary 151936, tied
@@ -568,6 +569,81 @@ def munisun_flops(cfg, tokens):
     return asked + head, run + head
 
 
+def salivik_cfg(size, n_layers, vocab, mixers="mixed", window=1024):
+    """A Salivik config.json of the given layer sizes.  mixers: "attention", "retention" or "latent"
+    (every layer of that kind) or "mixed" (latent attention, attention, retention in turn, the second
+    and third layer run twice: n_layers layer runs of n_layers - 2 layers).  Every second layer's
+    feed-forward is routed: eight experts of an eighth of the dense width, two per token, and a shared
+    expert of an eighth; the others are dense.  The retention is as wide as the model (heads of the
+    size's head size); the latent layers have the sizes of the Dunavik ones."""
+    dm, nh, nkv, hd, ff = DESIGN_SIZES[size]
+    C, Cq, D, R = LATENT_SIZES[size]
+    unit = {"limit": 7.0}
+    moe = {"expert": dict(unit, ff=ff // 8), "kind": "moe", "router": {"experts": 8, "top": 2},
+           "shared": dict(unit, ff=ff // 8)}
+    kinds = ["latent", "attention", "retention"]
+    mixed = mixers == "mixed"
+    layers = []
+    for i in range(n_layers - 2 if mixed else n_layers):
+        kind = kinds[i % 3] if mixed else mixers
+        if kind == "attention":
+            layer = {"type": "attention", "mixer": {
+                "dim": hd, "heads": nh, "kv_heads": nkv, "mask": {"size": window}, "scale": hd ** -0.5, "vdim": hd,
+                "rot": {"base": 500000.0, "dims": hd // 2}}}
+        elif kind == "retention":
+            lh = dm // hd
+            layer = {"type": "retention", "mixer": {
+                "decay": [1.0 - 2.0 ** (-5.0 - 3.0 * a / max(1, lh - 1)) for a in range(lh)], "dim": hd, "heads": lh,
+                "vdim": hd, "rot": {"base": 500000.0, "dims": hd}}}
+        else:
+            layer = {"type": "latent_attention", "mixer": {
+                "dim": D, "heads": nh, "kv_rank": C, "q_rank": Cq, "rot_dim": R, "vdim": hd, "scale": (D + R) ** -0.5,
+                "mask": {"size": window},
+                "rot": {"base": 500000.0, "dims": R,
+                        "scaling": {"factor": 4.0, "fast": 32.0, "original": 4096, "slow": 1.0}}}}
+        layer["mlp"] = moe if i % 2 else dict(unit, ff=ff, kind="dense")
+        layers.append(layer)
+    return {"architecture": "Salivik", "layers": layers, "norm": {"eps": 1e-5}, "vocab": vocab, "width": dm,
+            "loop": {"start": 1, "stop": 3, "times": 2} if mixed else None}
+
+
+def salivik_flops(cfg, tokens):
+    """Multiply-adds times two of one prompt of a Salivik model: (what the design asks for: the chosen
+    experts' products; what the engine runs: every expert's for every token).  Both with the mixers'
+    products in the per-head form, the attention over the keys a row sees, the recurrences (4 N P per
+    head and token), the join in front of every pass and the head for one row."""
+    dm, asked, run = cfg["width"], 0.0, 0.0
+    n, lp = len(cfg["layers"]), cfg.get("loop")
+    order = list(range(n))
+    if lp:
+        order = order[:lp["start"]] + lp["times"] * order[lp["start"]:lp["stop"]] + order[lp["stop"]:]
+        asked = run = lp["times"] * 4.0 * dm * dm * tokens
+    for i in order:
+        layer, m = cfg["layers"][i], cfg["layers"][i]["mixer"]
+        H, D = m["heads"], m["dim"]
+        w = (m.get("mask") or {}).get("size") or tokens
+        pairs = sum(min(t + 1, w) for t in range(tokens))
+        if layer["type"] == "attention":
+            mats, attn = dm * D * (3 * H + m["kv_heads"]), 4 * H * D * pairs
+        elif layer["type"] == "retention":
+            mats, attn = dm * H * (2 * D + 3 * m["vdim"]), 4 * H * D * m["vdim"] * tokens
+        else:
+            R, Dv, C, Cq = m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+            mats = dm * (Cq + C + R) + Cq * H * (D + R) + C * H * (D + Dv) + H * Dv * dm
+            attn = 2 * H * (D + R + Dv) * pairs
+        f = layer["mlp"]
+        if f["kind"] == "dense":
+            up = up_run = 3 * dm * f["ff"]
+        else:
+            ro, ef, sf = f["router"], f["expert"]["ff"], (f.get("shared") or {}).get("ff", 0)
+            up = dm * ro["experts"] + 3 * dm * (ro["top"] * ef + sf)
+            up_run = dm * ro["experts"] + 3 * dm * (ro["experts"] * ef + sf)
+        asked += 2 * (mats + up) * tokens + attn
+        run += 2 * (mats + up_run) * tokens + attn
+    head = 2 * dm * cfg["vocab"]
+    return asked + head, run + head
+
+
 def qwen3_cfg(size, n_layers, vocab, max_positions):
     dm, nh, nkv, hd, ff = DESIGN_SIZES[size]
     return dict(QWEN3_4B, num_hidden_layers=n_layers, hidden_size=dm, num_attention_heads=nh,
@@ -652,6 +728,13 @@ def design_compare(args):
             designs = [("kefesun-mixed", kefesun_cfg(size, n_layers, vocab, "mixed", args.window))]
             designs += [(f"munisun-{mx}", munisun_cfg(size, n_layers, vocab, mx))
                         for mx in args.mixers.replace("attention", "parallel").replace("latent", "parallel2").split(",")]
+        if args.only == "salivik":
+            # beside Munisun's linear-attention layers (a recurrence with a decay per head, gated
+            # routed experts, RMS norms) and Dunavik's latent layers
+            designs = [("munisun-parallel2", munisun_cfg(size, n_layers, vocab, "parallel2")),
+                       ("dunavik-latent", dunavik_cfg(size, n_layers, vocab, "latent", args.window))]
+            kinds = args.mixers + ",retention" if args.mixers == ap_default_mixers() else args.mixers
+            designs += [(f"salivik-{mx}", salivik_cfg(size, n_layers, vocab, mx, args.window)) for mx in kinds.split(",")]
         for design, cfg in designs:
             rng = np.random.default_rng(0)
             eng = Engine.open_random(cfg, seed=0, dtype=args.dtype, max_tokens=max(room * batch, T + 64),
@@ -662,6 +745,8 @@ def design_compare(args):
                 flops, flops_run = kefesun_flops(cfg, T)
             elif design.startswith("munisun"):
                 flops, flops_run = munisun_flops(cfg, T)
+            elif design.startswith("salivik"):
+                flops, flops_run = salivik_flops(cfg, T)
             else:
                 flops = (dunavik_flops(cfg, T, args.window) if design.startswith("dunavik")
                          else design_flops(design.split("-")[0], size, n_layers, T, vocab))
@@ -704,6 +789,10 @@ def design_compare(args):
     return 0
 
 
+def ap_default_mixers():
+    return "mixed,attention,latent"
+
+
 def other_config(model, extra):
     """Runs this program for another model size in a process of its own (its
     weights and cache are given back when it ends); returns its JSON line."""
@@ -732,7 +821,7 @@ def main():
                     help="skip decoding at batch 1 and 64 and the 32-bit points")
     ap.add_argument("--all-configs", action="store_true",
                     help="also the 8B workload (unequal prompts, 256 steps) and the 32B points")
-    ap.add_argument("--mixers", default="mixed,attention,latent",
+    ap.add_argument("--mixers", default=ap_default_mixers(),
                     help="--only dunavik: which layer mixes to run (mixed, attention, latent), with commas")
     ap.add_argument("--window", type=int, default=1024, help="--only dunavik: the attention layers' window")
     ap.add_argument("--design-size", default="", choices=[""] + sorted(DESIGN_SIZES),
@@ -740,7 +829,7 @@ def main():
     ap.add_argument("--share", type=int, default=0,
                     help="--only zuzelorn: also a model whose layers share keys and values in groups of this many")
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "timeline", "prefill-timeline", "generate",
-                                                    "zuzelorn", "dunavik", "kefesun", "munisun"],
+                                                    "zuzelorn", "dunavik", "kefesun", "munisun", "salivik"],
                     help="run one part only and print its time (for profiling; no JSON line "
                          "but for generate); prefill-timeline: each kernel's share of one prefill "
                          "step; timeline: when each kernel of one replayed decode "
@@ -758,7 +847,7 @@ def main():
     if args.gpus != 1:
         print("bench.py: this engine runs on one GPU; --gpus must be 1")
         return 2
-    if args.only in ("zuzelorn", "dunavik", "kefesun", "munisun"):
+    if args.only in ("zuzelorn", "dunavik", "kefesun", "munisun", "salivik"):
         args.warmup = max(args.warmup, 3)
         return design_compare(args)
     full_layers = MODELS[args.model]["num_hidden_layers"]

@@ -107,14 +107,6 @@ __device__ __forceinline__ float add_partials(float v, const float *__restrict__
     return v;
 }
 
-// Programmatic dependent launch.  Every kernel of this library is launched with
-// the attribute that lets its CTAs start while the kernel before it in the
-// stream is still running.  pdl_trigger() (early in a kernel) allows the next
-// kernel's CTAs to be scheduled once all of this kernel's CTAs have started;
-// pdl_wait() blocks until the kernel before this one has completed and its
-// writes are visible.  What a kernel does before pdl_wait() must not touch
-// anything an earlier kernel writes or reads-and-frees: only its own shared and
-// tensor memory and the (immutable) weights.
 // A gated unit of a feed-forward: g sigmoid(alpha g) (u + shift), with limit > 0 both sides cut
 // off first: g <- min(g, limit), u <- clamp(u, -limit, limit).  {1, 0, 0} is SiLU(g) u.
 struct GatedUnit {
@@ -129,6 +121,14 @@ __device__ __forceinline__ float gated_unit(float g, float u, const GatedUnit &p
     return g / (1.0f + expf(-p.alpha * g)) * (u + p.shift);
 }
 
+// Programmatic dependent launch.  Every kernel of this library is launched with
+// the attribute that lets its CTAs start while the kernel before it in the
+// stream is still running.  pdl_trigger() (early in a kernel) allows the next
+// kernel's CTAs to be scheduled once all of this kernel's CTAs have started;
+// pdl_wait() blocks until the kernel before this one has completed and its
+// writes are visible.  What a kernel does before pdl_wait() must not touch
+// anything an earlier kernel writes or reads-and-frees: only its own shared and
+// tensor memory and the (immutable) weights.
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_trigger()
 {

@@ -141,11 +141,110 @@ __global__ void latent_q_split_kernel(const float *__restrict__ Q, int S, size_t
 __device__ __forceinline__ float4 sum4(const float *__restrict__ p, int S, size_t stride)
 {
     float4 v = load4(p);
-    for (int s = 1; s < S; s++) {
-        float4 w = load4(p + (size_t)s * stride);
-        v = make_float4(v.x + w.x, v.y + w.y, v.z + w.z, v.w + w.w);
+    for (int s0 = 1; s0 < S; s0 += 4) {
+        // four terms fetched together, added in order
+        float4 w[4];
+#pragma unroll
+        for (int u = 0; u < 4; u++)
+            w[u] = s0 + u < S ? load4(p + (size_t)(s0 + u) * stride) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+        for (int u = 0; u < 4; u++)
+            if (s0 + u < S)
+                v = make_float4(v.x + w[u].x, v.y + w[u].y, v.z + w[u].z, v.w + w[u].w);
     }
     return v;
+}
+
+// latent_down with four neighbouring values of the row to a thread at a time, up to U times, all
+// held in registers: both sums of squares cross the block together, and the shared key part
+// passes through shared memory for the rotation.  q_rank, kv_rank, rot_dim and the columns are
+// multiples of four.
+template <typename TC, int U>
+__global__ void __launch_bounds__(128)
+latent_down_vec_kernel(const float *__restrict__ P, int S, size_t stride, int ld, int q_col0, int q_rank,
+                       const float *__restrict__ wq, int kv_col0, int kv_rank,
+                       const float *__restrict__ wkv, int rot_dim, const float *__restrict__ cs,
+                       const float *__restrict__ sn, int rot_half, const int32_t *__restrict__ row_pos,
+                       const int32_t *__restrict__ row_seq, const int32_t *__restrict__ block_table,
+                       int bt_stride, TC *__restrict__ cq_out, TC *__restrict__ k_cache,
+                       TC *__restrict__ rows_out, float eps, int halves)
+{
+    extern __shared__ __align__(16) float zr[];      // rot_dim sums of this row
+    __shared__ float red[2][4];
+    pdl_trigger();
+    size_t row = blockIdx.x;
+    int pos = row_pos[row];
+    int page = block_table[(size_t)row_seq[row] * bt_stride + pos / PAGE];
+    int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int both = q_rank + kv_rank, all = both + rot_dim;
+    pdl_wait();
+    const float *pq = P + row * ld + q_col0, *pc = P + row * ld + kv_col0 - q_rank;
+    float4 v[U];
+    float sq = 0.0f, sc = 0.0f;
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+        int i = 4 * (threadIdx.x + 128 * u);
+        if (i >= all)
+            continue;
+        v[u] = sum4(i < q_rank ? pq + i : pc + i, S, stride);
+        float ss = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, fmaf(v[u].z, v[u].z, v[u].w * v[u].w)));
+        if (i < q_rank)
+            sq += ss;
+        else if (i < both)
+            sc += ss;
+        else
+            store4(zr + i - both, v[u]);
+    }
+    sq = warp_sum(sq);
+    sc = warp_sum(sc);
+    if (lane == 0) {
+        red[0][warp] = sq;
+        red[1][warp] = sc;
+    }
+    __syncthreads();
+    sq = red[0][0] + red[0][1] + red[0][2] + red[0][3];
+    sc = red[1][0] + red[1][1] + red[1][2] + red[1][3];
+    float iq = 1.0f / sqrtf(sq / (float)max(q_rank, 1) + eps), ic = 1.0f / sqrtf(sc / (float)kv_rank + eps);
+    int hd = kv_rank + rot_dim;
+    TC *dst = k_cache + ((size_t)page * PAGE + pos % PAGE) * hd;
+    TC *dst2 = rows_out != nullptr ? rows_out + row * hd : nullptr;
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+        int i = 4 * (threadIdx.x + 128 * u);
+        if (i >= all)
+            continue;
+        if (i < both) {
+            bool is_q = i < q_rank;
+            float4 w = load4(is_q ? wq + i : wkv + i - q_rank);
+            float inv = is_q ? iq : ic;
+            float4 o = make_float4(v[u].x * inv * w.x, v[u].y * inv * w.y, v[u].z * inv * w.z, v[u].w * inv * w.w);
+            if (is_q) {
+                store4(cq_out + row * q_rank + i, o);
+            } else {
+                store4(dst + i - q_rank, o);
+                if (dst2 != nullptr)
+                    store4(dst2 + i - q_rank, o);
+            }
+            continue;
+        }
+        int e0 = i - both;
+        float o[4] = {v[u].x, v[u].y, v[u].z, v[u].w};
+#pragma unroll
+        for (int k = 0; k < 4; k++) {
+            int e = e0 + k;
+            if (e < 2 * rot_half) {
+                bool high = halves ? e >= rot_half : (e & 1) != 0;
+                int f = halves ? (high ? e - rot_half : e) : e / 2;
+                float c = cs[(size_t)pos * rot_half + f], s = sn[(size_t)pos * rot_half + f];
+                float other = zr[halves ? (high ? e - rot_half : e + rot_half) : e ^ 1];
+                o[k] = high ? fmaf(o[k], c, other * s) : fmaf(o[k], c, -other * s);
+            }
+        }
+        float4 t = make_float4(o[0], o[1], o[2], o[3]);
+        store4(dst + i - q_rank, t);
+        if (dst2 != nullptr)
+            store4(dst2 + i - q_rank, t);
+    }
 }
 
 // latent_q_split with four neighbouring values of a head per thread (D, R and C multiples
@@ -396,6 +495,30 @@ extern "C" int jb_latent_down_rows(const float *P, int S, long long stride, int 
     size_t smem = (size_t)(q_rank + kv_rank + rot_dim) * 4;
     if (smem > 48 * 1024)
         return JB_EINVAL;
+    size_t esz = cache_dt == JB_F32 ? 4 : 2;
+    auto at = [](const void *p, size_t to) { return (uintptr_t)p % to == 0; };
+    int quads = (q_rank + kv_rank + rot_dim) / 4, U = (quads + 127) / 128;
+    if (q_rank % 4 == 0 && kv_rank % 4 == 0 && rot_dim % 4 == 0 && q_col0 % 4 == 0 && kv_col0 % 4 == 0 && ld % 4 == 0 &&
+        stride % 4 == 0 && at(P, 16) && at(wq, 16) && at(wkv, 16) && at(cq_out, 4 * esz) && at(k_cache, 4 * esz) &&
+        at(rows_out, 4 * esz) && U <= 8 && (cache_dt == JB_F32 || cache_dt == JB_BF16)) {
+#define JB_LDV(TC, UU)                                                                                       \
+    launch(latent_down_vec_kernel<TC, UU>, n, 128, (size_t)rot_dim * 4, st, P, S, (size_t)stride, ld, q_col0,  \
+           q_rank, wq, kv_col0, kv_rank, wkv, rot_dim, cs, sn, rot_half, row_pos, row_seq, block_table,      \
+           bt_stride, (TC *)cq_out, (TC *)k_cache, (TC *)rows_out, eps, halves)
+#define JB_LDV_U(TC)                          \
+    do {                                      \
+        if (U <= 2) JB_LDV(TC, 2);            \
+        else if (U <= 4) JB_LDV(TC, 4);       \
+        else JB_LDV(TC, 8);                   \
+    } while (0)
+        if (cache_dt == JB_F32)
+            JB_LDV_U(float);
+        else
+            JB_LDV_U(bf16);
+#undef JB_LDV_U
+#undef JB_LDV
+        return launch_status();
+    }
 #define JB_LD(TC, ONE)                                                                          \
     launch(latent_down_kernel<TC, ONE>, n, 256, smem, st, P, S, (size_t)stride, ld, q_col0, q_rank, wq, \
            kv_col0, kv_rank, wkv, rot_dim, cs, sn, rot_half, row_pos, row_seq, block_table,      \

@@ -474,60 +474,79 @@ gated_part_norm_warp_kernel(const float *__restrict__ y, const float *__restrict
 // q, k and v of a linear attention ahead of its recurrence, float32: out[r] = [q | k | v] from the
 // sums' columns col0 .. (H D, H D and H Dv values), with the first 2 rot_half values of every q and
 // k head turned (value i with value i + rot_half, angle tables [position, i]) and k times key_scale
-// after that.  VEC values per thread: 4 where D, Dv and rot_half are multiples of four and
-// everything lies on 16-byte boundaries.
+// after that.  A thread has VEC neighbouring values, and where they turn their partners too.  VEC
+// is 4 where D, Dv and rot_half are multiples of four and everything lies on 16-byte boundaries.
+template <int VEC>
+__device__ __forceinline__ void turn_load(const float *p, int S, size_t stride, float (&v)[VEC])
+{
+    if (VEC == 4) {
+        float4 a = load4(p);
+        for (int k = 1; k < S; k++) {
+            float4 t = load4(p + (size_t)k * stride);
+            a = make_float4(a.x + t.x, a.y + t.y, a.z + t.z, a.w + t.w);
+        }
+        v[0] = a.x; v[1 % VEC] = a.y; v[2 % VEC] = a.z; v[3 % VEC] = a.w;
+    } else {
+        v[0] = add_partials(0.0f, p, S, stride);
+    }
+}
+
+template <int VEC>
+__device__ __forceinline__ void turn_store(float *p, const float (&v)[VEC])
+{
+    if (VEC == 4)
+        store4(p, make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]));
+    else
+        p[0] = v[0];
+}
+
 template <int VEC>
 __global__ void __launch_bounds__(256)
 turn_heads_kernel(const float *__restrict__ src, int S, size_t stride, int ld, int col0, int H, int D, int Dv,
                   const float *__restrict__ cs, const float *__restrict__ sn, int rot_half,
-                  const int32_t *__restrict__ row_pos, float key_scale, float *__restrict__ out, int width)
+                  const int32_t *__restrict__ row_pos, float key_scale, float *__restrict__ out, int width,
+                  int units)
 {
     pdl_trigger();
-    int r = blockIdx.x, c = (int)(blockIdx.y * blockDim.x + threadIdx.x) * VEC;
-    if (c >= width)
+    // a row's units: per q and k head the turned pairs, then the values that stay; then v
+    int r = blockIdx.x, u = (int)(blockIdx.y * blockDim.x + threadIdx.x);
+    if (u >= units)
         return;
-    int d = c < 2 * H * D ? c % D : 2 * rot_half;          // v is not turned
-    bool turned = d < 2 * rot_half, high = d >= rot_half;
-    float f = c >= H * D && c < 2 * H * D ? key_scale : 1.0f;
+    int pairs = rot_half / VEC, per = D / VEC - pairs;
+    bool is_v = u >= 2 * H * per;
+    int h = is_v ? 0 : u / per, i = is_v ? u - 2 * H * per : u - h * per;
+    bool turned = !is_v && i < pairs;
+    // the first value's column: pair i, or what lies behind the turned part
+    int c = is_v ? 2 * H * D + i * VEC : h * D + (turned ? i : pairs + i) * VEC;
+    float f = !is_v && h >= H ? key_scale : 1.0f;
     float co[VEC], si[VEC];
     if (turned) {
-        size_t at = (size_t)row_pos[r] * rot_half + (high ? d - rot_half : d);
+        size_t at = (size_t)row_pos[r] * rot_half + (size_t)i * VEC;
 #pragma unroll
-        for (int u = 0; u < VEC; u++) {
-            co[u] = cs[at + u];
-            si[u] = high ? sn[at + u] : -sn[at + u];
+        for (int e = 0; e < VEC; e++) {
+            co[e] = cs[at + e];
+            si[e] = sn[at + e];
         }
     }
     pdl_wait();
-    const float *p = src + (size_t)r * ld + col0 + c, *o = p + (high ? -rot_half : rot_half);
+    const float *p = src + (size_t)r * ld + col0 + c;
+    float *dst = out + (size_t)r * width + c;
     float v[VEC], w[VEC];
-    if (VEC == 4) {
-        float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f), b = a;
-        for (int k = 0; k < S; k++) {
-            float4 t = load4(p + (size_t)k * stride);
-            a = make_float4(a.x + t.x, a.y + t.y, a.z + t.z, a.w + t.w);
-            if (turned) {
-                t = load4(o + (size_t)k * stride);
-                b = make_float4(b.x + t.x, b.y + t.y, b.z + t.z, b.w + t.w);
-            }
+    turn_load<VEC>(p, S, stride, v);
+    if (turned) {
+        turn_load<VEC>(p + rot_half, S, stride, w);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) {
+            float a = v[e], b = w[e];
+            v[e] = fmaf(a, co[e], -(b * si[e]));
+            w[e] = fmaf(b, co[e], a * si[e]) * f;
         }
-        v[0] = a.x; v[1 % VEC] = a.y; v[2 % VEC] = a.z; v[3 % VEC] = a.w;
-        w[0] = b.x; w[1 % VEC] = b.y; w[2 % VEC] = b.z; w[3 % VEC] = b.w;
-    } else {
-        v[0] = add_partials(0.0f, p, S, stride);
-        w[0] = turned ? add_partials(0.0f, o, S, stride) : 0.0f;
+        turn_store<VEC>(dst + rot_half, w);
     }
 #pragma unroll
-    for (int u = 0; u < VEC; u++) {
-        if (turned)
-            v[u] = fmaf(v[u], co[u], w[u] * si[u]);
-        v[u] *= f;
-    }
-    float *dst = out + (size_t)r * width + c;
-    if (VEC == 4)
-        store4(dst, make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]));
-    else
-        dst[0] = v[0];
+    for (int e = 0; e < VEC; e++)
+        v[e] *= f;
+    turn_store<VEC>(dst, v);
 }
 
 // The same for few rows: a cluster of C CTAs per (row, part), each with `cols` columns of the part
@@ -869,16 +888,19 @@ extern "C" int jb_turn_heads(const float *src, int S, long long stride, int ld, 
         return JB_EINVAL;
     bool vec = D % 4 == 0 && Dv % 4 == 0 && rot_half % 4 == 0 && ld % 4 == 0 && stride % 4 == 0 && col0 % 4 == 0 &&
                (uintptr_t)src % 16 == 0 && (uintptr_t)out % 16 == 0;
-    long long per_row = vec ? width / 4 : width;
-    if ((per_row + 255) / 256 > 65535)
+    const int V = vec ? 4 : 1;
+    long long units = 2ll * H * (D / V - rot_half / V) + (long long)H * (Dv / V);
+    // few rows: smaller blocks, so that a row's units spread over more SMs
+    const int threads = n <= 64 ? 64 : 256;
+    if ((units + threads - 1) / threads > 65535)
         return JB_EINVAL;
-    dim3 grid((unsigned)n, (unsigned)((per_row + 255) / 256));
+    dim3 grid((unsigned)n, (unsigned)((units + threads - 1) / threads));
     if (vec)
-        launch(turn_heads_kernel<4>, grid, 256, 0, st, src, S, (size_t)stride, ld, col0, H, D, Dv, cs, sn, rot_half,
-               row_pos, key_scale, out, (int)width);
+        launch(turn_heads_kernel<4>, grid, threads, 0, st, src, S, (size_t)stride, ld, col0, H, D, Dv, cs, sn, rot_half,
+               row_pos, key_scale, out, (int)width, (int)units);
     else
-        launch(turn_heads_kernel<1>, grid, 256, 0, st, src, S, (size_t)stride, ld, col0, H, D, Dv, cs, sn, rot_half,
-               row_pos, key_scale, out, (int)width);
+        launch(turn_heads_kernel<1>, grid, threads, 0, st, src, S, (size_t)stride, ld, col0, H, D, Dv, cs, sn, rot_half,
+               row_pos, key_scale, out, (int)width, (int)units);
     return launch_status();
 }
 

@@ -1,5 +1,6 @@
 // Causal grouped-query attention over the paged cache on the tensor cores
-// (tcgen05), for bfloat16 heads of 64 or 128 values.  Keys and values come in
+// (tcgen05), for bfloat16 heads of 64 or 128 values (prompts also with keys of 192 and
+// values of 128).  Keys and values come in
 // chunks of 128 positions, two cache pages, straight from the pages into shared
 // memory by TMA; V is read as an MN-major operand as it lies in the page
 // ([position][value]).  Three kernels:
@@ -386,28 +387,33 @@ attn_tc_rows_kernel(const __grid_constant__ CUtensorMap map_q,
 // float range); then the row thread scales its row of O and its sum by
 // 2^(m_old - m_new) before it hands P over.  After the first chunks that is rare.
 //
-// Tensor memory: S_A [0, 128), S_B [128, 256), O_A [256, 256 + HD), O_B after it.
+// Tensor memory: S_A [0, 128), S_B [128, 256), O_A [256, 256 + VD), O_B after it.
 // Shared memory: Q_A, Q_B, P_A, P_B, and a ring of three units that hold keys and
 // values in the order of their use: K0 K1 V0 K2 V1 K3 ...
+//
+// Keys (and queries) of KD values, values of VD.  Keys of 192 leave room for one block of
+// 128 rows alone: its runs hold R positions instead of 2 R.
 constexpr int PF_THREADS = 320;     // warp 0 loads, warp 1 issues MMAs, 2..5 rows of A, 6..9 of B
 constexpr int PF_UNITS = 3;
 constexpr float PF_LAZY = 8.0f;     // how far (in powers of two) a maximum may run ahead of m
 
-template <int HD> struct PrefillCfg {
-    static constexpr int NB = HD / 64;
-    static constexpr int Q_TILE = NB * BLK_BYTES;          // 128 rows x HD
+template <int KD, int VD> struct PrefillCfg {
+    static constexpr int TILES = KD > 128 ? 1 : 2;         // blocks of rows
+    static constexpr int NBK = KD / 64, NBV = VD / 64;
+    static constexpr int Q_TILE = NBK * BLK_BYTES;         // 128 rows x KD
     static constexpr int P_TILE = 2 * BLK_BYTES;           // 128 rows x 128 keys
-    static constexpr int UNIT = NB * BLK_BYTES;            // 128 positions x HD
+    static constexpr int UNIT = (NBK > NBV ? NBK : NBV) * BLK_BYTES;      // 128 positions x KD (or VD)
     static constexpr int TAIL = 3072;                      // barriers and the like
-    static constexpr int SMEM_BYTES = 2 * Q_TILE + 2 * P_TILE + PF_UNITS * UNIT + TAIL;
+    static constexpr int SMEM_BYTES = TILES * (Q_TILE + P_TILE) + PF_UNITS * UNIT + TAIL;
     static constexpr int TMEM_COLS = 512;
+    static_assert(SMEM_BYTES <= 227 * 1024, "more shared memory than a block may have");
 };
 
 // MODE 0: softmax; 1: softmax of scores with a cap or slopes (ScoreExt); 2: weights that are
 // sigmoid(score + score_bias[head]), not normalized over the keys.  keep_first > 0 (with a
 // window): the first keep_first positions stay visible beside the window; their chunks, as
 // far as they lie before the run's first chunk, come first in the CTA's order of chunks.
-template <int HD, int MODE>
+template <int KD, int VD, int MODE>
 __global__ void __launch_bounds__(PF_THREADS, 1)
 attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
                        const __grid_constant__ CUtensorMap map_k,
@@ -418,13 +424,12 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
                        const float *__restrict__ sink, const ScoreExt x, int keep_first,
                        const float *__restrict__ score_bias)
 {
-    using Cfg = PrefillCfg<HD>;
-    constexpr int NB = Cfg::NB;
+    using Cfg = PrefillCfg<KD, VD>;
     constexpr bool EXT = MODE == 1, SIG = MODE == 2;
     extern __shared__ __align__(1024) uint8_t smem[];
-    uint8_t *q_s = smem;                           // two tiles
-    uint8_t *p_s = q_s + 2 * Cfg::Q_TILE;          // two tiles
-    uint8_t *kv_s = p_s + 2 * Cfg::P_TILE;
+    uint8_t *q_s = smem;                                    // a tile per block of rows
+    uint8_t *p_s = q_s + Cfg::TILES * Cfg::Q_TILE;          // the same
+    uint8_t *kv_s = p_s + Cfg::TILES * Cfg::P_TILE;
     uint64_t *bars = (uint64_t *)(kv_s + PF_UNITS * Cfg::UNIT);
     // bars: 0 q_full | 1..3 unit full | 4..6 unit free | 7,8 s_full A,B | 9,10 p_full A,B |
     //       11,12 pv_done A,B | 13,14 s_free A,B
@@ -442,7 +447,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
     int kvh = blockIdx.x % nkv;
     const int32_t *b = qblk + 4 * (blockIdx.x / nkv);
     int q_row = b[0], q_count = b[1], q_pos = b[2], seq = b[3];
-    bool has_b = q_count > R;                                    // the second block has rows
+    bool has_b = Cfg::TILES == 2 && q_count > R;                 // the second block has rows
     int lo0 = window > 0 && q_pos + 1 > window ? q_pos + 1 - window : 0;
     int c_first = lo0 / AT_KEYS;
     int c_last = (q_pos + q_count - 1) / AT_KEYS;
@@ -486,10 +491,10 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
 
     if (warp == 0 && lane == 0) {
         // ---------------------------------------------------------- TMA loads
-        mbar_expect_tx(bar(0), (uint32_t)((has_b ? 2 : 1) * R * G * HD * 2));
+        mbar_expect_tx(bar(0), (uint32_t)((has_b ? 2 : 1) * R * G * KD * 2));
         for (int t = 0; t < (has_b ? 2 : 1); t++)
 #pragma unroll
-            for (int bb = 0; bb < NB; bb++)
+            for (int bb = 0; bb < Cfg::NBK; bb++)
                 tma_load_3d(smem_u32(q_s + t * Cfg::Q_TILE + bb * BLK_BYTES), &map_q, bar(0),
                             bb * 64, kvh * G, q_row + t * R);
         const int32_t *bt = block_table + (size_t)seq * bt_stride;
@@ -499,9 +504,10 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
             uint32_t ph = (u / PF_UNITS) & 1;
             if (!mbar_wait(bar(4 + s), ph ^ 1, abort, err, 21))
                 break;
-            mbar_expect_tx(bar(1 + s), Cfg::UNIT);
             uint32_t dst = smem_u32(kv_s + s * Cfg::UNIT);
             bool is_v = u == 2 * n_chunks - 1 || (u > 0 && (u & 1) == 0);
+            const int nb = is_v ? Cfg::NBV : Cfg::NBK;
+            mbar_expect_tx(bar(1 + s), (uint32_t)(nb * BLK_BYTES));
             int chunk = u == 0 ? 0 : u == 2 * n_chunks - 1 ? n_chunks - 1 : is_v ? (u - 2) / 2
                                                                             : (u + 1) / 2;
             const CUtensorMap *map = is_v ? &map_v : &map_k;
@@ -514,8 +520,9 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
                     page = 0;          // not there: every position of it is masked
                 int y = (page * nkv + kvh) * PAGE;
 #pragma unroll
-                for (int bb = 0; bb < NB; bb++)
-                    tma_load_2d(dst + bb * BLK_BYTES + pg * (PAGE * 128), map, bar(1 + s), bb * 64, y);
+                for (int bb = 0; bb < Cfg::UNIT / BLK_BYTES; bb++)
+                    if (bb < nb)
+                        tma_load_2d(dst + bb * BLK_BYTES + pg * (PAGE * 128), map, bar(1 + s), bb * 64, y);
             }
             armed |= 1u << s;
             last_parity = (last_parity & ~(1u << s)) | (ph << s);
@@ -529,7 +536,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
     } else if (warp == 1 && lane == 0) {
         // --------------------------------------------------------------- MMAs
         constexpr uint32_t idesc_s = instr_desc_bf16(AT_ROWS, AT_KEYS, false);
-        constexpr uint32_t idesc_pv = instr_desc_bf16(AT_ROWS, HD, true);
+        constexpr uint32_t idesc_pv = instr_desc_bf16(AT_ROWS, VD, true);
         int tiles = has_b ? 2 : 1;
         // The ring's units in the order of their use: K0, then for every chunk the next
         // chunk's keys before this chunk's values (K1 V0 K2 V1 ...), so that a unit is
@@ -545,7 +552,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
             uint64_t dk = smem_desc_sw128(
                 smem_u32(kv_s + (unit_k(it) % PF_UNITS) * Cfg::UNIT), 16, 1024);
 #pragma unroll
-            for (int kk = 0; kk < HD / 16; kk++) {
+            for (int kk = 0; kk < KD / 16; kk++) {
                 uint64_t off = (uint64_t)(((kk / 4) * BLK_BYTES + (kk % 4) * 32) >> 4);
                 tc_mma(tmem + t * AT_KEYS, dq + off, dk + off, idesc_s, kk != 0);
             }
@@ -591,7 +598,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
                 for (int kk = 0; kk < AT_KEYS / 16; kk++) {
                     uint64_t p_off = (uint64_t)(((kk / 4) * BLK_BYTES + (kk % 4) * 32) >> 4);
-                    tc_mma(tmem + 2 * AT_KEYS + t * HD, dp + p_off, dv + (uint64_t)(kk * 128),
+                    tc_mma(tmem + 2 * AT_KEYS + t * VD, dp + p_off, dv + (uint64_t)(kk * 128),
                            idesc_pv, (it | kk) != 0);
                 }
                 tc_commit(bar(11 + t));
@@ -616,7 +623,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
         int lo_last = window > 0 && pos_last + 1 > window ? pos_last + 1 - window : 0;
         uint32_t lane_addr = (uint32_t)(qw * 32) << 16;
         uint32_t tmem_s = tmem + t * AT_KEYS + lane_addr;
-        uint32_t tmem_o = tmem + 2 * AT_KEYS + t * HD + lane_addr;
+        uint32_t tmem_o = tmem + 2 * AT_KEYS + t * VD + lane_addr;
         // scores in units of log2(e); a head may have a factor of its own (positive:
         // the maximum below is taken before the factor is applied)
         const float c2 = scale * 1.4426950408889634f *
@@ -760,7 +767,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
             if (ok && it > 0 && __any_sync(0xffffffffu, move)) {
                 // the warp's rows of O, 32 values at a time; rows that stay keep factor 1
 #pragma unroll 1
-                for (int db = 0; db < HD / 32; db++) {
+                for (int db = 0; db < VD / 32; db++) {
                     uint32_t ov[32];
                     tc_ld32_nowait(tmem_o + db * 32, ov);
                     tc_ld_wait();
@@ -801,9 +808,9 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
                     inv = 1.0f / (l_run + exp2f(s2 - m_use));
                 }
             }
-            bf16 *dst = out + ((size_t)(q_row + jq) * nh + kvh * G + g) * HD;
+            bf16 *dst = out + ((size_t)(q_row + jq) * nh + kvh * G + g) * VD;
 #pragma unroll 1
-            for (int db = 0; db < HD / 32; db++) {
+            for (int db = 0; db < VD / 32; db++) {
                 float ov[32];
                 if (ok)
                     tc_ld32(tmem_o + db * 32, ov);
@@ -1420,11 +1427,24 @@ extern "C" int jb_attn_tc_ok(int nh, int nkv, int hd)
            nkv <= 65535;
 }
 
+// The prefill kernel's sizes: keys and values of 64 or of 128, and keys of 192 with values of 128.
+extern "C" int jb_attn_tc_prefill_ok(int nh, int nkv, int hd, int vd)
+{
+    return nkv > 0 && nh % nkv == 0 && nh / nkv <= AT_ROWS && nkv <= 65535 &&
+           ((hd == vd && (hd == 64 || hd == 128)) || (hd == 192 && vd == 128));
+}
+
 // Positions of one sequence that a CTA of the prefill kernel holds (an entry of qblk).
 extern "C" int jb_attn_tc_block_positions(int nh, int nkv)
 {
     int G = nh / nkv;
     return 2 * (AT_ROWS / G);      // a CTA of the prefill kernel holds two blocks of 128 rows
+}
+
+// The same by the keys' size: one block of rows where they have more than 128 values.
+extern "C" int jb_attn_tc_block_positions_kd(int nh, int nkv, int hd)
+{
+    return (hd > 128 ? 1 : 2) * (AT_ROWS / (nh / nkv));
 }
 
 // Prefill rows.  q, out: [n, nh, hd] bfloat16; caches [n_pages, nkv, PAGE, hd].
@@ -1466,23 +1486,27 @@ extern "C" int jb_attn_tc_prefill_ext(const void *q, const void *k_cache, const 
                                       const float *slopes, cudaStream_t st)
 {
     return jb_attn_tc_prefill_gen(q, k_cache, v_cache, n_pages, qblk, n_blocks, block_table, bt_stride,
-                                  out, n, nh, nkv, hd, window, scale, head_scale, sink, softcap, slopes,
+                                  out, n, nh, nkv, hd, hd, window, scale, head_scale, sink, softcap, slopes,
                                   0, nullptr, st);
 }
 
 // The same with two more things.  keep_first > 0 (with a window): the first keep_first
 // positions of a sequence stay visible beside the window, at their true positions.
 // score_bias (float [nh], or null): a key's weight is sigmoid(score + score_bias[head]), not
-// normalized over the keys; it goes with no sink, head factor, cap or slopes.
+// normalized over the keys; it goes with no sink, head factor, cap or slopes.  vd: the values'
+// size (jb_attn_tc_prefill_ok); out is [n, nh, vd].  Keys of 192 take no cap, slopes or sigmoids, and
+// their qblk's runs hold half as many positions (jb_attn_tc_block_positions_kd).
 extern "C" int jb_attn_tc_prefill_gen(const void *q, const void *k_cache, const void *v_cache,
                                       long long n_pages, const int32_t *qblk, int n_blocks,
                                       const int32_t *block_table, int bt_stride, void *out, int n,
-                                      int nh, int nkv, int hd, int window, float scale,
+                                      int nh, int nkv, int hd, int vd, int window, float scale,
                                       const float *head_scale, const float *sink, float softcap,
                                       const float *slopes, int keep_first, const float *score_bias,
                                       cudaStream_t st)
 {
-    if (!jb_attn_tc_ok(nh, nkv, hd) || n <= 0 || softcap < 0.0f || keep_first < 0)
+    if (!jb_attn_tc_prefill_ok(nh, nkv, hd, vd) || n <= 0 || softcap < 0.0f || keep_first < 0)
+        return JB_EINVAL;
+    if (hd == 192 && (softcap > 0.0f || slopes != nullptr || score_bias != nullptr))
         return JB_EINVAL;
     if (score_bias != nullptr && (sink != nullptr || head_scale != nullptr || softcap > 0.0f || slopes != nullptr))
         return JB_EINVAL;
@@ -1494,22 +1518,25 @@ extern "C" int jb_attn_tc_prefill_gen(const void *q, const void *k_cache, const 
     CUtensorMap mq, mk, mv;
     if (!attn_tensor_map(q, hd, nh, n, G, R, &mq) ||
         !attn_tensor_map(k_cache, hd, n_pages * nkv * PAGE, 0, PAGE, 0, &mk) ||
-        !attn_tensor_map(v_cache, hd, n_pages * nkv * PAGE, 0, PAGE, 0, &mv))
+        !attn_tensor_map(v_cache, vd, n_pages * nkv * PAGE, 0, PAGE, 0, &mv))
         return JB_EINVAL;
     if (n_blocks <= 0)
         return JB_OK;
-#define JB_PF(HDV, MODE)                                                                       \
+#define JB_PF(HDV, MODE) JB_PF_KV(HDV, HDV, MODE)
+#define JB_PF_KV(KDV, VDV, MODE)                                                                     \
     do {                                                                                       \
         static unsigned long long smem_allowed = 0;                                            \
-        auto kern = attn_tc_prefill_kernel<HDV, MODE>;                                         \
-        if (!allow_dynamic_smem(kern, PrefillCfg<HDV>::SMEM_BYTES, smem_allowed))              \
+        auto kern = attn_tc_prefill_kernel<KDV, VDV, MODE>;                                    \
+        if (!allow_dynamic_smem(kern, PrefillCfg<KDV, VDV>::SMEM_BYTES, smem_allowed))         \
             return JB_ELAUNCH;                                                                 \
         launch(kern, dim3((unsigned)n_blocks * nkv), PF_THREADS,                               \
-               PrefillCfg<HDV>::SMEM_BYTES, st, mq, mk, mv, qblk, block_table, bt_stride,      \
+               PrefillCfg<KDV, VDV>::SMEM_BYTES, st, mq, mk, mv, qblk, block_table, bt_stride, \
                (bf16 *)out, nh, nkv, G, R, window, scale, head_scale, sink, x, keep_first,     \
                score_bias);                                                                    \
     } while (0)
-    if (hd == 128 && score_bias != nullptr)
+    if (hd == 192)
+        JB_PF_KV(192, 128, 0);
+    else if (hd == 128 && score_bias != nullptr)
         JB_PF(128, 2);
     else if (hd == 128 && x.on())
         JB_PF(128, 1);
@@ -1522,6 +1549,7 @@ extern "C" int jb_attn_tc_prefill_gen(const void *q, const void *k_cache, const 
     else
         JB_PF(64, 0);
 #undef JB_PF
+#undef JB_PF_KV
     return launch_status();
 }
 

@@ -208,6 +208,8 @@ int jb_add_row_scaled(float *y, const void *skip, int skip_dt, const float *coef
 int jb_attn_tc_decode_runs(int nh, int nkv, int hd);
 int jb_attn_tc_ok(int nh, int nkv, int hd);
 int jb_attn_tc_block_positions(int nh, int nkv);
+int jb_attn_tc_block_positions_kd(int nh, int nkv, int hd);
+int jb_attn_tc_prefill_ok(int nh, int nkv, int hd, int vd);
 int jb_attn_tc_prefill(const void *q, const void *k_cache, const void *v_cache, long long n_pages,
                        const int32_t *qblk, int n_blocks, const int32_t *block_table,
                        int bt_stride, void *out, int n, int nh, int nkv, int hd, int window,
@@ -257,7 +259,7 @@ int jb_attn_tc_decode_ext(const void *q, const void *k_cache, const void *v_cach
 int jb_attn_tc_prefill_gen(const void *q, const void *k_cache, const void *v_cache,
                            long long n_pages, const int32_t *qblk, int n_blocks,
                            const int32_t *block_table, int bt_stride, void *out, int n, int nh,
-                           int nkv, int hd, int window, float scale, const float *head_scale,
+                           int nkv, int hd, int vd, int window, float scale, const float *head_scale,
                            const float *sink, float softcap, const float *slopes, int keep_first,
                            const float *score_bias, cudaStream_t st);
 int jb_attn_tc_decode_gen(const void *q, const void *k_cache, const void *v_cache,

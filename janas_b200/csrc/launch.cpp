@@ -627,7 +627,8 @@ Buf qk_norm_rope_append(Device &d, const Stack &qkv, const DevTensor *q_w, const
     return q;
 }
 
-int attention_block_positions(int nh, int nkv) { return jb_attn_tc_block_positions(nh, nkv); }
+int attention_block_positions(int nh, int nkv, int hd) { return jb_attn_tc_block_positions_kd(nh, nkv, hd); }
+bool attention_prefill_ok(int nh, int nkv, int hd, int vd) { return jb_attn_tc_prefill_ok(nh, nkv, hd, vd) != 0; }
 bool attention_tc_ok(int nh, int nkv, int hd) { return jb_attn_tc_ok(nh, nkv, hd) != 0; }
 
 Buf attention_blocks(Device &d, const long long *row0, const long long *pos0, const long long *len,
@@ -672,8 +673,11 @@ Buf attention(Device &d, const void *q, long long n, const AttnCache &c, const A
     int ni = as_int(n, "rows");
     int vd = g.value_dim();
     Buf out = d.pool.get((size_t)n * (size_t)g.nh * (size_t)vd * dtype_size(c.dt));
-    bool tc = !force_simt && vd == g.hd && c.dt == BF16 && (decode || blocks != nullptr) &&
-              !c.v_ld && !head_major && attention_tc_ok(g.nh, g.nkv, g.hd) &&
+    bool takes = decode ? vd == g.hd && attention_tc_ok(g.nh, g.nkv, g.hd)
+                        : attention_prefill_ok(g.nh, g.nkv, g.hd, vd) &&
+                              (g.hd == vd || (g.softcap == 0.0f && !g.slopes && !g.score_bias));
+    bool tc = !force_simt && takes && c.dt == BF16 && (decode || blocks != nullptr) &&
+              !c.v_ld && !head_major &&
               (decode || !g.head_scale || g.head_scale_positive);
     // kept first tokens and weights that are sigmoids: the prefill kernel has them for all its
     // sizes, of the decode kernels the one that runs over several chunks
@@ -683,7 +687,7 @@ Buf attention(Device &d, const void *q, long long n, const AttnCache &c, const A
         tc = false;
     if (tc && !decode) {
         check(jb_attn_tc_prefill_gen(q, c.k, c.v, c.n_pages, blocks, n_blocks, c.block_table, c.bt_stride,
-                                     out.ptr, ni, g.nh, g.nkv, g.hd, g.window, g.scale, g.head_scale,
+                                     out.ptr, ni, g.nh, g.nkv, g.hd, vd, g.window, g.scale, g.head_scale,
                                      g.sink, g.softcap, g.slopes, g.keep_first, g.score_bias, d.stream),
               "attention (tcgen05, prefill)");
         return out;

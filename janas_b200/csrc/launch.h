@@ -326,8 +326,10 @@ int attention_kept_chunks(int window, int keep_first);
 // uploaded to a temporary.  n_blocks comes back.
 Buf attention_blocks(Device &d, const long long *seq_row0, const long long *seq_pos0,
                      const long long *seq_len, int n_seqs, int positions_per_block, int *n_blocks);
-int attention_block_positions(int nh, int nkv);
+int attention_block_positions(int nh, int nkv, int hd = 64);
 bool attention_tc_ok(int nh, int nkv, int hd);
+// whether the tensor-core kernel for prompts takes keys of hd and values of vd
+bool attention_prefill_ok(int nh, int nkv, int hd, int vd);
 
 // Causal GQA attention of every row over its sequence's cache pages: q [n, heads,
 // hd] of the cache's dtype -> out of the same shape and dtype.  max_chunks: the

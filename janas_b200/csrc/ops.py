@@ -826,9 +826,9 @@ def _scratch(device: torch.device, floats: int) -> torch.Tensor:
     return buf
 
 
-def attention_block_positions(num_heads: int, num_kv_heads: int) -> int:
+def attention_block_positions(num_heads: int, num_kv_heads: int, head_dim: int = 64) -> int:
     """Positions of one sequence that a block of the tensor-core prefill kernel holds."""
-    return int(lib().jb_attn_tc_block_positions(num_heads, num_kv_heads))
+    return int(lib().jb_attn_tc_block_positions_kd(num_heads, num_kv_heads, head_dim))
 
 
 def attention_blocks(seq_row0, seq_pos0, seq_len, positions_per_block: int,
@@ -907,9 +907,10 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
     L = lib()
     if score_bias is not None:
         _need(score_bias, "score_bias", torch.float32, (nh,))
-    tc = (not force_simt and vd == hd and q.dtype == torch.bfloat16
+    takes = (vd == hd and L.jb_attn_tc_ok(nh, nkv, hd)) if decode else L.jb_attn_tc_prefill_ok(nh, nkv, hd, vd)
+    tc = (not force_simt and bool(takes) and q.dtype == torch.bfloat16
           and v_ld == 0 and not head_major
-          and (decode or blocks is not None) and bool(L.jb_attn_tc_ok(nh, nkv, hd))
+          and (decode or blocks is not None)
           and (decode or head_scale is None or bool((head_scale > 0).all())))
     # kept first tokens and sigmoid weights: the prefill kernel has them for all its sizes, of
     # the decode kernels the one that runs over several chunks
@@ -924,7 +925,7 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
         _check(L.jb_attn_tc_prefill_gen(_p(q), _p(k_cache), _p(v_cache),
                                         int(k_cache.shape[0]), _p(blocks),
                                         blocks.shape[0], _p(block_table), block_table.shape[1],
-                                        _p(out), n, nh, nkv, hd, window, float(scale),
+                                        _p(out), n, nh, nkv, hd, vd, window, float(scale),
                                         _p(head_scale), _p(sink), float(softcap), _p(slopes),
                                         int(keep_first), _p(score_bias), _stream()),
                "attention (tcgen05, prefill)")

@@ -615,9 +615,9 @@ private:
 // over rows gathered head by head (ops::linear_heads).
 //
 // A step of whole prompts in bfloat16 whose per-head sizes the tensor-core attention
-// kernel takes (D + R and Dv up to 64 or up to 128, padded with zeros to that where they
-// are not; padded values want a mixer without a gate) forms keys and values per head after
-// all, for that step alone, in pages of its own: [Wuk_head c | kr] and Wuv_head c are one
+// kernel takes (D + R and Dv up to 64 or up to 128, or up to 192 and 128, padded with zeros to
+// that where they are not; padded values want a mixer without a gate) forms keys and values per
+// head after all, for that step alone, in pages of its own: [Wuk_head c | kr] and Wuv_head c are one
 // product of the rows [c | kr] with a matrix made at load time (the heads' key and
 // value matrices with an identity for the shared part).  The cache gets the latents
 // as always, and decoding goes on from them.
@@ -672,10 +672,11 @@ public:
         if (g_.window < 0) config_error("latent_attention: window must not be negative");
         sink_ = s.has("sink") && s.params.get("sink").as_bool();
         n_sink_ = leaf("sink", "sink");
-        // the head size that prompts per head run with: the next one that the kernel takes
+        // the head sizes that prompts per head run with: the next ones that the kernel takes
         long long need = std::max(D_ + R_, Dv_);
-        P_ = need <= 64 ? 64 : need <= 128 ? 128 : 0;
-        if (gate_ && P_ != Dv_) P_ = 0;
+        K_ = need <= 64 ? 64 : need <= 128 ? 128 : need <= 192 && Dv_ <= 128 ? 192 : 0;
+        P_ = std::min(K_, 128ll);
+        if (gate_ && P_ != Dv_) K_ = P_ = 0;
     }
 
     void tensors(const std::string &p, TensorList &out) const override {
@@ -712,7 +713,7 @@ public:
             sinks_ = take(t, name(p, n_sink_));
             g_.sink = (const float *)sinks_.ptr;
         }
-        if (per_head_prompts_ && dtype == BF16 && P_ > 0 && ops::attention_tc_ok(H_, H_, (int)P_) &&
+        if (per_head_prompts_ && dtype == BF16 && P_ > 0 && ops::attention_prefill_ok(H_, H_, (int)K_, (int)P_) &&
             w_uv_.dt == BF16 && w_ukT_.dt == BF16 && w_o_.dt == BF16) {
             make_expander(take_back_uk());
             if (P_ != Dv_) {
@@ -734,12 +735,12 @@ public:
     }
 
     // Rows [c | kr] times this matrix are, head by head, [Wuk_head c | kr], and after
-    // all heads' keys the values Wuv c: [H P + H P, C + R], P the padded head size (the rows past
+    // all heads' keys the values Wuv c: [H K + H P, C + R], K and P the padded sizes (the rows past
     // D + R and past Dv are zeros).
     void make_expander(const DevTensor &uk) {
         size_t es = dtype_size(uk.dt);
-        long long W = C_ + R_, hd = P_;
-        w_expand_ = dev->tensor(uk.dt, {2 * H_ * hd, W}, true);
+        long long W = C_ + R_, hd = K_;
+        w_expand_ = dev->tensor(uk.dt, {H_ * (hd + P_), W}, true);
         std::vector<uint16_t> eye((size_t)(R_ * R_), 0);
         for (long long i = 0; i < R_; i++) eye[(size_t)(i * R_ + i)] = 0x3f80;      // 1.0 in bfloat16
         char *dst = (char *)w_expand_.ptr;
@@ -751,7 +752,7 @@ public:
                                         R_ * es, R_, cudaMemcpyHostToDevice), "placing the shared part's identity");
         }
         for (int h = 0; h < H_; h++)
-            cuda_check(cudaMemcpy2D(dst + (size_t)((H_ + h) * hd) * W * es, W * es,
+            cuda_check(cudaMemcpy2D(dst + (size_t)(H_ * hd + h * P_) * W * es, W * es,
                                     (const char *)w_uv_.ptr + (size_t)h * Dv_ * C_ * es, C_ * es, C_ * es, Dv_,
                                     cudaMemcpyDeviceToDevice), "placing a head's value matrix");
         dev->sync();
@@ -814,12 +815,12 @@ public:
     Stack forward_per_head(StepContext &ctx, Stack &P, LayerCache &cache, int rot_half) {
         Device &d = *ctx.dev;
         long long n = ctx.n_rows;
-        int hd = (int)P_;
+        int hd = (int)K_, vd = (int)P_;
         Buf rows;
         Buf cq = ops::latent_down(d, P, 0, Cq_, (const float *)wq_norm_.ptr, Cq_, C_,
                                   (const float *)wc_norm_.ptr, R_, position_->cos(), position_->sin(), rot_half,
                                   ctx.row_pos, ctx.row_seq, cache.kv, eps_, ctx.dtype, &rows, halves());
-        // whole queries [n, H, P], the rotated part turned
+        // whole queries [n, H, K], the rotated part turned
         Buf q = d.pool.get((size_t)n * (size_t)H_ * (size_t)hd * 2);
         {
             Stack Q = ops::linear(d, cq.ptr, ctx.dtype, n, Cq_, w_uq_);
@@ -838,8 +839,8 @@ public:
                 table[(size_t)i * (size_t)stride + (size_t)p] = (int32_t)n_pages++;
         Buf bt = d.pool.get(std::max<size_t>(table.size() * 4, 16));
         d.upload(bt.ptr, table.data(), table.size() * 4);
-        size_t page_vals = (size_t)H_ * PAGE * (size_t)hd;
-        Buf kp = d.pool.get((size_t)n_pages * page_vals * 2), vp = d.pool.get((size_t)n_pages * page_vals * 2);
+        size_t page_rows = (size_t)n_pages * (size_t)H_ * PAGE;
+        Buf kp = d.pool.get(page_rows * (size_t)hd * 2), vp = d.pool.get(page_rows * (size_t)vd * 2);
         // slots past a sequence's end are never seen but are multiplied by weights of 0
         cuda_check(cudaMemsetAsync(kp.ptr, 0, kp.bytes, d.stream), "clearing a step's key pages");
         cuda_check(cudaMemsetAsync(vp.ptr, 0, vp.bytes, d.stream), "clearing a step's value pages");
@@ -852,15 +853,16 @@ public:
         own.bt_stride = stride;
         {
             Stack kv = ops::linear(d, rows.ptr, ctx.dtype, n, C_ + R_, w_expand_);
-            ops::kv_append(d, kv, ctx.row_pos, ctx.row_seq, own, H_, hd, hd);
+            ops::kv_append(d, kv, ctx.row_pos, ctx.row_seq, own, H_, hd, vd);
         }
         ops::AttnGeometry g;
         g.nh = g.nkv = H_;
-        g.hd = g.vd = hd;
+        g.hd = hd;
+        g.vd = vd;
         g.scale = scale_;
         g.window = g_.window;
         g.sink = g_.sink;
-        int per = ops::attention_block_positions(g.nh, g.nkv);
+        int per = ops::attention_block_positions(g.nh, g.nkv, hd);
         std::string key = "attention_blocks/" + std::to_string(per);
         auto it = ctx.extras.find(key);
         if (it == ctx.extras.end()) {
@@ -890,7 +892,7 @@ private:
     // the rotation's pairs are (i, i + rotary_dim / 2)
     bool halves() const { return !position_->pairs(); }
 
-    long long hidden_, D_, R_, Dv_, C_, Cq_, P_ = 0;     // P: the head size of prompts per head (0: none)
+    long long hidden_, D_, R_, Dv_, C_, Cq_, K_ = 0, P_ = 0;     // the head sizes of prompts per head (0: none)
     bool sink_ = false;
     std::string n_sink_;
     DevTensor sinks_, w_o_pad_;

@@ -99,8 +99,15 @@ SD = config(96, 211, [lat(1, 32, 12, 16, 40, 32, 0.25, rotation(10000.0, 12, (4.
 SE = config(32, 77, [att(2, 1, 8, 0.6, None, None, dense(16, 1.0)), ret(2, 8, 8, [0.9, 0.5], None, None),
                      lat(2, 8, 4, 8, 12, 12, 0.5, None, None, moe(2, 8, 1.0, 1))])
 
-CONFIGS = {"SA": SA, "SB": SB, "SC": SC, "SD": SD, "SE": SE}
-SEEDS = {"SA": 61, "SB": 62, "SC": 63, "SD": 64, "SE": 65}
+# latent heads of more than 128 key values: at the size that the tensor cores take prompts per head with,
+# padded to it, and above it (prompts on the latents)
+SF = config(104, 150, [lat(2, 128, 64, 128, 72, 56, 0.08, rotation(10000.0, 64, (16.0, 32.0, 512, 1.0)), 150, dense(64, 1.0)),
+                       lat(3, 100, 40, 72, 88, 40, 0.1, rotation(5000.0, 40), None, moe(3, 16, 1.1, 2, (24, 0.8))),
+                       lat(1, 180, 60, 96, 64, 48, 0.07, rotation(5000.0, 60), 70, dense(48, 0.7))],
+            loop=(0, 1, 2))
+
+CONFIGS = {"SA": SA, "SB": SB, "SC": SC, "SD": SD, "SE": SE, "SF": SF}
+SEEDS = {"SA": 61, "SB": 62, "SC": 63, "SD": 64, "SE": 65, "SF": 66}
 
 
 def tensor_shapes(c):

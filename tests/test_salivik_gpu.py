@@ -397,6 +397,55 @@ def test_a_sink_takes_its_share(dtype, mode, nh, nkv, hd, rot, decode):
 
 
 # ------------------------------------------------------------ latent attention
+@pytest.mark.parametrize("nh,nkv,window", [(2, 2, 0), (3, 1, 130), (4, 4, 64), (1, 1, 1), (8, 2, 200)])
+def test_keys_of_192_and_values_of_128_on_the_tensor_cores(nh, nkv, window):
+    """Prompt rows of unequal sequences, whole and from a later position on, with a sink; then one key made
+    to stand out just inside and just outside the window, and far back without one."""
+    hd, vd, scale = 192, 128, 0.05
+    assert ops().lib().jb_attn_tc_prefill_ok(nh, nkv, hd, vd)
+    sink = torch.linspace(-1.0, 2.0, nh)
+    per = ops().attention_block_positions(nh, nkv, hd)
+    assert per == 128 // (nh // nkv)
+
+    def run(lens, rows, qs, ks, vs):
+        P = Paged(lens, 11)
+        want = torch.cat([ps.window_attention(qs[i], ks[i][:p0 + cnt], vs[i][:p0 + cnt], scale, window or None, sink, p0)
+                          for i, (p0, cnt) in enumerate(rows)])
+        row_pos, row_seq = row_arrays(rows)
+        r0, at = [], 0
+        for (_, cnt) in rows:
+            r0.append(at)
+            at += cnt
+        blocks = ops().attention_blocks(r0, [p for p, _ in rows], [c for _, c in rows], per, torch.device(DEV))
+        chunk = ops().attention_chunk()
+        got = ops().attention(torch.cat(qs).to(torch.bfloat16).to(DEV), P.fill(ks, torch.bfloat16), P.fill(vs, torch.bfloat16),
+                              row_pos.to(DEV), row_seq.to(DEV), P.table.to(DEV), window, scale,
+                              int(row_pos.max()) // chunk + 1, blocks=blocks, sink=sink.to(DEV)).float().cpu()
+        assert ops().attn_tc_error() == 0
+        return got, want
+
+    lens, rows = [1, 300, 131, 520], [(0, 1), (0, 300), (100, 31), (0, 520)]
+    qs = [bf(rnd(cnt, nh, hd, seed=i)) for i, (_, cnt) in enumerate(rows)]
+    ks = [bf(rnd(n, nkv, hd, seed=10 + i)) for i, n in enumerate(lens)]
+    vs = [bf(rnd(n, nkv, vd, seed=20 + i)) for i, n in enumerate(lens)]
+    got, want = run(lens, rows, qs, ks, vs)
+    close(got, want, 2e-2)
+    for qp in (max(window - 1, 0), window + 3, 383, 599):
+        for kp, inside in ((max(0, qp + 1 - window) if window else 3, True), (qp - window, False)):
+            if kp < 0 or kp > qp or (not window and not inside):
+                continue
+            rows = [(max(0, qp - 30), min(31, qp + 1))]
+            q, k, v = bf(rnd(rows[0][1], nh, hd, seed=kp)), bf(rnd(600, nkv, hd, scale=0.3, seed=kp + 1)), bf(rnd(600, nkv, vd, seed=kp + 2))
+            q[-1] = 0.0
+            q[-1, :, 150] = 20.0                    # a place that only the keys' third part has
+            k[:, :, 150] = 0.0
+            k[kp, :, 150] = 24.0
+            v[kp] = 5.0
+            got, want = run([600], rows, [q], [k], [v])
+            close(got, want, 2e-2, f"query {qp} key {kp}")
+            assert (float(got[-1].mean()) > 4.5) == inside
+
+
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("H,D,R,dims,Dv,C,Cq,window,halves", [(4, 16, 8, 8, 24, 40, 24, 37, True), (3, 10, 6, 6, 6, 22, 14, 0, True),
                                                               (2, 64, 64, 64, 128, 96, 48, 130, True), (1, 24, 16, 12, 40, 64, 32, 64, True),
@@ -503,7 +552,7 @@ def test_a_latent_just_inside_and_outside_a_window(dtype, C, R, H, window):
 
 # ------------------------------------------------------------------ whole models
 LENGTHS = {"SA": [1, 2, 9, 70, 131, 260], "SB": [1, 3, 64, 65, 200, 410], "SC": [2, 17, 128, 129, 300, 520],
-           "SD": [1, 5, 33, 64, 190, 330], "SE": [1, 2, 4, 30, 66, 140]}
+           "SD": [1, 5, 33, 64, 190, 330], "SE": [1, 2, 4, 30, 66, 140], "SF": [1, 3, 40, 129, 257, 420]}
 FP32_TOL = 5e-5
 BF16_TOL = 5e-2
 CLOSE_CALL = 5e-2
@@ -714,12 +763,12 @@ def test_every_pass_has_places_of_its_own():
     assert groups == {(m[0]["kv_rank"] + m[0]["rot_dim"], 37, True): 1, (m[1]["dim"], 64, False): 3}
 
 
-def test_prompts_per_head_against_prompts_on_the_latents():
+@pytest.mark.parametrize("name", ["SC", "SF"])
+def test_prompts_per_head_against_prompts_on_the_latents(name):
     """In bfloat16 whole prompts may form keys and values per head (at their own size, or padded to the
     kernel's); on the latents, as every other step, the same prompts give the same logits."""
     from janas_b200.config import config_from_dict
     from janas_b200.engine import Engine
-    name = "SC"
     _, c, w = model(name)
     e = engine(name, "bfloat16")
     d = config_from_dict(c).to_model_spec().to_json()
@@ -728,7 +777,7 @@ def test_prompts_per_head_against_prompts_on_the_latents():
         if l["mixer"]["kind"] == "latent_attention":
             l["mixer"]["params"]["per_head_prompts"] = False
             n += 1
-    assert n == 2
+    assert n == {"SC": 2, "SF": 3}[name]
     from janas_b200.config import ModelSpec
     other = Engine.from_spec(ModelSpec.from_json(d), {k: v.to(torch.bfloat16).to(DEV) for k, v in w.items()}, dtype="bfloat16",
                              max_tokens=2048)

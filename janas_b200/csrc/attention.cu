@@ -473,9 +473,11 @@ __global__ void __launch_bounds__(LD_THREADS)
 latent_decode_mma_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ k_cache,
                          const int32_t *__restrict__ row_pos, const int32_t *__restrict__ row_seq,
                          const int32_t *__restrict__ block_table, int bt_stride,
-                         float *__restrict__ part, int row0, int nh, int hd, int vd, int window,
-                         float scale, int max_chunks)
+                         float *__restrict__ part, int row0, int all_heads, int heads_per, int hd, int vd,
+                         int window, float scale, int max_chunks)
 {
+    // this CTA's heads: heads_per (a multiple of 16, or all of them) from h_base on
+    const int h_base = blockIdx.y * heads_per, nh = min(heads_per, all_heads - h_base);
     extern __shared__ __align__(16) uint8_t ld_smem[];
     const int ks = hd + 8;                                   // row strides, in values: 16 bytes of padding
     const int nh16 = (nh + 15) / 16 * 16;
@@ -518,7 +520,7 @@ latent_decode_mma_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ k_
         int h = i / pieces, pc = i - h * pieces;
         bf16 *dst = Qs + (size_t)h * ks + pc * 8;
         if (h < nh)
-            copy16(dst, q + ((size_t)row * nh + h) * hd + pc * 8);
+            copy16(dst, q + ((size_t)row * all_heads + h_base + h) * hd + pc * 8);
         else
             *reinterpret_cast<uint4 *>(dst) = zero4;
     }
@@ -532,14 +534,31 @@ latent_decode_mma_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ k_
         int a_row = lane & 15, a_k = (lane >> 4) * 8;
         int b_row = (lane & 7) + (lane >> 4) * 8, b_k = ((lane >> 3) & 1) * 8;
         for (int h0 = 0; h0 < nh16; h0 += 16) {
+            // the steps along k in two chains, even and odd, joined at the end
             float acc[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
-            for (int k0 = 0; k0 < hd; k0 += 16) {
-                uint32_t a[4], b[4];
-                ldmatrix_x4(a, Qs + (size_t)(h0 + a_row) * ks + k0 + a_k);
-                ldmatrix_x4(b, Ks + (size_t)(j0 + b_row) * ks + k0 + b_k);
+            float odd[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+            const bf16 *qp = Qs + (size_t)(h0 + a_row) * ks + a_k, *kp = Ks + (size_t)(j0 + b_row) * ks + b_k;
+            for (int k0 = 0; k0 < hd; k0 += 32) {
+                uint32_t a[4], b[4], a2[4], b2[4];
+                const bool more = k0 + 16 < hd;
+                ldmatrix_x4(a, qp + k0);
+                ldmatrix_x4(b, kp + k0);
+                if (more) {
+                    ldmatrix_x4(a2, qp + k0 + 16);
+                    ldmatrix_x4(b2, kp + k0 + 16);
+                }
                 mma_bf16(acc[0], a, b[0], b[1]);
                 mma_bf16(acc[1], a, b[2], b[3]);
+                if (more) {
+                    mma_bf16(odd[0], a2, b2[0], b2[1]);
+                    mma_bf16(odd[1], a2, b2[2], b2[3]);
+                }
             }
+#pragma unroll
+            for (int t = 0; t < 2; t++)
+#pragma unroll
+                for (int e = 0; e < 4; e++)
+                    acc[t][e] += odd[t][e];
 #pragma unroll
             for (int t = 0; t < 2; t++)
 #pragma unroll
@@ -580,36 +599,55 @@ latent_decode_mma_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ k_
         }
         l = warp_sum(l);
         if (lane == 0) {
-            float *dst = part + part_at((size_t)lrow, nh, h, max_chunks, ci, vd);
+            float *dst = part + part_at((size_t)lrow, all_heads, h_base + h, max_chunks, ci, vd);
             dst[0] = m;
             dst[1] = l;
         }
     }
     __syncthreads();
-    // ---- values: 16 columns at a time per warp, 16 heads at a time
+    // ---- values: up to four blocks of 16 columns per warp at once, 16 heads at a time
     {
+        constexpr int CB = 4, STEP = (LD_THREADS / 32) * 16;
         int a_row = lane & 15, a_k = (lane >> 4) * 8;
         int b_row = (lane & 7) + ((lane >> 3) & 1) * 8, b_c = (lane >> 4) * 8;
-        for (int c0 = warp * 16; c0 < vd; c0 += (LD_THREADS / 32) * 16) {
-            for (int h0 = 0; h0 < nh16; h0 += 16) {
-                float acc[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+        for (int h0 = 0; h0 < nh16; h0 += 16) {
+            for (int c0 = warp * 16; c0 < vd; c0 += CB * STEP) {
+                float acc[CB][2][4];
+#pragma unroll
+                for (int u = 0; u < CB; u++)
+#pragma unroll
+                    for (int t = 0; t < 2; t++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++)
+                            acc[u][t][e] = 0.0f;
 #pragma unroll
                 for (int j0 = 0; j0 < ATT_CHUNK; j0 += 16) {
-                    uint32_t a[4], b[4];
+                    uint32_t a[4];
                     ldmatrix_x4(a, Ps + (size_t)(h0 + a_row) * ps + j0 + a_k);
-                    ldmatrix_x4_trans(b, Ks + (size_t)(j0 + b_row) * ks + c0 + b_c);
-                    mma_bf16(acc[0], a, b[0], b[1]);
-                    mma_bf16(acc[1], a, b[2], b[3]);
+#pragma unroll
+                    for (int u = 0; u < CB; u++) {
+                        if (c0 + u * STEP < vd) {
+                            uint32_t b[4];
+                            ldmatrix_x4_trans(b, Ks + (size_t)(j0 + b_row) * ks + c0 + u * STEP + b_c);
+                            mma_bf16(acc[u][0], a, b[0], b[1]);
+                            mma_bf16(acc[u][1], a, b[2], b[3]);
+                        }
+                    }
                 }
 #pragma unroll
-                for (int t = 0; t < 2; t++)
+                for (int u = 0; u < CB; u++) {
+                    if (c0 + u * STEP >= vd)
+                        continue;
 #pragma unroll
-                    for (int e = 0; e < 4; e++) {
-                        int h = h0 + (lane >> 2) + (e >> 1) * 8;
-                        int cc = c0 + t * 8 + (lane & 3) * 2 + (e & 1);
-                        if (h < nh)
-                            part[part_at((size_t)lrow, nh, h, max_chunks, ci, vd) + 2 + cc] = acc[t][e];
-                    }
+                    for (int t = 0; t < 2; t++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            int h = h0 + (lane >> 2) + (e >> 1) * 8;
+                            int cc = c0 + u * STEP + t * 8 + (lane & 3) * 2 + (e & 1);
+                            if (h < nh)
+                                part[part_at((size_t)lrow, all_heads, h_base + h, max_chunks, ci, vd) + 2 + cc] = acc[u][t][e];
+                        }
+                }
             }
         }
     }
@@ -872,10 +910,18 @@ extern "C" int jb_attention_gen(const void *q, const void *k_cache, const void *
         if (!allow_dynamic_smem(latent_decode_kernel, LD_SMEM_MAX, smem_allowed) ||
             !allow_dynamic_smem(latent_decode_mma_kernel, LD_SMEM_MAX, mma_allowed))
             return JB_ELAUNCH;
-        if (mma_bytes > 0)
-            launch(latent_decode_mma_kernel, dim3((unsigned)n_rows * max_chunks), LD_THREADS, mma_bytes, st,
-                   (const bf16 *)q, (const bf16 *)k_cache, row_pos, row_seq, block_table, bt_stride, scratch,
-                   row0, nh, hd, vd, window, scale, max_chunks);
+        if (mma_bytes > 0) {
+            // few rows: the heads shared out over more CTAs, 16 to each (every one of them brings the
+            // chunk's rows for itself), as long as all of them run at once
+            int per = nh;
+            if (nh > 16 && (long long)n_rows * max_chunks * ((nh + 15) / 16) <= sm_count()) {
+                per = 16;
+                mma_bytes = latent_decode_mma_smem(16, hd, vd);
+            }
+            launch(latent_decode_mma_kernel, dim3((unsigned)n_rows * max_chunks, (unsigned)((nh + per - 1) / per)),
+                   LD_THREADS, mma_bytes, st, (const bf16 *)q, (const bf16 *)k_cache, row_pos, row_seq, block_table,
+                   bt_stride, scratch, row0, nh, per, hd, vd, window, scale, max_chunks);
+        }
         else
             launch(latent_decode_kernel, dim3((unsigned)n_rows * max_chunks), LD_THREADS, ld_bytes, st,
                    (const bf16 *)q, (const bf16 *)k_cache, row_pos, row_seq, block_table, bt_stride, scratch,

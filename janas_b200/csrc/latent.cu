@@ -141,14 +141,14 @@ __global__ void latent_q_split_kernel(const float *__restrict__ Q, int S, size_t
 __device__ __forceinline__ float4 sum4(const float *__restrict__ p, int S, size_t stride)
 {
     float4 v = load4(p);
-    for (int s0 = 1; s0 < S; s0 += 4) {
-        // four terms fetched together, added in order
-        float4 w[4];
+    for (int s0 = 1; s0 < S; s0 += 8) {
+        // eight terms fetched together, added in order
+        float4 w[8];
 #pragma unroll
-        for (int u = 0; u < 4; u++)
+        for (int u = 0; u < 8; u++)
             w[u] = s0 + u < S ? load4(p + (size_t)(s0 + u) * stride) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
-        for (int u = 0; u < 4; u++)
+        for (int u = 0; u < 8; u++)
             if (s0 + u < S)
                 v = make_float4(v.x + w[u].x, v.y + w[u].y, v.z + w[u].z, v.w + w[u].w);
     }
@@ -156,11 +156,11 @@ __device__ __forceinline__ float4 sum4(const float *__restrict__ p, int S, size_
 }
 
 // latent_down with four neighbouring values of the row to a thread at a time, up to U times, all
-// held in registers: both sums of squares cross the block together, and the shared key part
+// held in registers (NT threads a row): both sums of squares cross the block together, and the shared key part
 // passes through shared memory for the rotation.  q_rank, kv_rank, rot_dim and the columns are
 // multiples of four.
-template <typename TC, int U>
-__global__ void __launch_bounds__(128)
+template <typename TC, int U, int NT>
+__global__ void __launch_bounds__(NT)
 latent_down_vec_kernel(const float *__restrict__ P, int S, size_t stride, int ld, int q_col0, int q_rank,
                        const float *__restrict__ wq, int kv_col0, int kv_rank,
                        const float *__restrict__ wkv, int rot_dim, const float *__restrict__ cs,
@@ -170,7 +170,7 @@ latent_down_vec_kernel(const float *__restrict__ P, int S, size_t stride, int ld
                        TC *__restrict__ rows_out, float eps, int halves)
 {
     extern __shared__ __align__(16) float zr[];      // rot_dim sums of this row
-    __shared__ float red[2][4];
+    __shared__ float red[2][NT / 32];
     pdl_trigger();
     size_t row = blockIdx.x;
     int pos = row_pos[row];
@@ -183,7 +183,7 @@ latent_down_vec_kernel(const float *__restrict__ P, int S, size_t stride, int ld
     float sq = 0.0f, sc = 0.0f;
 #pragma unroll
     for (int u = 0; u < U; u++) {
-        int i = 4 * (threadIdx.x + 128 * u);
+        int i = 4 * (threadIdx.x + NT * u);
         if (i >= all)
             continue;
         v[u] = sum4(i < q_rank ? pq + i : pc + i, S, stride);
@@ -202,15 +202,19 @@ latent_down_vec_kernel(const float *__restrict__ P, int S, size_t stride, int ld
         red[1][warp] = sc;
     }
     __syncthreads();
-    sq = red[0][0] + red[0][1] + red[0][2] + red[0][3];
-    sc = red[1][0] + red[1][1] + red[1][2] + red[1][3];
+    sq = sc = 0.0f;
+#pragma unroll
+    for (int w = 0; w < NT / 32; w++) {
+        sq += red[0][w];
+        sc += red[1][w];
+    }
     float iq = 1.0f / sqrtf(sq / (float)max(q_rank, 1) + eps), ic = 1.0f / sqrtf(sc / (float)kv_rank + eps);
     int hd = kv_rank + rot_dim;
     TC *dst = k_cache + ((size_t)page * PAGE + pos % PAGE) * hd;
     TC *dst2 = rows_out != nullptr ? rows_out + row * hd : nullptr;
 #pragma unroll
     for (int u = 0; u < U; u++) {
-        int i = 4 * (threadIdx.x + 128 * u);
+        int i = 4 * (threadIdx.x + NT * u);
         if (i >= all)
             continue;
         if (i < both) {
@@ -501,18 +505,21 @@ extern "C" int jb_latent_down_rows(const float *P, int S, long long stride, int 
     if (q_rank % 4 == 0 && kv_rank % 4 == 0 && rot_dim % 4 == 0 && q_col0 % 4 == 0 && kv_col0 % 4 == 0 && ld % 4 == 0 &&
         stride % 4 == 0 && at(P, 16) && at(wq, 16) && at(wkv, 16) && at(cq_out, 4 * esz) && at(k_cache, 4 * esz) &&
         at(rows_out, 4 * esz) && U <= 8 && (cache_dt == JB_F32 || cache_dt == JB_BF16)) {
-#define JB_LDV(TC, UU)                                                                                       \
-    launch(latent_down_vec_kernel<TC, UU>, n, 128, (size_t)rot_dim * 4, st, P, S, (size_t)stride, ld, q_col0,  \
+        // few rows in bfloat16: more threads to a row (the 32-bit path adds in one order whatever the batch)
+#define JB_LDV(TC, UU, NT)                                                                                   \
+    launch(latent_down_vec_kernel<TC, UU, NT>, n, NT, (size_t)rot_dim * 4, st, P, S, (size_t)stride, ld, q_col0,  \
            q_rank, wq, kv_col0, kv_rank, wkv, rot_dim, cs, sn, rot_half, row_pos, row_seq, block_table,      \
            bt_stride, (TC *)cq_out, (TC *)k_cache, (TC *)rows_out, eps, halves)
 #define JB_LDV_U(TC)                          \
     do {                                      \
-        if (U <= 2) JB_LDV(TC, 2);            \
-        else if (U <= 4) JB_LDV(TC, 4);       \
-        else JB_LDV(TC, 8);                   \
+        if (U <= 2) JB_LDV(TC, 2, 128);       \
+        else if (U <= 4) JB_LDV(TC, 4, 128);  \
+        else JB_LDV(TC, 8, 128);              \
     } while (0)
         if (cache_dt == JB_F32)
             JB_LDV_U(float);
+        else if (n <= 64 && U <= 4)
+            JB_LDV(bf16, 1, 512);
         else
             JB_LDV_U(bf16);
 #undef JB_LDV_U

@@ -521,8 +521,9 @@ def test_latent_attention_steps(dtype, H, D, R, dims, Dv, C, Cq, window, halves)
 
 
 @pytest.mark.parametrize("dtype,C,R,H", [(torch.float32, 40, 8, 3), (torch.bfloat16, 40, 8, 3), (torch.bfloat16, 96, 32, 5),
-                                         (torch.bfloat16, 22, 6, 2)])
-@pytest.mark.parametrize("window", [1, 64, 72, 200])
+                                         (torch.bfloat16, 22, 6, 2), (torch.bfloat16, 64, 16, 20),
+                                         (torch.bfloat16, 128, 64, 40)])
+@pytest.mark.parametrize("window", [1, 64, 75, 200])
 def test_a_latent_just_inside_and_outside_a_window(dtype, C, R, H, window):
     """A cached row at a window's edge dominates a query's scores: inside, the weighted sum is that row's
     latent part; outside, it does not show."""

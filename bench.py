@@ -273,14 +273,18 @@ def decode_timeline(eng, slots, tokens, warmup):
 
 
 def step_bytes(eng, batch, context):
-    """Bytes a decode step has to move: every weight once, the keys and values of
-    the live sequences, and their recurrent state there and back."""
+    """Bytes a decode step has to move: every weight once, the keys and values that the
+    live sequences' rows see, and their recurrent state there and back."""
     info = eng.info()
     esz = 2 if info["dtype"] == "bfloat16" else 4
     kv = 0
     for g in info["cache"]["groups"]:
-        per_token = 2 * len(g["entries"]) * g["num_kv_heads"] * g["head_dim"] * esz
-        kv += per_token * batch * context
+        # (a group whose values lie in its keys' rows has one row per position; a window's
+        # earlier positions are not read)
+        rows = 1 if g.get("values_in_keys") else 2
+        per_token = rows * len(g["entries"]) * g["num_kv_heads"] * g["head_dim"] * esz
+        seen = min(context, g["window"] + g.get("keep_first", 0)) if g.get("window") else context
+        kv += per_token * batch * seen
     # the mixers' fixed-size state of every live sequence, read and written once a step
     for b in info["cache"].get("state_bytes", []):
         kv += 2 * b * batch

@@ -156,6 +156,7 @@ class ModelSpec:
     embedding_norm_name: str = "model.embed_norm"
     token_table_name: str = ""         # a second table of vectors per token that the layers' blocks read; "": none
     token_table_width: int = 0
+    streams: int = 0                   # > 0: the residual stream is this many streams per row
     join_name: str = ""                # the matrix of the entries with join_embedding; "": none
 
     def to_json(self) -> Dict[str, Any]:
@@ -179,6 +180,8 @@ class ModelSpec:
         if self.token_table_name:
             d["token_table_name"] = self.token_table_name
             d["token_table_width"] = self.token_table_width
+        if self.streams:
+            d["streams"] = self.streams
         if self.join_name:
             d["join_name"] = self.join_name
         if self.embedding_norm:
@@ -195,7 +198,7 @@ class ModelSpec:
             embedding_scale=d.get("embedding_scale", 1.0),
             token_table_name=d.get("token_table_name", ""),
             token_table_width=d.get("token_table_width", 0),
-            join_name=d.get("join_name", ""),
+            streams=d.get("streams", 0), join_name=d.get("join_name", ""),
             embedding_norm=PartSpec.from_json(d["embedding_norm"]) if d.get("embedding_norm") else None,
             embedding_norm_name=d.get("embedding_norm_name", "model.embed_norm"),
             architecture=d["architecture"], hidden_size=d["hidden_size"],
@@ -383,8 +386,42 @@ class SalivikConfig:
         return hash(json.dumps(self.to_dict(), sort_keys=True))
 
 
+@dataclass(frozen=True)
+class DafalixConfig:
+    """The Dafalix decoder's ``config.json`` keys, as the library read them."""
+    vocab: int
+    width: int
+    norm_eps: float
+    streams: int
+    residual_mult: float
+    loop: Optional[Mapping[str, int]]         # start, stop, times; None: every layer runs once
+    layers: Tuple[Mapping[str, Any], ...]     # each: type, mixer {...}, mlp {...} or None
+    eos_token_ids: Tuple[int, ...] = ()
+    architecture: str = "Dafalix"
+    _json: Mapping[str, Any] = field(default_factory=dict, compare=False, repr=False)
+    _spec: Mapping[str, Any] = field(default_factory=dict, compare=False, repr=False)
+
+    @classmethod
+    def from_dict(cls, d: Mapping[str, Any]) -> "DafalixConfig":
+        return _wrap(_call("config.parse", config=dict(d)))
+
+    def to_dict(self) -> Dict[str, Any]:
+        return dict(self._json)
+
+    def to_model_spec(self) -> ModelSpec:
+        return ModelSpec.from_json(self._spec)
+
+    def __hash__(self) -> int:
+        return hash(json.dumps(self.to_dict(), sort_keys=True))
+
+
 def _wrap(r: Mapping[str, Any]):
     c = r["config"]
+    if r["architecture"] == "Dafalix":
+        return DafalixConfig(
+            vocab=c["vocab"], width=c["width"], norm_eps=c["norm"]["eps"], streams=c["streams"],
+            residual_mult=c["residual_mult"], loop=dict(c["loop"]) if c["loop"] else None,
+            layers=tuple(c["layers"]), eos_token_ids=tuple(r["eos_token_ids"]), _json=c, _spec=r["spec"])
     if r["architecture"] == "Salivik":
         return SalivikConfig(
             vocab=c["vocab"], width=c["width"], norm_eps=c["norm"]["eps"],
@@ -441,4 +478,4 @@ def config_from_dir(model_dir: str):
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "Qwen3Config",
            "ZuzelornConfig", "DunavikConfig", "KefesunConfig", "MunisunConfig",
-           "SalivikConfig", "config_from_dict", "config_from_dir", "known_architectures"]
+           "SalivikConfig", "DafalixConfig", "config_from_dict", "config_from_dir", "known_architectures"]

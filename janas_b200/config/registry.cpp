@@ -39,6 +39,7 @@ static Tables &ready() {
         register_kefesun();
         register_munisun();
         register_salivik();
+        register_dafalix();
     });
     return raw_tables();
 }

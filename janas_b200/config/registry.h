@@ -37,12 +37,13 @@ std::string architecture_name(const Json &config_json);
 std::unique_ptr<ArchConfig> config_from_json(const Json &config_json);
 std::unique_ptr<ArchConfig> config_from_dir(const std::string &model_dir);
 
-// defined in qwen3.cpp, zuzelorn.cpp, dunavik.cpp, kefesun.cpp, munisun.cpp and salivik.cpp; called once by the registry
+// defined in qwen3.cpp, zuzelorn.cpp, dunavik.cpp, kefesun.cpp, munisun.cpp, salivik.cpp and dafalix.cpp; called once by the registry
 void register_qwen3();
 void register_zuzelorn();
 void register_dunavik();
 void register_kefesun();
 void register_munisun();
 void register_salivik();
+void register_dafalix();
 
 }  // namespace jb

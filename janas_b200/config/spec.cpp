@@ -51,6 +51,7 @@ void ModelSpec::validate() const {
         if (layers[i].feed_forward.kind.empty() && !layers[i].ffn_norm.kind.empty())
             config_error(fmt("layer %zu: a norm for a feed-forward that the layer does not have", i));
     if (run_order.empty()) config_error("the run order is empty");
+    if (streams < 0) config_error("streams must not be negative");
     for (size_t at = 0; at < run_order.size(); at++) {
         const RunEntry &e = run_order[at];
         if (e.layer < 0 || e.layer >= (int)layers.size())
@@ -60,6 +61,8 @@ void ModelSpec::validate() const {
             config_error(fmt("run order entry %zu joins the embedding output and the model names no join matrix", at));
         if (e.join_embedding && e.add_embedding)
             config_error(fmt("run order entry %zu both adds and joins the embedding output", at));
+        if (streams > 0 && (e.join_embedding || e.add_embedding))
+            config_error(fmt("run order entry %zu: a residual stream of several streams takes the embedding output once", at));
         if (e.cache_of >= 0) {
             if (e.cache_of >= (int)at)
                 config_error(fmt("run order entry %zu reads the cache of entry %d, which has not run "
@@ -122,6 +125,7 @@ Json ModelSpec::to_json() const {
         j.set("token_table_width", token_table_width);
     }
     if (!join_name.empty()) j.set("join_name", join_name);
+    if (streams > 0) j.set("streams", streams);
     j.set("embedding_name", embedding_name);
     j.set("final_norm_name", final_norm_name);
     j.set("head_name", head_name);
@@ -182,6 +186,7 @@ ModelSpec ModelSpec::from_json(const Json &j) {
     s.token_table_name = str_or(j, "token_table_name", "");
     if (j.get("token_table_width").is_number()) s.token_table_width = j.get("token_table_width").as_int();
     s.join_name = str_or(j, "join_name", "");
+    if (j.get("streams").is_number()) s.streams = j.get("streams").as_int();
     s.embedding_name = str_or(j, "embedding_name", s.embedding_name);
     s.final_norm_name = str_or(j, "final_norm_name", s.final_norm_name);
     s.head_name = str_or(j, "head_name", s.head_name);

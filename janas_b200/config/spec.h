@@ -109,6 +109,9 @@ struct ModelSpec {
     // the layers' blocks read by columns (a per-layer input of the token itself)
     std::string token_table_name;
     long long token_table_width = 0;
+    // > 0: the residual stream is this many streams per row, all the embedding output at the start and
+    // summed at the end; every layer's arrangement must then be one that reads and writes streams
+    long long streams = 0;
     // the matrix of the run-order entries with join_embedding ("": the model has none)
     std::string join_name;
     std::string embedding_name = "model.embed_tokens.weight";

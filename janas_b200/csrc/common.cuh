@@ -129,6 +129,9 @@ __device__ __forceinline__ float gated_unit(float g, float u, const GatedUnit &p
 // writes are visible.  What a kernel does before pdl_wait() must not touch
 // anything an earlier kernel writes or reads-and-frees: only its own shared and
 // tensor memory and the (immutable) weights.
+// A kernel argument that an earlier kernel writes and that is read right after pdl_wait() should not be
+// const __restrict__: the compiler takes such memory for read-only and may move the load ahead of the
+// wait.
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_trigger()
 {

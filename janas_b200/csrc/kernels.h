@@ -172,15 +172,23 @@ int jb_moe_route(const float *P, int S, long long stride, int ld, int col0, cons
                  int keep, int top, int first_identity, float scale, int score, int group_best,
                  cudaStream_t st);
 int jb_gated_weighted(const float *z, int S, long long stride, int ld, const float *weights, int w_ld,
-                      int n_experts, int ff, int shared_ff, int kind, const float *unit, void *out,
-                      int out_dt, int n, cudaStream_t st);
+                      int n_experts, int ff, int shared_ff, int kind, const float *unit, int on_input,
+                      void *out, int out_dt, int n, cudaStream_t st);
 int jb_turn_heads(const float *src, int S, long long stride, int ld, int col0, int H, int D, int Dv,
                   const float *cs, const float *sn, int rot_half, const int32_t *row_pos, float key_scale,
                   float *out, int n, cudaStream_t st);
 int jb_causal_conv(const float *u, int S, long long stride, int ld, int col0, const float *w,
                    const float *bias, float *state, long long slot_stride, const int32_t *row_pos,
                    const int32_t *row_seq, const int32_t *seq_slot, void *out, int out_dt, int out_ld,
-                   int n, int C, int taps, int act, int what, cudaStream_t st);
+                   int n, int C, int taps, int act, int what, const float *in_bias, void *parts,
+                   int parts_dt, int part, cudaStream_t st);
+int jb_lru_piece(void);
+long long jb_lru_scratch(int n, int n_seqs, int max_len, int W);
+int jb_lru(const float *G, int gS, int part, const float *rb, const float *ib, const float *lam,
+           const float *u, const float *P, int S, long long stride, int ld, int y_col0, const float *yb,
+           float *state, long long slot_stride, const int32_t *row_seq, const int32_t *seq_slot,
+           float *scratch, void *out, int out_dt, int n, int n_seqs, int W, int every_row_starts,
+           int max_len, cudaStream_t st);
 int jb_matrix_state_scan(const float *src, int S, long long stride, int ld, int val_col0, int key_col0,
                          int qry_col0, int silu, const float *dt, int dt_S, long long dt_stride,
                          int dt_ld, int dt_col0, const float *dt_bias, const float *a_log,
@@ -190,6 +198,26 @@ int jb_matrix_state_scan(const float *src, int S, long long stride, int ld, int 
                          cudaStream_t st);
 int jb_matrix_state_piece(void);
 long long jb_matrix_state_scratch(int n_seqs, int max_len, int H, int N, int P);
+long long jb_gated_memory_scratch(int n, int n_seqs, int max_len, int H, int N, int P,
+                                  int every_row_starts);
+int jb_gated_memory_scan(const float *src, int S, long long stride, int ld, int val_col0, int key_col0,
+                         int qry_col0, int i_col0, int f_col0, const float *i_bias, const float *f_bias,
+                         float cap, float q_scale, float *state, long long slot_stride,
+                         const int32_t *row_seq, const int32_t *seq_slot, float *y, float *nq, float *em,
+                         int n, int n_seqs, int H, int N, int P, int every_row_starts, float *scratch,
+                         int max_len, cudaStream_t st);
+int jb_gated_memory_norm(const float *y, const float *nq, const float *em, float floor, const float *src,
+                         int S, long long stride, int ld, int g_col0, int i_col0, int f_col0,
+                         const float *i_bias, const float *f_bias, float cap, float *state,
+                         long long slot_stride, const int32_t *row_seq, const int32_t *seq_slot,
+                         const float *w, float eps, void *out, int out_dt, int n, int H, int N, int P,
+                         cudaStream_t st);
+int jb_max_streams(void);
+int jb_spread_streams(const float *e, float *x, int ns, int n, int dm, cudaStream_t st);
+int jb_streams(float *x, int ns, const float *y, int S, long long stride, const float *ls,
+               const float *out_w, const float *mix, float mult, const int32_t *rows, const float *in_w,
+               const float *w, const float *b, float eps, void *out, int out_dt, int n, int dm,
+               int few_rows, cudaStream_t st);
 int jb_gated_part_norm(const float *y, const float *pre, int pre_S, long long pre_stride, int pre_ld,
                        int pre_col0, const float *post, int post_S, long long post_stride, int post_ld,
                        int post_col0, int post_silu, const float *w, float eps, void *out, int out_dt,

@@ -216,7 +216,8 @@ Buf moe_route(Device &d, const Stack &P, long long col0, const RouteParams &r, B
 }
 
 Buf gated_weighted(Device &d, const Stack &z, const float *weights, int w_ld, int n_experts, long long ff,
-                   int kind, DType out_dt, long long shared_ff, UnitParams unit, UnitParams shared_unit) {
+                   int kind, DType out_dt, long long shared_ff, UnitParams unit, UnitParams shared_unit,
+                   bool on_input) {
     need_float(out_dt, "activation output");
     long long width = (long long)n_experts * ff + shared_ff;
     if (width <= 0 || 2 * width > z.m) fail(JB_LLM_EINVAL, "gated_weighted: the product is narrower than the experts");
@@ -224,23 +225,30 @@ Buf gated_weighted(Device &d, const Stack &z, const float *weights, int w_ld, in
     const float u[6] = {unit.alpha, unit.limit, unit.shift, shared_unit.alpha, shared_unit.limit, shared_unit.shift};
     check(jb_gated_weighted(z.data(), z.S, z.stride(), as_int(z.m, "width"), weights, w_ld, n_experts,
                             as_int(ff, "width"), as_int(shared_ff, "width"), kind, kind == JB_ACT_SILU ? u : nullptr,
-                            out.ptr, out_dt, as_int(z.n, "rows"), d.stream),
+                            on_input ? 1 : 0, out.ptr, out_dt, as_int(z.n, "rows"), d.stream),
           "gated_weighted");
     return out;
 }
 
 Buf causal_conv(Device &d, const Stack &u, long long col0, long long C, const float *w, const float *bias,
                 int taps, float *state, long long slot_stride, const int32_t *row_pos, const int32_t *row_seq,
-                const int32_t *seq_slot, bool silu, DType out_dt, bool write_out, bool write_state) {
+                const int32_t *seq_slot, bool silu, DType out_dt, bool write_out, bool write_state,
+                const float *in_bias, Buf *parts, DType parts_dt, long long part) {
     need_float(out_dt, "causal_conv output");
     if (!u || col0 < 0 || C <= 0 || col0 + C > u.m) fail(JB_LLM_EINVAL, "causal_conv: the columns lie outside the product");
     Buf out;
     if (write_out) out = d.pool.get((size_t)u.n * (size_t)C * dtype_size(out_dt));
+    if (part <= 0 || !write_out) parts = nullptr;
+    if (parts) {
+        need_float(parts_dt, "causal_conv output");
+        *parts = d.pool.get((size_t)u.n * (size_t)C * dtype_size(parts_dt));
+    }
     int what = (write_out ? 1 : 0) | (write_state && taps > 1 ? 2 : 0);
     if (!what) return out;
     check(jb_causal_conv(u.data(), u.S, u.stride(), as_int(u.m, "width"), (int)col0, w, bias, state, slot_stride,
                          row_pos, row_seq, seq_slot, out.ptr, out_dt, as_int(C, "width"), as_int(u.n, "rows"),
-                         as_int(C, "width"), taps, silu ? 1 : 0, what, d.stream), "causal_conv");
+                         as_int(C, "width"), taps, silu ? 1 : 0, what, in_bias, parts ? parts->ptr : nullptr, parts_dt,
+                         (int)part, d.stream), "causal_conv");
     return out;
 }
 
@@ -276,6 +284,72 @@ Buf gated_part_norm(Device &d, const float *y, long long n, long long width, int
                              post ? post->S : 0, post ? post->stride() : 0, post ? as_int(post->m, "width") : 0,
                              (int)post_col0, post_silu ? 1 : 0, w, eps, out.ptr, out_dt, as_int(n, "rows"),
                              as_int(width, "width"), parts, few_rows ? 1 : 0, d.stream), "gated_part_norm");
+    return out;
+}
+
+Buf gated_memory(Device &d, const Stack &src, const GatedMemory &m, float *state, long long slot_stride,
+                 const int32_t *row_seq, const int32_t *seq_slot, int n_seqs, bool every_row_starts,
+                 long long max_len, DType out_dt) {
+    need_float(out_dt, "gated_memory output");
+    if (!src || !state) fail(JB_LLM_EINVAL, "gated_memory: no input or no state");
+    int n = as_int(src.n, "rows"), longest = (int)std::min<long long>(max_len, 0x7fffffff), starts = every_row_starts ? 1 : 0;
+    size_t values = (size_t)n * (size_t)m.H * (size_t)m.P, heads = (size_t)n * (size_t)m.H;
+    Buf y = d.pool.get(std::max<size_t>(values * 4, 16)), nq = d.pool.get(std::max<size_t>(heads * 4, 16)), em, scratch;
+    if (!every_row_starts) {
+        em = d.pool.get(std::max<size_t>(heads * 4, 16));
+        scratch = d.pool.get(std::max<size_t>((size_t)jb_gated_memory_scratch(n, n_seqs, longest, m.H, m.N, m.P, 0) * 4, 16));
+    }
+    check(jb_gated_memory_scan(src.data(), src.S, src.stride(), as_int(src.m, "width"), (int)m.val_col0, (int)m.key_col0,
+                               (int)m.qry_col0, (int)m.i_col0, (int)m.f_col0, m.i_bias, m.f_bias, m.cap, m.q_scale, state,
+                               slot_stride, row_seq, seq_slot, y.as<float>(), nq.as<float>(), em.as<float>(), n, n_seqs, m.H,
+                               m.N, m.P, starts, scratch.as<float>(), longest, d.stream), "gated_memory",
+          every_row_starts ? 1 : jb_matrix_state_scratch(n_seqs, longest, m.H, m.N, m.P) > 0 ? 4 : 2);
+    scratch = Buf();
+    Buf out = d.pool.get(std::max<size_t>(values * dtype_size(out_dt), 16));
+    check(jb_gated_memory_norm(y.as<float>(), nq.as<float>(), em.as<float>(), m.floor, src.data(), src.S, src.stride(),
+                               as_int(src.m, "width"), (int)m.gate_col0, (int)m.i_col0, (int)m.f_col0, m.i_bias, m.f_bias,
+                               m.cap, state, slot_stride, row_seq, seq_slot, m.w, m.eps, out.ptr, out_dt, n, m.H, m.N, m.P,
+                               d.stream), "gated_memory_norm");
+    return out;
+}
+
+Buf spread_streams(Device &d, const float *e, int ns, long long n, long long dm) {
+    Buf x = d.pool.get(std::max<size_t>((size_t)n * (size_t)ns * (size_t)dm * 4, 16));
+    check(jb_spread_streams(e, x.as<float>(), ns, as_int(n, "rows"), as_int(dm, "width"), d.stream), "spread_streams");
+    return x;
+}
+
+int max_streams() { return jb_max_streams(); }
+
+Buf streams(Device &d, float *x, int ns, long long n, long long dm, Stack *y, const StreamWrite *w,
+            const StreamRead *read, DType out_dt, const int32_t *rows, long long n_out, bool few_rows) {
+    need_float(out_dt, "streams output");
+    if (y && (!w || rows || y->n != n || y->m != dm)) fail(JB_LLM_EINVAL, "streams: the sublayer's result is not of the rows");
+    if (y) resolve_bias(d, *y);
+    long long outs = rows ? n_out : n;
+    Buf out;
+    if (read) out = d.pool.get(std::max<size_t>((size_t)outs * (size_t)dm * dtype_size(out_dt), 16));
+    check(jb_streams(x, ns, y ? y->data() : nullptr, y ? y->S : 0, y ? y->stride() : 0, y ? w->ls : nullptr,
+                     y ? w->out : nullptr, y ? w->mix : nullptr, y ? w->mult : 1.0f, rows, read ? read->in : nullptr,
+                     read ? read->norm.w : nullptr, read ? read->norm.b : nullptr, read ? read->norm.eps : 0.0f, out.ptr,
+                     out_dt, as_int(outs, "rows"), as_int(dm, "width"), few_rows ? 1 : 0, d.stream), "streams");
+    return out;
+}
+
+Buf lru(Device &d, const HeadStack &G, const LruParams &p, const float *u, long long W, const Stack &P, long long y_col0,
+        float *state, long long slot_stride, const int32_t *row_seq, const int32_t *seq_slot, int n_seqs,
+        bool every_row_starts, long long max_len, DType out_dt) {
+    need_float(out_dt, "lru output");
+    if (G.n != P.n || G.H <= 0 || G.m % 2 || (long long)G.H * (G.m / 2) != W)
+        fail(JB_LLM_EINVAL, "lru: the gates' products do not cover the channels");
+    int n = as_int(P.n, "rows"), w = as_int(W, "width"), longest = (int)std::min<long long>(max_len, 0x7fffffff);
+    long long need = every_row_starts ? 0 : jb_lru_scratch(n, n_seqs, longest, w);
+    Buf scratch;
+    if (need > 0) scratch = d.pool.get((size_t)need * 4);
+    Buf out = d.pool.get(std::max<size_t>((size_t)P.n * (size_t)W * dtype_size(out_dt), 16));
+    check(jb_lru(G.data(), G.S, (int)(G.m / 2), p.rb, p.ib, p.lam, u, P.data(), P.S, P.stride(), as_int(P.m, "width"),
+                 (int)y_col0, p.yb, state, slot_stride, row_seq, seq_slot, need > 0 ? scratch.as<float>() : nullptr, out.ptr,
+                 out_dt, n, n_seqs, w, every_row_starts ? 1 : 0, longest, d.stream), "lru", need > 0 ? 3 : 1);
     return out;
 }
 

@@ -140,19 +140,23 @@ Buf activation_weighted(Device &d, const Stack &z, long long width, const float 
                         long long ff, int kind, DType out_dt);
 
 // The same for experts with a gate: per expert [gate (ff) | up (ff)] in z's columns;
-// act(gate) * up * weights[row, expert] (silu: the gated unit), then the shared expert's shared_ff
+// act(gate) * up * weights[row, expert] (silu: the gated unit; on_input: act(w gate) * (w up), the weight w on
+// the expert's input), then the shared expert's shared_ff
 // values from the columns after the experts', without a weight: [n, n_experts ff + shared_ff] in out_dt.
 Buf gated_weighted(Device &d, const Stack &z, const float *weights, int w_ld, int n_experts, long long ff,
                    int kind, DType out_dt, long long shared_ff = 0, UnitParams unit = UnitParams(),
-                   UnitParams shared_unit = UnitParams());
+                   UnitParams shared_unit = UnitParams(), bool on_input = false);
 
 // A causal convolution over time on C columns (from col0) of a product's sums u, without
 // the input added: act(bias + sum_j w[:, j] u_{t - taps + 1 + j}) as [n, C] in out_dt (act:
 // "" or "silu"; bias float32 [C] or null; w float32 [C, taps]).  state: float32
 // [taps - 1, C] per slot, slot_stride floats apart.  write_out / write_state as short_conv.
+// in_bias: float32 [C] or null, added to the sums (the state holds them with it).  parts: with part > 0 the
+// result once more in parts_dt, equal parts of `part` columns, one part's rows together [C / part, n, part].
 Buf causal_conv(Device &d, const Stack &u, long long col0, long long C, const float *w, const float *bias,
                 int taps, float *state, long long slot_stride, const int32_t *row_pos, const int32_t *row_seq,
-                const int32_t *seq_slot, bool silu, DType out_dt, bool write_out, bool write_state);
+                const int32_t *seq_slot, bool silu, DType out_dt, bool write_out, bool write_state,
+                const float *in_bias = nullptr, Buf *parts = nullptr, DType parts_dt = F32, long long part = 0);
 
 // A recurrence with a matrix of N x P values per head as state (csrc/matrix_state.cu):
 // S_t = a_t S_{t-1} + b_t k_t v_t^T, y_t = S_t^T q_t + d v_t; y comes back as float32 [n, H P].
@@ -172,6 +176,36 @@ struct MatrixScan {
 Buf matrix_state_scan(Device &d, const Stack &src, const MatrixScan &m, float *state, long long slot_stride,
                       const int32_t *row_seq, const int32_t *seq_slot, int n_seqs, bool every_row_starts,
                       long long max_len = 0);
+// The matrix memory with exponential gates (csrc/matrix_state.cu): H heads of N key and P value values; src holds
+// v, k, q, the output gate and the two log gates, columns as given.  Returns, per head and row, the memory's
+// answer to q times q_scale divided by max(|n . q| q_scale, e^(-m)) + floor, RMS-normed per head, times w [H P],
+// times sigmoid of the output gate: [n, H P] in out_dt.  state: [H, (N P | N)] and [H] float32 per slot.
+struct GatedMemory {
+    int H = 0, N = 0, P = 0;
+    long long val_col0 = 0, key_col0 = 0, qry_col0 = 0, gate_col0 = 0, i_col0 = 0, f_col0 = 0;
+    const float *i_bias = nullptr, *f_bias = nullptr, *w = nullptr;
+    float cap = 1.0f, q_scale = 1.0f, floor = 0.0f, eps = 0.0f;
+};
+Buf gated_memory(Device &d, const Stack &src, const GatedMemory &m, float *state, long long slot_stride,
+                 const int32_t *row_seq, const int32_t *seq_slot, int n_seqs, bool every_row_starts,
+                 long long max_len, DType out_dt);
+// A residual stream of several streams per row, float32 [n, ns, dm] (csrc/streams.cu).
+// every stream of x from e [n, dm]
+Buf spread_streams(Device &d, const float *e, int ns, long long n, long long dm);
+int max_streams();
+// X_t <- sum_s mix[s, t] X_s + mult out[t] (ls * y), and with `read` the next reader's
+// u = sum_s in[s] X_s (in null: all ones) through a layer norm, [n, dm] in out_dt.  y null: the read alone, of the rows
+// `rows` (n_out indices on the device; null: all).  norm.w null: u itself, float32.
+struct StreamWrite {
+    const float *ls = nullptr, *out = nullptr, *mix = nullptr;
+    float mult = 1.0f;
+};
+struct StreamRead {
+    const float *in = nullptr;
+    LnParams norm;
+};
+Buf streams(Device &d, float *x, int ns, long long n, long long dm, Stack *y, const StreamWrite *w,
+            const StreamRead *read, DType out_dt, const int32_t *rows, long long n_out, bool few_rows);
 // A linear attention's q, k and v ahead of its recurrence: [q | k | v] (H D, H D and H Dv columns from
 // col0 of the sums) as one float32 stack, the first 2 rot_half values of every q and k head turned
 // (value i with value i + rot_half), k times key_scale.
@@ -229,6 +263,15 @@ struct HeadStack {
 };
 HeadStack linear_heads(Device &d, const void *a, DType a_dt, int H, long long n, long long k,
                        const DevTensor &w);
+// The real-gated linear recurrent unit (csrc/recurrent.cu): G the gates' product per block of channels [blocks, S, n,
+// r | i], u the convolved branch float32 [n, W], P the sums with the other branch in columns y_col0..; biases and lam
+// float32 [W].  S * gelu_tanh(y) as [n, W] in out_dt; state: float32 [W] per slot.
+struct LruParams {
+    const float *rb = nullptr, *ib = nullptr, *lam = nullptr, *yb = nullptr;
+};
+Buf lru(Device &d, const HeadStack &G, const LruParams &p, const float *u, long long W, const Stack &P, long long y_col0,
+        float *state, long long slot_stride, const int32_t *row_seq, const int32_t *seq_slot, int n_seqs,
+        bool every_row_starts, long long max_len, DType out_dt);
 // Into how many parts of k the tensor-core product is cut when the caller leaves it open.
 int linear_parts(long long n, long long m, long long k);
 // SiLU(a . gate^T) * (a . up^T) in one tensor-core kernel; an empty Buf when the

@@ -7,6 +7,10 @@
 //       k = B_g, q = C_g (N values), v = x_h (P values), d = D_h
 //   linear attention with a decay per head: a = decay_h, b = 1, d = 0, k, q, v the silu of
 //       the products' sums, G = H
+//   matrix memory with exponential gates (mLSTM): log gates i = c(zi), f = log sigmoid(c(zf)), c(z) =
+//       cap tanh(z / cap), a running maximum m_t = max(f + m_{t-1}, i), a = e^(f + m_{t-1} - m_t),
+//       b = e^(i - m_t), d = 0, G = H, and beside S a vector n_t = a n_{t-1} + b k_t per head, whose
+//       product with q divides y: y / (max(|n . q|, e^(-m_t)) + floor)
 //
 // and what follows them: a gate and an RMS norm in equal parts of the row, and the sum of
 // two mixers' results.  Everything here is float32: steps, decays, exponentials, the
@@ -20,6 +24,16 @@
 
 namespace jb {
 
+// The sums of a gated memory's two log gates: H columns each of [S, n, ld], biases [H], the soft cap.
+struct LogGates {
+    const float *src;
+    int S;
+    size_t stride;
+    int ld, i_col0, f_col0;
+    const float *i_bias, *f_bias;
+    float cap;
+};
+
 struct ScanIn {
     const float *src;          // sums [S, n, ld] that hold v, k and q
     int S;
@@ -32,12 +46,29 @@ struct ScanIn {
     int dt_ld, dt_col0;
     const float *dt_bias, *a_log, *skip;      // [H] each (with dt)
     const float *decay;                       // [H] (without dt)
+    // exponential gates (GATED kernels): per row and head a and b as they are ([n, H] each), or with
+    // coef_a null from the gates' sums and the running maximum in the state (a decode step's rows)
+    const float *coef_a, *coef_b;
+    LogGates gates;
+    float q_scale;             // y and nq are multiplied by it
+    float *nq;                 // [n, H]: n . q
 };
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
 // log(1 + e^v), the same number as the direct form wherever that does not overflow
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
+
+// row r's log input gate and log forget gate of head h
+__device__ __forceinline__ void log_gates(const LogGates &g, int r, int h, float &i, float &f)
+{
+    const float *row = g.src + (size_t)r * g.ld + h;
+    float zi = add_partials(g.i_bias[h], row + g.i_col0, g.S, g.stride);
+    float zf = add_partials(g.f_bias[h], row + g.f_col0, g.S, g.stride);
+    i = g.cap * tanhf(zi / g.cap);
+    zf = g.cap * tanhf(zf / g.cap);
+    f = fminf(zf, 0.0f) - log1pf(expf(-fabsf(zf)));
+}
 
 // an asynchronous copy of BYTES (4 or 16) from global to shared memory, and the wait for all of a thread's
 template <int BYTES>
@@ -62,6 +93,149 @@ __device__ __forceinline__ int first_row_of(const int32_t *__restrict__ row_seq,
     return lo;
 }
 
+// The gates of a step's rows ahead of a prompt's recurrence: a, b and e^(-m) per row and head, and the
+// slots' running maximum after the step (at m_off + h of a slot's state).  A block per (head,
+// sequence); a thread has consecutive rows, whose maps m -> max(m + F, M) are composed across the
+// block to give every thread the maximum it starts from.
+__global__ void __launch_bounds__(256)
+log_gates_kernel(LogGates g, float *__restrict__ state, size_t slot_stride, size_t m_off,
+                 const int32_t *__restrict__ row_seq, const int32_t *__restrict__ seq_slot,
+                 float *__restrict__ coef_a, float *__restrict__ coef_b, float *__restrict__ em, int n, int H)
+{
+    __shared__ float wF[8], wM[8], last[256];
+    pdl_trigger();
+    int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    int r0 = first_row_of(row_seq, n, seq), r1 = first_row_of(row_seq, n, seq + 1);
+    if (r0 >= r1)
+        return;
+    int per = (r1 - r0 + 255) / 256;
+    int t0 = min(r1, r0 + tid * per), t1 = min(r1, t0 + per);
+    float *mp = state + (size_t)seq_slot[seq] * slot_stride + m_off + h;
+    pdl_wait();
+    float m0 = *mp, F = 0.0f, M = -INFINITY;
+    for (int r = t0; r < t1; r++) {
+        float i, f;
+        log_gates(g, r, h, i, f);
+        F += f;
+        M = fmaxf(M + f, i);
+    }
+#pragma unroll
+    for (int o = 1; o < 32; o *= 2) {
+        float eF = __shfl_up_sync(0xffffffffu, F, o), eM = __shfl_up_sync(0xffffffffu, M, o);
+        if (lane >= o) {
+            M = fmaxf(eM + F, M);
+            F += eF;
+        }
+    }
+    if (lane == 31) {
+        wF[warp] = F;
+        wM[warp] = M;
+    }
+    F = __shfl_up_sync(0xffffffffu, F, 1);
+    M = __shfl_up_sync(0xffffffffu, M, 1);
+    __syncthreads();
+    float m = m0;
+    for (int w = 0; w < warp; w++)
+        m = fmaxf(m + wF[w], wM[w]);
+    if (lane > 0)
+        m = fmaxf(m + F, M);
+    // The first row's a is taken from the maximum that the thread before arrived at, not from the
+    // composed one, which differs from it in rounding: the products of the a telescope exactly.
+    float first_f = 0.0f, first_m = 0.0f;
+    for (int r = t0; r < t1; r++) {
+        float i, f;
+        log_gates(g, r, h, i, f);
+        float mn = fmaxf(f + m, i);
+        if (r == t0) {
+            first_f = f;
+            first_m = mn;
+        } else {
+            coef_a[(size_t)r * H + h] = expf(f + m - mn);
+        }
+        coef_b[(size_t)r * H + h] = expf(i - mn);
+        em[(size_t)r * H + h] = expf(-mn);
+        m = mn;
+    }
+    last[tid] = m;
+    __syncthreads();
+    if (t0 < t1) {
+        float before = tid > 0 ? last[tid - 1] : m0;
+        coef_a[(size_t)t0 * H + h] = expf(first_f + before - first_m);
+        if (t1 == r1)
+            *mp = m;
+    }
+}
+
+// The vector n of a gated memory over rows r0 .. r1 - 1 of one head: n <- a n + b k, and n . q
+// times q_scale to in.nq (MODE as in the kernel below: MODE 1 gives no n . q).  128 threads, one value
+// each, 128 values of n after the others.  from null: zeros; to null: nothing is written back.
+template <int MODE>
+__device__ __forceinline__ void normaliser_rows(const ScanIn &in, const float *from, float *to, int r0, int r1,
+                                                int H, int h, int N, float m_before, float (*red)[8])
+{
+    constexpr int TB = 8;
+    int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    auto sum = [&in](const float *p) {
+        float v = p[0];
+#pragma unroll 1
+        for (int k = 1; k < in.S; k++)
+            v += p[(size_t)k * in.stride];
+        return v;
+    };
+#pragma unroll 1
+    for (int n0 = 0; n0 < N; n0 += 128) {
+        bool live = n0 + tid < N;
+        float nv = from != nullptr && live ? from[n0 + tid] : 0.0f;
+        const float *col = in.src + (size_t)h * N + n0 + tid;
+#pragma unroll 1
+        for (int c0 = r0; c0 < r1; c0 += TB) {
+            int tb = min(TB, r1 - c0);
+            float k[TB], part[TB], a[TB], b[TB];
+#pragma unroll
+            for (int tt = 0; tt < TB; tt++) {
+                int r = min(c0 + tt, r1 - 1);
+                const float *row = col + (size_t)r * in.ld;
+                k[tt] = live ? sum(row + in.key_col0) : 0.0f;
+                part[tt] = MODE != 1 && live ? sum(row + in.qry_col0) : 0.0f;
+                if (in.coef_a != nullptr) {
+                    a[tt] = in.coef_a[(size_t)r * H + h];
+                    b[tt] = in.coef_b[(size_t)r * H + h];
+                }
+            }
+            if (in.coef_a == nullptr) {          // a decode step: one row
+                float i, f;
+                log_gates(in.gates, c0, h, i, f);
+                float mn = fmaxf(f + m_before, i);
+                a[0] = expf(f + m_before - mn);
+                b[0] = expf(i - mn);
+            }
+#pragma unroll
+            for (int tt = 0; tt < TB; tt++)
+                if (tt < tb) {
+                    nv = fmaf(b[tt], k[tt], a[tt] * nv);
+                    part[tt] *= nv;
+                }
+            if (MODE != 1) {
+#pragma unroll
+                for (int tt = 0; tt < TB; tt++) {
+                    part[tt] = warp_sum(part[tt]);
+                    if (lane == 0)
+                        red[warp][tt] = part[tt];
+                }
+                __syncthreads();
+                if (tid < tb) {
+                    float *o = in.nq + (size_t)(c0 + tid) * H + h;
+                    float v = ((red[0][tid] + red[1][tid]) + (red[2][tid] + red[3][tid])) * in.q_scale;
+                    *o = n0 > 0 ? *o + v : v;
+                }
+                __syncthreads();
+            }
+        }
+        if (to != nullptr && live)
+            to[n0 + tid] = nv;
+    }
+}
+
 // A block of 128 threads per (tile of P, head, sequence or piece of one).  A warp has
 // PW = 32 / nsplit columns p of the state, consecutive in memory, and nsplit lanes to a column;
 // the lanes of a column hold the rows n = (i nsplit + ns) 4 + j of it in registers (up to NR),
@@ -77,8 +251,10 @@ __device__ __forceinline__ int first_row_of(const int32_t *__restrict__ row_seq,
 //         by a sequence's last piece the slot's state.
 // With pieces, blockIdx.z counts (sequence, piece); pieces that hold no row return.
 // NS: the split where it is fixed at compile time (0: nsplit_arg says it).
+// GATED: exponential gates.  The state per head is then [N P | N] with n behind S, all heads' running
+// maxima follow ([H]), and one block more along x walks n.  The running maximum is not written here.
 // state: [H, N, P] per slot, slot_stride floats apart.  y: float32 [n, H P].
-template <int NR, int TB, int MODE, int NS>
+template <int NR, int TB, int MODE, int NS, bool GATED>
 __global__ void __launch_bounds__(128, NR <= 16 ? 5 : 3)
 matrix_state_scan_kernel(ScanIn in, float *__restrict__ state, size_t slot_stride,
                          const int32_t *__restrict__ row_seq, const int32_t *__restrict__ seq_slot,
@@ -125,12 +301,22 @@ matrix_state_scan_kernel(ScanIn in, float *__restrict__ state, size_t slot_strid
     }
     if (r0 >= r1)
         return;
-    float *st = MODE == 0 ? state + (size_t)seq_slot[seq] * slot_stride + (size_t)h * N * P
-                          : local + ((size_t)blockIdx.z * H + h) * N * P;
+    const size_t per_head = (size_t)N * P + (GATED ? N : 0);
+    float *slot = state + (size_t)seq_slot[seq] * slot_stride;
+    float *st = MODE == 0 ? slot + (size_t)h * per_head : local + ((size_t)blockIdx.z * H + h) * per_head;
     bool live = p < P;
-    float dskip = in.dt != nullptr && in.skip != nullptr ? in.skip[h] : 0.0f;
-    float a_neg = in.dt != nullptr ? -expf(in.a_log[h]) : 0.0f;
+    float dskip = !GATED && in.dt != nullptr && in.skip != nullptr ? in.skip[h] : 0.0f;
+    float a_neg = !GATED && in.dt != nullptr ? -expf(in.a_log[h]) : 0.0f;
     pdl_wait();
+    float m_before = GATED && in.coef_a == nullptr ? slot[(size_t)H * per_head + h] : 0.0f;
+    if (GATED && blockIdx.x == gridDim.x - 1) {
+        __shared__ float red[4][8];
+        const float *from = MODE == 1 ? nullptr : st + (size_t)N * P;
+        float *to = MODE != 2 ? st + (size_t)N * P
+                              : last_piece ? slot + (size_t)h * per_head + (size_t)N * P : nullptr;
+        normaliser_rows<MODE>(in, from, to, r0, r1, H, h, N, m_before, red);
+        return;
+    }
     float s[NR];
 #pragma unroll
     for (int i = 0; i < NR; i++) {
@@ -229,7 +415,18 @@ matrix_state_scan_kernel(ScanIn in, float *__restrict__ state, size_t slot_strid
             }
         }
         if (tid < tb) {
-            if (in.dt != nullptr) {
+            if (GATED) {
+                if (in.coef_a != nullptr) {
+                    a_s[tid] = in.coef_a[(size_t)(c0 + tid) * H + h];
+                    b_s[tid] = in.coef_b[(size_t)(c0 + tid) * H + h];
+                } else {
+                    float i, f;
+                    log_gates(in.gates, c0 + tid, h, i, f);
+                    float mn = fmaxf(f + m_before, i);
+                    a_s[tid] = expf(f + m_before - mn);
+                    b_s[tid] = expf(i - mn);
+                }
+            } else if (in.dt != nullptr) {
                 float d = add_partials(in.dt_bias[h], in.dt + (size_t)(c0 + tid) * in.dt_ld + in.dt_col0 + h, in.dt_S,
                                        in.dt_stride);
                 d = softplus_f(d);
@@ -298,14 +495,14 @@ matrix_state_scan_kernel(ScanIn in, float *__restrict__ state, size_t slot_strid
                 for (int o = 16; o >= PW; o >>= 1)
                     acc += __shfl_xor_sync(0xffffffffu, acc, o);
                 if (ns == 0 && live)
-                    y[(size_t)(c0 + tt) * H * P + (size_t)h * P + p] = fmaf(dskip, v, acc);
+                    y[(size_t)(c0 + tt) * H * P + (size_t)h * P + p] = GATED ? acc * in.q_scale : fmaf(dskip, v, acc);
             }
         }
     }
     // MODE 2: a sequence's last piece has walked the state to its end in the order of the one-pass
     // form; that is what the slot keeps (the carry pass's own end state differs from it in rounding)
     if (MODE == 2)
-        st = state + (size_t)seq_slot[seq] * slot_stride + (size_t)h * N * P;
+        st = slot + (size_t)h * per_head;
     if ((MODE != 2 || last_piece) && live) {
 #pragma unroll
         for (int i = 0; i < NR; i++) {
@@ -324,7 +521,7 @@ matrix_state_scan_kernel(ScanIn in, float *__restrict__ state, size_t slot_strid
 __global__ void __launch_bounds__(256)
 matrix_state_carry_kernel(float *__restrict__ state, size_t slot_stride, const int32_t *__restrict__ row_seq,
                           const int32_t *__restrict__ seq_slot, float *__restrict__ local,
-                          const float *__restrict__ decays, int n, int H, size_t per_head, int piece, int pieces)
+                          const float *decays, int n, int H, size_t per_head, int piece, int pieces)
 {
     pdl_trigger();
     int seq = blockIdx.y;
@@ -359,25 +556,59 @@ matrix_state_carry_kernel(float *__restrict__ state, size_t slot_stride, const i
     (void)S;         // the slot's state is written by the second pass's last piece
 }
 
+// A gated memory's division ahead of the norm: part `part` of row r is first divided by
+// max(|nq[r, part]|, e^(-m)) + floor.  em [n, parts] gives e^(-m); with em null (a decode step's rows) the
+// gates are taken again from their sums and the running maximum in the slot's state, and the
+// maximum after the row is written there.  nq null: no division.
+struct PartScale {
+    const float *nq, *em;
+    float floor;
+    LogGates gates;
+    float *state;
+    size_t slot_stride, m_off;
+    const int32_t *row_seq, *seq_slot;
+};
+
+// the factor on part `part` of row r, and where (null: nowhere) which maximum is to be written after
+// every thread of the part has called this
+__device__ __forceinline__ float part_factor(const PartScale &ps, int r, int part, int parts, float *&mp, float &m)
+{
+    mp = nullptr;
+    if (ps.nq == nullptr)
+        return 1.0f;
+    float e;
+    if (ps.em != nullptr) {
+        e = ps.em[(size_t)r * parts + part];
+    } else {
+        mp = ps.state + (size_t)ps.seq_slot[ps.row_seq[r]] * ps.slot_stride + ps.m_off + part;
+        float i, f;
+        log_gates(ps.gates, r, part, i, f);
+        m = fmaxf(f + *mp, i);
+        e = expf(-m);
+    }
+    return 1.0f / (fmaxf(fabsf(ps.nq[(size_t)r * parts + part]), e) + ps.floor);
+}
+
 // out[r, c] = rms_part(y[r, :] * pre)[c] * w[c] * post, where pre = silu of the sums in
 // columns pre_col0.. of `pre` (null: 1), post = sigmoid (post_silu: silu) of the sums in columns
 // post_col0.. of `post` (null: 1), w null is a weight of 1, and the row is normed in `parts` equal parts, each by its own root
 // mean square.  A block per (row, part).
 template <typename TO>
 __global__ void __launch_bounds__(256)
-gated_part_norm_kernel(const float *__restrict__ y, const float *__restrict__ pre, int pre_S, size_t pre_stride,
-                       int pre_ld, int pre_col0, const float *__restrict__ post, int post_S, size_t post_stride,
+gated_part_norm_kernel(const float *y, const float *pre, int pre_S, size_t pre_stride,
+                       int pre_ld, int pre_col0, const float *post, int post_S, size_t post_stride,
                        int post_ld, int post_col0, const float *__restrict__ w, float eps, TO *__restrict__ out,
-                       int width, int parts, int keep, int post_silu)
+                       int width, int parts, int keep, int post_silu, PartScale ps)
 {
     extern __shared__ float held[];          // the part's gated values, where they fit (keep != 0)
     __shared__ float red[32];
     pdl_trigger();
     int r = blockIdx.x, part = blockIdx.y, len = width / parts, c0 = part * len;
     pdl_wait();
-    float ss = 0.0f;
+    float ss = 0.0f, m_new = 0.0f, *mp;
+    const float div = part_factor(ps, r, part, parts, mp, m_new);
     for (int c = c0 + threadIdx.x; c < c0 + len; c += blockDim.x) {
-        float v = y[(size_t)r * width + c];
+        float v = y[(size_t)r * width + c] * div;
         if (pre != nullptr)
             v *= silu_f(add_partials(0.0f, pre + (size_t)r * pre_ld + pre_col0 + c, pre_S, pre_stride));
         if (keep)
@@ -385,13 +616,15 @@ gated_part_norm_kernel(const float *__restrict__ y, const float *__restrict__ pr
         ss = fmaf(v, v, ss);
     }
     ss = block_sum(ss, red);
+    if (mp != nullptr && threadIdx.x == 0)
+        *mp = m_new;           // every thread has read the old one: block_sum met them all
     float scale = 1.0f / sqrtf(ss / (float)len + eps);
     for (int c = c0 + threadIdx.x; c < c0 + len; c += blockDim.x) {
         float v;
         if (keep) {
             v = held[c - c0];
         } else {
-            v = y[(size_t)r * width + c];
+            v = y[(size_t)r * width + c] * div;
             if (pre != nullptr)
                 v *= silu_f(add_partials(0.0f, pre + (size_t)r * pre_ld + pre_col0 + c, pre_S, pre_stride));
         }
@@ -410,10 +643,10 @@ gated_part_norm_kernel(const float *__restrict__ y, const float *__restrict__ pr
 // a lane and up to U of those; lengths, columns and rows are multiples of four.
 template <typename TO, int U>
 __global__ void __launch_bounds__(256)
-gated_part_norm_warp_kernel(const float *__restrict__ y, const float *__restrict__ pre, int pre_S, size_t pre_stride,
-                            int pre_ld, int pre_col0, const float *__restrict__ post, int post_S, size_t post_stride,
+gated_part_norm_warp_kernel(const float *y, const float *pre, int pre_S, size_t pre_stride,
+                            int pre_ld, int pre_col0, const float *post, int post_S, size_t post_stride,
                             int post_ld, int post_col0, const float *__restrict__ w, float eps, TO *__restrict__ out,
-                            int width, int parts, int post_silu, unsigned tasks)
+                            int width, int parts, int post_silu, unsigned tasks, PartScale ps)
 {
     pdl_trigger();
     unsigned task = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -432,7 +665,8 @@ gated_part_norm_warp_kernel(const float *__restrict__ y, const float *__restrict
     };
     pdl_wait();
     float4 v[U], g[U];
-    float ss = 0.0f;
+    float ss = 0.0f, m_new = 0.0f, *mp;
+    const float div = part_factor(ps, (int)r, c0 / len, parts, mp, m_new);
 #pragma unroll
     for (int u = 0; u < U; u++) {
         int c = c0 + 4 * (lane + 32 * u);
@@ -440,6 +674,7 @@ gated_part_norm_warp_kernel(const float *__restrict__ y, const float *__restrict
         if (c >= c0 + len)
             continue;
         v[u] = load4(y + (size_t)r * width + c);
+        v[u] = make_float4(v[u].x * div, v[u].y * div, v[u].z * div, v[u].w * div);
         if (post != nullptr)
             g[u] = sums4(post + (size_t)r * post_ld + post_col0 + c, post_S, post_stride);
         if (pre != nullptr) {
@@ -449,6 +684,8 @@ gated_part_norm_warp_kernel(const float *__restrict__ y, const float *__restrict
         ss = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, fmaf(v[u].z, v[u].z, fmaf(v[u].w, v[u].w, ss))));
     }
     ss = warp_sum(ss);
+    if (mp != nullptr && lane == 0)
+        *mp = m_new;           // every lane has read the old one: warp_sum met them all
     float scale = 1.0f / sqrtf(ss / (float)len + eps);
 #pragma unroll
     for (int u = 0; u < U; u++) {
@@ -553,8 +790,8 @@ turn_heads_kernel(const float *__restrict__ src, int S, size_t stride, int ld, i
 // held in shared memory; the CTAs exchange their sums of squares through one another's shared memory.
 template <typename TO, int C>
 __global__ void __launch_bounds__(256)
-gated_part_norm_cluster_kernel(const float *__restrict__ y, const float *__restrict__ pre, int pre_S,
-                               size_t pre_stride, int pre_ld, int pre_col0, const float *__restrict__ post,
+gated_part_norm_cluster_kernel(const float *y, const float *pre, int pre_S,
+                               size_t pre_stride, int pre_ld, int pre_col0, const float *post,
                                int post_S, size_t post_stride, int post_ld, int post_col0,
                                const float *__restrict__ w, float eps, TO *__restrict__ out, int width, int parts,
                                int cols, int post_silu)
@@ -601,7 +838,7 @@ gated_part_norm_cluster_kernel(const float *__restrict__ y, const float *__restr
 // out = sl * rms(sum L) wl + sr * rms(sum R) wr (each normed over the whole row).
 // A block per row; out: float32 [n, m].
 __global__ void __launch_bounds__(256)
-pair_combine_kernel(const float *__restrict__ L, int SL, size_t strideL, const float *__restrict__ R, int SR,
+pair_combine_kernel(const float *L, int SL, size_t strideL, const float *R, int SR,
                     size_t strideR, const float *__restrict__ wl, const float *__restrict__ wr, float sl, float sr,
                     float eps, float *__restrict__ out, int m)
 {
@@ -637,7 +874,7 @@ pair_combine_kernel(const float *__restrict__ L, int SL, size_t strideL, const f
 // shared memory; the CTAs exchange their sums of squares through one another's shared memory.
 template <int C>
 __global__ void __launch_bounds__(256)
-pair_combine_cluster_kernel(const float *__restrict__ L, int SL, size_t strideL, const float *__restrict__ R, int SR,
+pair_combine_cluster_kernel(const float *L, int SL, size_t strideL, const float *R, int SR,
                             size_t strideR, const float *__restrict__ wl, const float *__restrict__ wr, float sl,
                             float sr, float eps, float *__restrict__ out, int m, int cols)
 {
@@ -726,35 +963,24 @@ static int scan_nsplit(int N, int P, int per_lane)
 // rows to a piece when long sequences are cut into pieces that run side by side
 extern "C" int jb_matrix_state_piece(void) { return 128; }
 // Floats of scratch for a step whose longest sequence brings max_len rows (0: one pass does it).
-extern "C" long long jb_matrix_state_scratch(int n_seqs, int max_len, int H, int N, int P)
+static long long matrix_scratch(int n_seqs, int max_len, int H, size_t per_head)
 {
     int piece = jb_matrix_state_piece();
     if (max_len < 2 * piece)
         return 0;
     long long pieces = (max_len + piece - 1) / piece;
-    long long need = (long long)n_seqs * pieces * ((long long)H * N * P + H);
+    long long need = (long long)n_seqs * pieces * ((long long)H * (long long)per_head + H);
     return need > (1ll << 28) ? 0 : need;       // more than 1 GiB of scratch: one pass after all
 }
-
-// src: float32 [S, n, ld] holding v (H P columns from val_col0), k and q (G N columns each);
-// with dt (sums [dt_S, n, dt_ld], H columns from dt_col0) the selective form, otherwise
-// decay [H].  state: [H, N, P] per slot.  y: float32 [n, H P].  scratch (with max_len, the most
-// rows a sequence brings): jb_matrix_state_scratch floats, or null for one pass.
-extern "C" int jb_matrix_state_scan(const float *src, int S, long long stride, int ld, int val_col0, int key_col0,
-                                    int qry_col0, int silu, const float *dt, int dt_S, long long dt_stride,
-                                    int dt_ld, int dt_col0, const float *dt_bias, const float *a_log,
-                                    const float *skip, const float *decay, float *state, long long slot_stride,
-                                    const int32_t *row_seq, const int32_t *seq_slot, float *y, int n, int n_seqs,
-                                    int H, int G, int N, int P, int every_row_starts, float *scratch, int max_len,
-                                    cudaStream_t st)
+extern "C" long long jb_matrix_state_scratch(int n_seqs, int max_len, int H, int N, int P)
 {
-    if (n <= 0 || n_seqs <= 0)
-        return JB_OK;
-    if (H <= 0 || G <= 0 || H % G || N <= 0 || N > 1024 || P <= 0 || S <= 0 || src == nullptr || state == nullptr ||
-        y == nullptr || (dt != nullptr && (dt_bias == nullptr || a_log == nullptr || dt_S <= 0)) ||
-        (dt == nullptr && decay == nullptr) || H > 65535 || n_seqs > 65535 ||
-        ld < val_col0 + H * P || ld < key_col0 + G * N || ld < qry_col0 + G * N)
-        return JB_EINVAL;
+    return matrix_scratch(n_seqs, max_len, H, (size_t)N * P);
+}
+
+static int scan_launch(const ScanIn &in, bool gated, float *state, long long slot_stride, const int32_t *row_seq,
+                       const int32_t *seq_slot, float *y, int n, int n_seqs, int H, int G, int N, int P,
+                       int every_row_starts, float *scratch, int max_len, cudaStream_t st)
+{
     // 16 state values to a lane (more blocks, fewer registers, a shorter chain per row) where 32
     // lanes to a column are enough for that; 32 otherwise
     // (a decode step's one row per sequence moves the state and little else: fewer lanes to a
@@ -766,30 +992,33 @@ extern "C" int jb_matrix_state_scan(const float *src, int S, long long stride, i
     constexpr int TB = 16;
     int PT = 128 / nsplit;
     int NP = (N + 4 * nsplit - 1) / (4 * nsplit) * (4 * nsplit);
-    ScanIn in{src, S, (size_t)stride, ld, val_col0, key_col0, qry_col0, silu, dt, dt_S, (size_t)dt_stride, dt_ld,
-              dt_col0, dt_bias, a_log, skip, decay};
-    unsigned ptiles = (unsigned)((P + PT - 1) / PT);
+    unsigned ptiles = (unsigned)((P + PT - 1) / PT) + (gated ? 1u : 0u);     // gated: a block more for n
     size_t smem = (size_t)TB * (2 * NP + PT + 2) * 4;
+    const size_t per_head = (size_t)N * P + (gated ? N : 0);
     int piece = jb_matrix_state_piece();
-    bool whole = scratch == nullptr || every_row_starts || jb_matrix_state_scratch(n_seqs, max_len, H, N, P) == 0;
+    bool whole = scratch == nullptr || every_row_starts || matrix_scratch(n_seqs, max_len, H, per_head) == 0;
     int pieces = whole ? 1 : (max_len + piece - 1) / piece;
     if ((long long)n_seqs * pieces > 65535)
         return JB_EINVAL;
-    size_t per_head = (size_t)N * P;
     float *local = scratch, *decays = whole ? nullptr : scratch + (size_t)n_seqs * pieces * H * per_head;
     dim3 grid(ptiles, (unsigned)H, (unsigned)(n_seqs * pieces));
-#define JB_SCAN_N(NRV, MODE, NSV, SMEM)                                                                        \
+#define JB_SCAN_G(NRV, MODE, NSV, GT, SMEM)                                                                        \
     do {                                                                                                       \
         if ((SMEM) > 48 * 1024) {                                                                              \
             /* long states: the rows in shared memory need more than a kernel gets unasked */                  \
-            static const bool asked = cudaFuncSetAttribute(matrix_state_scan_kernel<NRV, TB, MODE, NSV>,       \
+            static const bool asked = cudaFuncSetAttribute(matrix_state_scan_kernel<NRV, TB, MODE, NSV, GT>,   \
                                                            cudaFuncAttributeMaxDynamicSharedMemorySize,        \
                                                            160 * 1024) == cudaSuccess;                         \
             (void)asked;                                                                                       \
         }                                                                                                      \
-        launch(matrix_state_scan_kernel<NRV, TB, MODE, NSV>, grid, 128, (SMEM), st, in, state,                 \
+        launch(matrix_state_scan_kernel<NRV, TB, MODE, NSV, GT>, grid, 128, (SMEM), st, in, state,                 \
                (size_t)slot_stride, row_seq, seq_slot, y, local, decays, n, H, G, N, P, nsplit,                \
                whole ? every_row_starts : 0, whole ? 0 : piece, pieces);                                       \
+    } while (0)
+#define JB_SCAN_N(NRV, MODE, NSV, SMEM)                                        \
+    do {                                                                       \
+        if (gated) JB_SCAN_G(NRV, MODE, NSV, true, SMEM);                      \
+        else JB_SCAN_G(NRV, MODE, NSV, false, SMEM);                           \
     } while (0)
     // the commonest shapes have kernels of their own: 128 or 64 state rows, 16 to a lane (prompts),
     // 128 rows, 32 to a lane (decode rows)
@@ -812,13 +1041,85 @@ extern "C" int jb_matrix_state_scan(const float *src, int S, long long stride, i
     JB_SCAN(2, smem);
 #undef JB_SCAN
 #undef JB_SCAN_N
+#undef JB_SCAN_G
     return launch_status();
 }
 
-extern "C" int jb_gated_part_norm(const float *y, const float *pre, int pre_S, long long pre_stride, int pre_ld,
+// src: float32 [S, n, ld] holding v (H P columns from val_col0), k and q (G N columns each);
+// with dt (sums [dt_S, n, dt_ld], H columns from dt_col0) the selective form, otherwise
+// decay [H].  state: [H, N, P] per slot.  y: float32 [n, H P].  scratch (with max_len, the most
+// rows a sequence brings): jb_matrix_state_scratch floats, or null for one pass.
+extern "C" int jb_matrix_state_scan(const float *src, int S, long long stride, int ld, int val_col0, int key_col0,
+                                    int qry_col0, int silu, const float *dt, int dt_S, long long dt_stride,
+                                    int dt_ld, int dt_col0, const float *dt_bias, const float *a_log,
+                                    const float *skip, const float *decay, float *state, long long slot_stride,
+                                    const int32_t *row_seq, const int32_t *seq_slot, float *y, int n, int n_seqs,
+                                    int H, int G, int N, int P, int every_row_starts, float *scratch, int max_len,
+                                    cudaStream_t st)
+{
+    if (n <= 0 || n_seqs <= 0)
+        return JB_OK;
+    if (H <= 0 || G <= 0 || H % G || N <= 0 || N > 1024 || P <= 0 || S <= 0 || src == nullptr || state == nullptr ||
+        y == nullptr || (dt != nullptr && (dt_bias == nullptr || a_log == nullptr || dt_S <= 0)) ||
+        (dt == nullptr && decay == nullptr) || H > 65535 || n_seqs > 65535 ||
+        ld < val_col0 + H * P || ld < key_col0 + G * N || ld < qry_col0 + G * N)
+        return JB_EINVAL;
+    ScanIn in{src, S, (size_t)stride, ld, val_col0, key_col0, qry_col0, silu, dt, dt_S, (size_t)dt_stride, dt_ld,
+              dt_col0, dt_bias, a_log, skip, decay, nullptr, nullptr, LogGates(), 1.0f, nullptr};
+    return scan_launch(in, false, state, slot_stride, row_seq, seq_slot, y, n, n_seqs, H, G, N, P, every_row_starts,
+                       scratch, max_len, st);
+}
+
+// Floats of scratch of jb_gated_memory_scan: the gates' a and b per row and head (not in a decode
+// step), then what the pieces need.
+extern "C" long long jb_gated_memory_scratch(int n, int n_seqs, int max_len, int H, int N, int P, int every_row_starts)
+{
+    if (every_row_starts)
+        return 0;
+    return 2ll * n * H + matrix_scratch(n_seqs, max_len, H, (size_t)N * P + N);
+}
+
+// The gated memory's recurrence.  src: float32 [S, n, ld] holding v (H P columns), k and q (H N each) and
+// the two log gates (H each); i_bias, f_bias [H].  state per slot: [H, (N P | N)] and [H] running maxima.
+// y: [n, H P] and nq: [n, H], both times q_scale and not yet divided.  em: [n, H], e^(-m), written
+// unless every row starts (a decode step: the norm that follows takes the gates again and
+// writes the running maxima).
+extern "C" int jb_gated_memory_scan(const float *src, int S, long long stride, int ld, int val_col0, int key_col0,
+                                    int qry_col0, int i_col0, int f_col0, const float *i_bias, const float *f_bias,
+                                    float cap, float q_scale, float *state, long long slot_stride,
+                                    const int32_t *row_seq, const int32_t *seq_slot, float *y, float *nq, float *em,
+                                    int n, int n_seqs, int H, int N, int P, int every_row_starts, float *scratch,
+                                    int max_len, cudaStream_t st)
+{
+    if (n <= 0 || n_seqs <= 0)
+        return JB_OK;
+    if (H <= 0 || N <= 0 || N > 1024 || P <= 0 || S <= 0 || src == nullptr || state == nullptr || y == nullptr ||
+        nq == nullptr || i_bias == nullptr || f_bias == nullptr || !(cap > 0.0f) || H > 65535 || n_seqs > 65535 ||
+        (!every_row_starts && (scratch == nullptr || em == nullptr)) || ld < val_col0 + H * P || ld < key_col0 + H * N ||
+        ld < qry_col0 + H * N || ld < i_col0 + H || ld < f_col0 + H)
+        return JB_EINVAL;
+    LogGates g{src, S, (size_t)stride, ld, i_col0, f_col0, i_bias, f_bias, cap};
+    ScanIn in{src, S, (size_t)stride, ld, val_col0, key_col0, qry_col0, 0, nullptr, 0, 0, 0,
+              0, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, g, q_scale, nq};
+    if (!every_row_starts) {
+        size_t m_off = (size_t)H * ((size_t)N * P + N);
+        float *ca = scratch, *cb = scratch + (size_t)n * H;
+        launch(log_gates_kernel, dim3((unsigned)H, (unsigned)n_seqs), 256, 0, st, g, state, (size_t)slot_stride, m_off,
+               row_seq, seq_slot, ca, cb, em, n, H);
+        in.coef_a = ca;
+        in.coef_b = cb;
+        scratch += 2 * (size_t)n * H;
+        if (matrix_scratch(n_seqs, max_len, H, (size_t)N * P + N) == 0)
+            scratch = nullptr;
+    }
+    return scan_launch(in, true, state, slot_stride, row_seq, seq_slot, y, n, n_seqs, H, H, N, P, every_row_starts,
+                       scratch, max_len, st);
+}
+
+static int part_norm_launch(const float *y, const float *pre, int pre_S, long long pre_stride, int pre_ld,
                                   int pre_col0, const float *post, int post_S, long long post_stride, int post_ld,
                                   int post_col0, int post_silu, const float *w, float eps, void *out, int out_dt,
-                                  int n, int width, int parts, int few_rows, cudaStream_t st)
+                                  int n, int width, int parts, int few_rows, const PartScale &ps, cudaStream_t st)
 {
     if (n <= 0)
         return JB_OK;
@@ -826,7 +1127,7 @@ extern "C" int jb_gated_part_norm(const float *y, const float *pre, int pre_S, l
         (pre != nullptr && (pre_S <= 0 || pre_ld < pre_col0 + width)) ||
         (post != nullptr && (post_S <= 0 || post_ld < post_col0 + width)))
         return JB_EINVAL;
-    if (few_rows && n * parts <= 64 && width / parts >= 512 && out_dt == JB_BF16) {
+    if (few_rows && ps.nq == nullptr && n * parts <= 64 && width / parts >= 512 && out_dt == JB_BF16) {
         // few blocks otherwise: a cluster of CTAs per (row, part)
         constexpr int C = 4;
         int cols = (width / parts + C - 1) / C;
@@ -852,7 +1153,7 @@ extern "C" int jb_gated_part_norm(const float *y, const float *pre, int pre_S, l
 #define JB_GPN(TO, U)                                                                                          \
     launch(gated_part_norm_warp_kernel<TO, U>, g, 32 * warps, 0, st, y, pre, pre_S, (size_t)pre_stride, pre_ld,  \
            pre_col0, post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (TO *)out, width, parts,     \
-           post_silu, tasks)
+           post_silu, tasks, ps)
         if (out_dt == JB_F32) {
             if (len <= 128) JB_GPN(float, 1); else JB_GPN(float, 2);
         } else {
@@ -866,13 +1167,44 @@ extern "C" int jb_gated_part_norm(const float *y, const float *pre, int pre_S, l
     int threads = len >= 1024 ? 256 : 128;
     if (out_dt == JB_F32)
         launch(gated_part_norm_kernel<float>, grid, threads, smem, st, y, pre, pre_S, (size_t)pre_stride, pre_ld, pre_col0,
-               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (float *)out, width, parts, keep, post_silu);
+               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (float *)out, width, parts, keep, post_silu, ps);
     else if (out_dt == JB_BF16)
         launch(gated_part_norm_kernel<bf16>, grid, threads, smem, st, y, pre, pre_S, (size_t)pre_stride, pre_ld, pre_col0,
-               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (bf16 *)out, width, parts, keep, post_silu);
+               post, post_S, (size_t)post_stride, post_ld, post_col0, w, eps, (bf16 *)out, width, parts, keep, post_silu, ps);
     else
         return JB_EINVAL;
     return launch_status();
+}
+
+extern "C" int jb_gated_part_norm(const float *y, const float *pre, int pre_S, long long pre_stride, int pre_ld,
+                                  int pre_col0, const float *post, int post_S, long long post_stride, int post_ld,
+                                  int post_col0, int post_silu, const float *w, float eps, void *out, int out_dt,
+                                  int n, int width, int parts, int few_rows, cudaStream_t st)
+{
+    return part_norm_launch(y, pre, pre_S, pre_stride, pre_ld, pre_col0, post, post_S, post_stride, post_ld, post_col0,
+                            post_silu, w, eps, out, out_dt, n, width, parts, few_rows, PartScale(), st);
+}
+
+// What follows jb_gated_memory_scan: y [n, H P] divided per head by max(|nq|, e^(-m)) + floor, each head
+// RMS-normed, times w [H P], times the sigmoid of the sums in columns g_col0.. of src.  em as the scan
+// left it, or null for a decode step's rows (then the gates' sums and the state, as the scan took them).
+extern "C" int jb_gated_memory_norm(const float *y, const float *nq, const float *em, float floor, const float *src,
+                                    int S, long long stride, int ld, int g_col0, int i_col0, int f_col0,
+                                    const float *i_bias, const float *f_bias, float cap, float *state,
+                                    long long slot_stride, const int32_t *row_seq, const int32_t *seq_slot,
+                                    const float *w, float eps, void *out, int out_dt, int n, int H, int N, int P,
+                                    cudaStream_t st)
+{
+    if (n <= 0)
+        return JB_OK;
+    if (nq == nullptr || src == nullptr || S <= 0 || H <= 0 || N <= 0 || P <= 0 || ld < g_col0 + H * P ||
+        (em == nullptr && (state == nullptr || i_bias == nullptr || f_bias == nullptr || row_seq == nullptr ||
+                           seq_slot == nullptr || ld < i_col0 + H || ld < f_col0 + H || !(cap > 0.0f))))
+        return JB_EINVAL;
+    PartScale ps{nq, em, floor, LogGates{src, S, (size_t)stride, ld, i_col0, f_col0, i_bias, f_bias, cap}, state,
+                 (size_t)slot_stride, (size_t)H * ((size_t)N * P + N), row_seq, seq_slot};
+    return part_norm_launch(y, nullptr, 0, 0, 0, 0, src, S, stride, ld, g_col0, 0, w, eps, out, out_dt, n, H * P, H, 0,
+                            ps, st);
 }
 
 // src: sums [S, n, ld]; out: float32 [n, 2 H D + H Dv].  See turn_heads_kernel.

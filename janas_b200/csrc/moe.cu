@@ -228,13 +228,15 @@ __device__ __forceinline__ float gated_value(float g, float u, int kind, const G
 // The same for experts with a gate: expert e's sums are [gate (ff) | up (ff)] in columns
 // 2 e ff .. of z, and out[r, e ff + j] = act(gate_j) * up_j * weights[r, e]; then a shared expert's
 // shared_ff values without a weight, its sums [gate | up] after the experts'; out: [n, width].
+// on_input: the weight stands on the expert's input instead, act(weight gate_j) * (weight up_j).
 // V values per thread (V = 4: ff and shared_ff multiples of four and everything on 16-byte
 // boundaries).
 template <typename TO, int V>
 __global__ void __launch_bounds__(256)
 gated_weighted_kernel(const float *__restrict__ z, int S, size_t stride, int ld,
                       const float *__restrict__ weights, int w_ld, int n_experts, int ff, int shared_ff,
-                      int kind, GatedUnit unit, GatedUnit shared_unit, TO *__restrict__ out, int width)
+                      int kind, GatedUnit unit, GatedUnit shared_unit, TO *__restrict__ out, int width,
+                      int on_input)
 {
     pdl_trigger();
     int r = blockIdx.x, c = (int)(blockIdx.y * blockDim.x + threadIdx.x) * V;
@@ -262,6 +264,11 @@ gated_weighted_kernel(const float *__restrict__ z, int S, size_t stride, int ld,
                 u.x += b.x; u.y += b.y; u.z += b.z; u.w += b.w;
             }
         float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (on_input && wgt != 0.0f) {
+            g = make_float4(g.x * wgt, g.y * wgt, g.z * wgt, g.w * wgt);
+            u = make_float4(u.x * wgt, u.y * wgt, u.z * wgt, u.w * wgt);
+            wgt = 1.0f;
+        }
         if (wgt != 0.0f)
             v = make_float4(gated_value(g.x, u.x, kind, unit) * wgt, gated_value(g.y, u.y, kind, unit) * wgt,
                             gated_value(g.z, u.z, kind, unit) * wgt, gated_value(g.w, u.w, kind, unit) * wgt);
@@ -270,7 +277,7 @@ gated_weighted_kernel(const float *__restrict__ z, int S, size_t stride, int ld,
         float v = 0.0f;
         if (wgt != 0.0f) {
             float g = add_partials(0.0f, src, S, stride), u = add_partials(0.0f, src + up, S, stride);
-            v = gated_value(g, u, kind, unit) * wgt;
+            v = on_input ? gated_value(g * wgt, u * wgt, kind, unit) : gated_value(g, u, kind, unit) * wgt;
         }
         out[(size_t)r * width + c] = from_f<TO>(v);
     }
@@ -368,10 +375,11 @@ extern "C" int jb_activation_weighted(const float *z, int S, long long stride, i
 // then ff up values, and then a shared expert's 2 shared_ff columns (shared_ff 0: none); weights:
 // float32 [n, w_ld].  out: [n, n_experts ff + shared_ff] in out_dt.  unit: the three constants
 // {alpha, limit, shift} of the experts' gated unit and after them the shared expert's three, on
-// the host (null: SiLU(gate) * up); they are for JB_ACT_SILU alone.
+// the host (null: SiLU(gate) * up); they are for JB_ACT_SILU alone.  on_input: the weights stand on the
+// experts' inputs.
 extern "C" int jb_gated_weighted(const float *z, int S, long long stride, int ld, const float *weights, int w_ld,
-                                 int n_experts, int ff, int shared_ff, int kind, const float *unit, void *out,
-                                 int out_dt, int n, cudaStream_t st)
+                                 int n_experts, int ff, int shared_ff, int kind, const float *unit, int on_input,
+                                 void *out, int out_dt, int n, cudaStream_t st)
 {
     if (n <= 0)
         return JB_OK;
@@ -392,7 +400,7 @@ extern "C" int jb_gated_weighted(const float *z, int S, long long stride, int ld
     dim3 grid((unsigned)n, (unsigned)((per_row + 255) / 256));
 #define JB_GW(TO, V)                                                                                         \
     launch(gated_weighted_kernel<TO, V>, grid, 256, 0, st, z, S, (size_t)stride, ld, weights, w_ld, n_experts, ff, \
-           shared_ff, kind, u, us, (TO *)out, (int)width)
+           shared_ff, kind, u, us, (TO *)out, (int)width, on_input)
     if (out_dt == JB_F32) {
         if (vec) JB_GW(float, 4); else JB_GW(float, 1);
     } else if (out_dt == JB_BF16) {

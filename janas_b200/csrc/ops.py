@@ -538,11 +538,12 @@ def moe_route(P: torch.Tensor, col0: int, outputs: int, correction: Optional[tor
 
 def gated_weighted(z: torch.Tensor, weights: torch.Tensor, n_experts: int, ff: int, kind: str,
                    out_dtype: torch.dtype, shared_ff: int = 0,
-                   units: Optional[Tuple[float, ...]] = None) -> torch.Tensor:
+                   units: Optional[Tuple[float, ...]] = None, on_input: bool = False) -> torch.Tensor:
     """act(gate) * up * weights[row, expert] for experts whose sums lie [gate (ff) | up (ff)] one
     after the other in z [S, n, ld], then a shared expert's shared_ff values without a weight:
     [n, n_experts * ff + shared_ff].  units (silu alone): alpha, limit, shift of the experts' gated
-    unit and then of the shared expert's."""
+    unit and then of the shared expert's.  on_input: the weight stands on the expert's input,
+    act(weight gate) * (weight up)."""
     z = stack(z)
     _need(z, "z", torch.float32, (None, None, None))
     S, n, ld = z.shape
@@ -551,28 +552,123 @@ def gated_weighted(z: torch.Tensor, weights: torch.Tensor, n_experts: int, ff: i
     u = None if units is None else (ctypes.c_float * 6)(*units)
     kinds = {"relu2": 0, "relu": 1, "gelu_tanh": 2, "silu": 3}
     _check(lib().jb_gated_weighted(_p(z), S, n * ld, ld, _p(weights), weights.shape[1], n_experts, ff,
-                                   shared_ff, kinds[kind], u, _p(out), _DT[out_dtype], n, _stream()), "gated_weighted")
+                                   shared_ff, kinds[kind], u, 1 if on_input else 0, _p(out), _DT[out_dtype], n,
+                                   _stream()), "gated_weighted")
     return out
 
 
 def causal_conv(u: torch.Tensor, col0: int, C: int, w: torch.Tensor, bias: Optional[torch.Tensor],
                 state: Optional[torch.Tensor], row_pos: torch.Tensor, row_seq: torch.Tensor,
                 seq_slot: torch.Tensor, silu: bool, out_dtype: torch.dtype, write_out: bool = True,
-                write_state: bool = True, slot_stride: Optional[int] = None) -> Optional[torch.Tensor]:
+                write_state: bool = True, slot_stride: Optional[int] = None,
+                in_bias: Optional[torch.Tensor] = None, parts: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """A causal convolution over time on columns col0 .. col0 + C - 1 of the sums u [S, n, ld],
     without the input added: act(bias + sum_j w[:, j] u_{t - taps + 1 + j}); w float32 [C, taps];
-    state: float32, per slot a ring [taps - 1, C] of the last inputs (slot_stride floats apart)."""
+    state: float32, per slot a ring [taps - 1, C] of the last inputs (slot_stride floats apart).
+    in_bias [C] is added to the sums first; parts [C / part, n, part] gets the result once more."""
     u = stack(u)
     _need(u, "u", torch.float32, (None, None, None))
     S, n, ld = u.shape
     _need(w, "w", torch.float32, (C, None))
+    if parts is not None and (parts.shape[1] != n or parts.shape[0] * parts.shape[2] != C):
+        raise ValueError("parts must be [C / part, n, part]")
     taps = w.shape[1]
     out = torch.empty((n, C), dtype=out_dtype, device=u.device) if write_out else None
     what = (1 if write_out else 0) | (2 if write_state and taps > 1 else 0)
     stride = slot_stride if slot_stride is not None else (taps - 1) * C
     _check(lib().jb_causal_conv(_p(u), S, n * ld, ld, col0, _p(w), _p(bias), _p(state), stride, _p(row_pos),
                                 _p(row_seq), _p(seq_slot), _p(out), _DT[out_dtype], C, n, C, taps,
-                                1 if silu else 0, what, _stream()), "causal_conv")
+                                1 if silu else 0, what, _p(in_bias), _p(parts), 0 if parts is None else _DT[parts.dtype],
+                                1 if parts is None else parts.shape[2], _stream()), "causal_conv")
+    return out
+
+
+def lru(gates: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor, lam: torch.Tensor, u: torch.Tensor,
+        P: torch.Tensor, y_col0: int, y_bias: Optional[torch.Tensor], state: torch.Tensor, row_seq: torch.Tensor,
+        seq_slot: torch.Tensor, n_seqs: int, out_dtype: torch.dtype, every_row_starts: bool = False,
+        max_len: int = 0, slot_stride: Optional[int] = None) -> torch.Tensor:
+    """The real-gated linear recurrent unit over the rows of each sequence: gates [blocks, S, n, 2 part] the sums of
+    r and i per block of channels, u float32 [n, W], P [S, n, ld] with the other branch's sums from y_col0.  Returns
+    S_t * gelu_tanh(y) [n, W]; state: float32 [slots, W].  max_len: the most rows one sequence brings."""
+    P = stack(P)
+    _need(P, "P", torch.float32, (None, None, None))
+    S, n, ld = P.shape
+    _need(u, "u", torch.float32, (n, None))
+    W = u.shape[1]
+    blocks, gS, gn, two = gates.shape
+    if gates.dtype != torch.float32 or not gates.is_contiguous() or gn != n or blocks * two != 2 * W:
+        raise ValueError("gates must be contiguous float32 [blocks, S, n, 2 W / blocks]")
+    out = torch.empty((n, W), dtype=out_dtype, device=u.device)
+    need = 0 if every_row_starts else lib().jb_lru_scratch(n, n_seqs, max_len, W)
+    scratch = torch.empty((need,), dtype=torch.float32, device=u.device) if need > 0 else None
+    _check(lib().jb_lru(_p(gates), gS, two // 2, _p(r_bias), _p(i_bias), _p(lam), _p(u), _p(P), S, n * ld, ld, y_col0,
+                        _p(y_bias), _p(state), slot_stride if slot_stride is not None else W, _p(row_seq),
+                        _p(seq_slot), _p(scratch), _p(out), _DT[out_dtype], n, n_seqs, W,
+                        1 if every_row_starts else 0, max_len, _stream()), "lru", 3 if need > 0 else 1)
+    return out
+
+
+def gated_memory(src: torch.Tensor, H: int, N: int, P: int, cols: dict, i_bias: torch.Tensor, f_bias: torch.Tensor,
+                 cap: float, q_scale: float, floor: float, w: torch.Tensor, eps: float, state: torch.Tensor,
+                 row_seq: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int, out_dtype: torch.dtype,
+                 every_row_starts: bool = False, max_len: int = 0,
+                 slot_stride: Optional[int] = None) -> torch.Tensor:
+    """The matrix memory with exponential gates and its norm and output gate: [n, H P].  src [S, n, ld]; cols: the
+    first columns of q, k, v, g, i and f.  state: float32, per slot [H, N P + N] and then [H]."""
+    src = stack(src)
+    _need(src, "src", torch.float32, (None, None, None))
+    S, n, ld = src.shape
+    dev = src.device
+    stride = slot_stride if slot_stride is not None else H * (N * P + N + 1)
+    y = torch.empty((n, H * P), dtype=torch.float32, device=dev)
+    nq = torch.empty((n, H), dtype=torch.float32, device=dev)
+    em = scratch = None
+    starts = 1 if every_row_starts else 0
+    if not every_row_starts:
+        em = torch.empty((n, H), dtype=torch.float32, device=dev)
+        scratch = torch.empty((lib().jb_gated_memory_scratch(n, n_seqs, max_len, H, N, P, 0),), dtype=torch.float32,
+                              device=dev)
+    _check(lib().jb_gated_memory_scan(_p(src), S, n * ld, ld, cols["v"], cols["k"], cols["q"], cols["i"], cols["f"],
+                                      _p(i_bias), _p(f_bias), float(cap), float(q_scale), _p(state), stride,
+                                      _p(row_seq), _p(seq_slot), _p(y), _p(nq), _p(em), n, n_seqs, H, N, P, starts,
+                                      _p(scratch), max_len, _stream()), "gated_memory_scan")
+    out = torch.empty((n, H * P), dtype=out_dtype, device=dev)
+    _check(lib().jb_gated_memory_norm(_p(y), _p(nq), _p(em), float(floor), _p(src), S, n * ld, ld, cols["g"], cols["i"],
+                                      cols["f"], _p(i_bias), _p(f_bias), float(cap), _p(state), stride, _p(row_seq),
+                                      _p(seq_slot), _p(w), float(eps), _p(out), _DT[out_dtype], n, H, N, P, _stream()),
+           "gated_memory_norm")
+    return out
+
+
+def spread_streams(e: torch.Tensor, streams: int) -> torch.Tensor:
+    """[n, streams, dm] with every stream equal to e [n, dm]"""
+    _need(e, "e", torch.float32, (None, None))
+    n, dm = e.shape
+    x = torch.empty((n, streams, dm), dtype=torch.float32, device=e.device)
+    _check(lib().jb_spread_streams(_p(e), _p(x), streams, n, dm, _stream()), "spread_streams")
+    return x
+
+
+def streams(x: torch.Tensor, y: Optional[torch.Tensor] = None, ls: Optional[torch.Tensor] = None,
+            out_w: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, mult: float = 1.0,
+            read: bool = True, in_w: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None,
+            b: Optional[torch.Tensor] = None, eps: float = 0.0, rows: Optional[torch.Tensor] = None,
+            out_dtype: torch.dtype = torch.float32, few_rows: bool = False) -> Optional[torch.Tensor]:
+    """x [n, streams, dm] in place: with y [S, n, dm], X_t <- sum_s mix[s, t] X_s + mult out_w[t] (ls * y); with
+    read, the layer norm (w, b, eps; w None: none) of sum_s in_w[s] X_s (in_w None: ones), [n or rows, dm]."""
+    if x.dtype != torch.float32 or x.dim() != 3 or not x.is_contiguous():
+        raise ValueError("x must be contiguous float32 [n, streams, dm]")
+    n, ns, dm = x.shape
+    S = 0
+    if y is not None:
+        y = stack(y)
+        _need(y, "y", torch.float32, (None, n, dm))
+        S = y.shape[0]
+    outs = n if rows is None else rows.shape[0]
+    out = torch.empty((outs, dm), dtype=out_dtype, device=x.device) if read else None
+    _check(lib().jb_streams(_p(x), ns, _p(y), S, n * dm, _p(ls), _p(out_w), _p(mix), float(mult), _p(rows), _p(in_w),
+                            _p(w), _p(b), float(eps), _p(out), _DT[out_dtype], outs, dm, 1 if few_rows else 0,
+                            _stream()), "streams")
     return out
 
 

@@ -2,6 +2,7 @@
 // convolution over time on every channel of the residual stream, and the minGRU's
 // gated running value.  The state lives per slot in float32 and is carried from
 // step to step; everything here is computed in float32.
+// A third, the real-gated linear recurrent unit, is described at its kernels.
 //
 // Rows are the sequences' tokens one sequence after the other; row r belongs to
 // sequence row_seq[r] of the step (slot seq_slot[row_seq[r]]) and stands at position
@@ -11,6 +12,20 @@
 #include "kernels.h"
 
 namespace jb {
+
+// first row r with row_seq[r] >= s
+__device__ __forceinline__ int lower_row(const int32_t *__restrict__ row_seq, int n, int s)
+{
+    int lo = 0, hi = n;
+    while (lo < hi) {
+        int mid = (lo + hi) >> 1;
+        if (row_seq[mid] < s)
+            lo = mid + 1;
+        else
+            hi = mid;
+    }
+    return lo;
+}
 
 // ------------------------------------------------------------ short convolution
 //
@@ -162,14 +177,38 @@ short_conv_rows_kernel(const float *__restrict__ x, const float *__restrict__ w,
 // u = the sums in columns col0 .. col0 + C - 1 of [S, n, ld]; zeros before position 0.
 // State, `what` and the rule for one launch or two are short_conv_kernel's: a ring of the
 // last taps - 1 inputs per slot, [taps - 1, C].  act 1: silu.  out: [n, out_ld] with the
-// result in its first C columns.  One thread per (row, column).
+// result in its first C columns.  in_bias (null: none): added to the sums first; it is part of
+// the inputs that the state keeps.  A second copy of the result may go to `parts`: equal parts of
+// `part` columns each, one part's rows together ([C / part, n, part], 16-bit or float32).
+// One thread per (row, column).
+struct ConvParts {
+    void *out;
+    int dt, part;
+};
+__device__ __forceinline__ void store_part(const ConvParts &q, int n, int r, int c, float v)
+{
+    size_t at = ((size_t)(c / q.part) * n + r) * q.part + c % q.part;
+    if (q.dt == JB_BF16)
+        static_cast<bf16 *>(q.out)[at] = from_f<bf16>(v);
+    else
+        static_cast<float *>(q.out)[at] = v;
+}
+__device__ __forceinline__ void store_part4(const ConvParts &q, int n, int r, int c, float4 v)
+{
+    size_t at = ((size_t)(c / q.part) * n + r) * q.part + c % q.part;
+    if (q.dt == JB_BF16)
+        store4(static_cast<bf16 *>(q.out) + at, v);
+    else
+        store4(static_cast<float *>(q.out) + at, v);
+}
+
 template <typename TO>
 __global__ void __launch_bounds__(256)
 causal_conv_kernel(const float *__restrict__ u, int S, size_t stride, int ld, int col0,
                    const float *__restrict__ w, const float *__restrict__ bias, float *__restrict__ state,
                    size_t slot_stride, const int32_t *__restrict__ row_pos, const int32_t *__restrict__ row_seq,
                    const int32_t *__restrict__ seq_slot, TO *__restrict__ out, int out_ld, int n, int C, int taps,
-                   int act, int what)
+                   int act, int what, const float *__restrict__ in_bias, ConvParts parts)
 {
     pdl_trigger();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -180,7 +219,8 @@ causal_conv_kernel(const float *__restrict__ u, int S, size_t stride, int ld, in
     int keep = taps - 1;
     float *st = state != nullptr ? state + (size_t)seq_slot[seq] * slot_stride : nullptr;
     pdl_wait();
-    float cur = add_partials(0.0f, u + (size_t)r * ld + col0 + c, S, stride);
+    const float ib = in_bias != nullptr ? in_bias[c] : 0.0f;
+    float cur = add_partials(ib, u + (size_t)r * ld + col0 + c, S, stride);
     if (what & 1) {
         float acc = bias != nullptr ? bias[c] : 0.0f;
         acc = fmaf(w[(size_t)c * taps + taps - 1], cur, acc);
@@ -189,13 +229,15 @@ causal_conv_kernel(const float *__restrict__ u, int S, size_t stride, int ld, in
             if (p < 0)
                 break;
             float v = r - k >= 0 && row_seq[r - k] == seq
-                          ? add_partials(0.0f, u + (size_t)(r - k) * ld + col0 + c, S, stride)
+                          ? add_partials(ib, u + (size_t)(r - k) * ld + col0 + c, S, stride)
                           : st[(size_t)(p % keep) * C + c];
             acc = fmaf(w[(size_t)c * taps + taps - 1 - k], v, acc);
         }
         if (act == 1)
             acc = acc / (1.0f + expf(-acc));
         out[(size_t)r * out_ld + c] = from_f<TO>(acc);
+        if (parts.out != nullptr)
+            store_part(parts, n, r, c, acc);
     }
     if ((what & 2) && keep > 0 && (r + keep >= n || row_seq[r + keep] != seq))
         st[(size_t)(pos % keep) * C + c] = cur;
@@ -211,7 +253,7 @@ causal_conv_rows_kernel(const float *__restrict__ u, int ld, int col0, const flo
                         const float *__restrict__ bias, float *__restrict__ state, size_t slot_stride,
                         const int32_t *__restrict__ row_pos, const int32_t *__restrict__ row_seq,
                         const int32_t *__restrict__ seq_slot, TO *__restrict__ out, int out_ld, int n, int C,
-                        int act, int what)
+                        int act, int what, const float *__restrict__ in_bias, ConvParts parts)
 {
     constexpr int KEEP = TAPS - 1;
     pdl_trigger();
@@ -227,6 +269,8 @@ causal_conv_rows_kernel(const float *__restrict__ u, int ld, int col0, const flo
         wt[j] = make_float4(w[(size_t)c * TAPS + j], w[(size_t)(c + 1) * TAPS + j], w[(size_t)(c + 2) * TAPS + j],
                             w[(size_t)(c + 3) * TAPS + j]);
     float4 bs = bias != nullptr ? load4(bias + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 ib = in_bias != nullptr ? load4(in_bias + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    auto plus = [&ib](float4 v) { return make_float4(ib.x + v.x, ib.y + v.y, ib.z + v.z, ib.w + v.w); };
     pdl_wait();
     const float *in = u + col0 + c;
     float4 hist[KEEP];          // hist[k - 1]: the input k positions back
@@ -236,7 +280,7 @@ causal_conv_rows_kernel(const float *__restrict__ u, int ld, int col0, const flo
 #pragma unroll
     for (int q = 0; q < RB; q++) {
         int rr = min(r0 + q, r1 - 1);
-        in_rows[q] = load4(in + (size_t)rr * ld);
+        in_rows[q] = plus(load4(in + (size_t)rr * ld));
         in_pos[q] = row_pos[rr];
         in_seq[q] = row_seq[rr];
     }
@@ -254,7 +298,7 @@ causal_conv_rows_kernel(const float *__restrict__ u, int ld, int col0, const flo
                 if (p < 0)
                     hist[k - 1] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 else if (r - k >= 0 && row_seq[r - k] == seq)
-                    hist[k - 1] = load4(in + (size_t)(r - k) * ld);
+                    hist[k - 1] = plus(load4(in + (size_t)(r - k) * ld));
                 else
                     hist[k - 1] = load4(st + (size_t)(p % KEEP) * C + c);
             }
@@ -283,6 +327,8 @@ causal_conv_rows_kernel(const float *__restrict__ u, int ld, int col0, const flo
                 acc.w = acc.w / (1.0f + expf(-acc.w));
             }
             store4<TO>(out + (size_t)r * out_ld + c, acc);
+            if (parts.out != nullptr)
+                store_part4(parts, n, r, c, acc);
         }
         if ((what & 2) && (r + KEEP >= n || row_seq[r + KEEP] != seq))
             *reinterpret_cast<float4 *>(st + (size_t)(pos % KEEP) * C + c) = cur;
@@ -418,7 +464,7 @@ mingru_pieces_kernel(GruIn in, const float *__restrict__ state, const int32_t *_
 
 // The value each piece starts from: carry [pieces, W], piece after piece.
 __global__ void __launch_bounds__(128)
-mingru_carry_kernel(const float *__restrict__ AB, float *__restrict__ carry, int W, int pieces)
+mingru_carry_kernel(const float *AB, float *__restrict__ carry, int W, int pieces)
 {
     pdl_trigger();
     int ch = blockIdx.x * blockDim.x + threadIdx.x;
@@ -440,8 +486,8 @@ mingru_carry_kernel(const float *__restrict__ AB, float *__restrict__ carry, int
 template <typename TO, int GRU_U>
 __global__ void __launch_bounds__(128)
 mingru_scan_kernel(GruIn in, float *__restrict__ state, const int32_t *__restrict__ row_seq,
-                   const int32_t *__restrict__ seq_slot, const float *__restrict__ carry,
-                   const float *__restrict__ init, TO *__restrict__ out, int n, int piece)
+                   const int32_t *__restrict__ seq_slot, const float *carry,
+                   const float *init, TO *__restrict__ out, int n, int piece)
 {
     constexpr bool FAST = sizeof(TO) == 2;
     pdl_trigger();
@@ -496,9 +542,210 @@ mingru_scan_kernel(GruIn in, float *__restrict__ state, const int32_t *__restric
     }
 }
 
+// ---------------------------------------------------------- gated linear unit
+//
+//   r = sigmoid(G_r + rb);  i = sigmoid(G_i + ib);  log a = -8 r softplus(lam)
+//   S_t = a S_{t-1} + sqrt(1 - a^2) i u_t;   out_t = S_t * gelu_tanh(P_y + yb)
+//
+// channel by channel (the real-gated linear recurrent unit).  G: the sums of one product per block of `part`
+// channels, [blocks, S, n, 2 part] with r's columns and then i's.  u: float32 [n, W].  P: sums whose
+// columns from y_col0 are the other branch.  state: float32 [W] per slot, slot_stride apart.
+struct LruIn {
+    const float *G;
+    int gS, part;
+    const float *rb, *ib, *lam, *u, *P;
+    int S;
+    size_t stride;
+    int ld, y_col0;
+    const float *yb;
+    int n, W;
+};
+
+template <bool FAST> __device__ __forceinline__ float gelu_tanh_(float v)
+{
+    float t = 0.7978845608028654f * fmaf(0.044715f * v * v, v, v);
+    // tanh(t) = 1 - 2 / (1 + e^(2t)); the hardware's exponential where the result is rounded to 16 bits
+    float th = FAST ? 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * fminf(t, 40.0f))) : tanhf(t);
+    return 0.5f * v * (1.0f + th);
+}
+
+// a and b = sqrt(1 - a^2) i u of row r's channel ch; c = -8 softplus(lam), all in float32
+__device__ __forceinline__ void lru_coef(const LruIn &in, int r, int ch, float c, float rb, float ib, float &a, float &b)
+{
+    int blk = ch / in.part, j = ch - blk * in.part;
+    const float *g = in.G + ((size_t)blk * in.gS * in.n + r) * 2 * in.part + j;
+    size_t gs = (size_t)in.n * 2 * in.part;
+    float rg = sigmoidf_<false>(add_partials(rb, g, in.gS, gs));
+    float ig = sigmoidf_<false>(add_partials(ib, g + in.part, in.gS, gs));
+    float la = c * rg;
+    a = expf(la);
+    b = sqrtf(-expm1f(2.0f * la)) * ig * in.u[(size_t)r * in.W + ch];
+}
+
+// One thread per channel of a sequence's rows, or of a piece of `piece` of them (a sequence with
+// fewer than two pieces' rows stays whole, so that its bits do not depend on what else the step holds):
+// MODE 0: from the slot's state through all the rows; out and the state are written.
+// MODE 1: a piece from zero: every row's a and b go to coef [2, n, W], the piece's map S -> A S + B to AB.
+// MODE 2: a piece from carry, with a and b from coef; out and, with a sequence's last piece, the state.
+// blockIdx.y: the piece, blockIdx.z: the sequence.  U rows' loads go out together.
+// (What the kernel before this one writes is not a const __restrict__ argument: the compiler may fetch
+// such values through the read-only path ahead of pdl_wait.)
+template <typename TO, int MODE, int U>
+__global__ void __launch_bounds__(128)
+lru_kernel(LruIn in, float *__restrict__ state, size_t slot_stride, const int32_t *__restrict__ row_seq,
+           const int32_t *__restrict__ seq_slot, float *__restrict__ coef, float *__restrict__ AB,
+           const float *carry, TO *__restrict__ out, int every_row_starts, int piece)
+{
+    constexpr bool FAST = sizeof(TO) == 2;
+    pdl_trigger();
+    int ch = blockIdx.x * blockDim.x + threadIdx.x, pc = blockIdx.y, seq = blockIdx.z;
+    int r0 = seq, r1 = seq + 1;
+    if (!every_row_starts) {
+        r0 = lower_row(row_seq, in.n, seq);
+        r1 = lower_row(row_seq, in.n, seq + 1);
+    }
+    const int end = r1;
+    if (MODE != 0) {
+        if (r1 - r0 >= 2 * piece) {
+            r0 += pc * piece;
+            r1 = min(r1, r0 + piece);
+        } else if (pc > 0) {
+            return;
+        }
+    }
+    if (ch >= in.W || r0 >= r1)
+        return;
+    const float rb = in.rb[ch], ib = in.ib[ch], lam = in.lam[ch], yb = in.yb != nullptr ? in.yb[ch] : 0.0f;
+    const float c = -8.0f * (fmaxf(lam, 0.0f) + log1pf(expf(-fabsf(lam))));
+    const size_t cw = (size_t)in.n * in.W, z = (size_t)seq * gridDim.y + pc;
+    pdl_wait();
+    float *st = state + (size_t)seq_slot[seq] * slot_stride + ch;
+    float s = MODE == 0 ? *st : MODE == 1 ? 0.0f : carry[z * in.W + ch];
+    float A = 1.0f;
+    for (int rr = r0; rr < r1; rr += U) {
+        float a[U], b[U], g[U];
+#pragma unroll
+        for (int k = 0; k < U; k++) {
+            int r = min(rr + k, r1 - 1);
+            if (MODE == 2) {
+                a[k] = coef[(size_t)r * in.W + ch];
+                b[k] = coef[cw + (size_t)r * in.W + ch];
+            } else {
+                lru_coef(in, r, ch, c, rb, ib, a[k], b[k]);
+            }
+            if (MODE != 1)
+                g[k] = add_partials(yb, in.P + (size_t)r * in.ld + in.y_col0 + ch, in.S, in.stride);
+        }
+#pragma unroll
+        for (int k = 0; k < U; k++)
+            if (rr + k < r1) {
+                size_t at = (size_t)(rr + k) * in.W + ch;
+                s = fmaf(a[k], s, b[k]);
+                if (MODE == 1) {
+                    A *= a[k];
+                    coef[at] = a[k];
+                    coef[cw + at] = b[k];
+                } else {
+                    out[at] = from_f<TO>(s * gelu_tanh_<FAST>(g[k]));
+                }
+            }
+    }
+    if (MODE == 1) {
+        AB[(z * 2) * in.W + ch] = A;
+        AB[(z * 2 + 1) * in.W + ch] = s;
+    } else if (r1 == end) {
+        *st = s;
+    }
+}
+
+// The value each piece starts from, sequence by sequence: carry [sequences, pieces, W].
+__global__ void __launch_bounds__(128)
+lru_carry_kernel(const float *state, size_t slot_stride, const int32_t *__restrict__ row_seq,
+                 const int32_t *__restrict__ seq_slot, const float *AB, float *carry, int n,
+                 int W, int piece, int pieces)
+{
+    pdl_trigger();
+    int ch = blockIdx.x * blockDim.x + threadIdx.x, seq = blockIdx.y;
+    int rows = lower_row(row_seq, n, seq + 1) - lower_row(row_seq, n, seq);
+    if (ch >= W || rows <= 0)
+        return;
+    int used = rows >= 2 * piece ? (rows + piece - 1) / piece : 1;
+    pdl_wait();
+    float s = state[(size_t)seq_slot[seq] * slot_stride + ch];
+    for (int c0 = 0; c0 < used; c0 += 8) {
+        float A[8], B[8];
+#pragma unroll
+        for (int u = 0; u < 8; u++) {
+            size_t z = (size_t)seq * pieces + min(c0 + u, used - 1);
+            A[u] = AB[(z * 2) * W + ch];
+            B[u] = AB[(z * 2 + 1) * W + ch];
+        }
+#pragma unroll
+        for (int u = 0; u < 8; u++)
+            if (c0 + u < used) {
+                carry[((size_t)seq * pieces + c0 + u) * W + ch] = s;
+                s = fmaf(A[u], s, B[u]);
+            }
+    }
+}
+
 }  // namespace jb
 
 using namespace jb;
+
+// rows to a piece when long sequences are cut into pieces that run side by side
+extern "C" int jb_lru_piece(void) { return 32; }
+// Floats of scratch for a step whose longest sequence brings max_len of the n rows (0: one pass).
+extern "C" long long jb_lru_scratch(int n, int n_seqs, int max_len, int W)
+{
+    int piece = jb_lru_piece();
+    if (max_len < 2 * piece)
+        return 0;
+    long long pieces = (max_len + piece - 1) / piece;
+    return 2ll * n * W + 3ll * n_seqs * pieces * W;
+}
+
+// G: float32 [W / part, gS, n, 2 part]; rb, ib, lam [W]; u: float32 [n, W]; P: float32 [S, n, ld]; yb [W] or
+// null.  out: [n, W] in out_dt.  scratch: jb_lru_scratch floats, or null for one pass.
+extern "C" int jb_lru(const float *G, int gS, int part, const float *rb, const float *ib, const float *lam,
+                      const float *u, const float *P, int S, long long stride, int ld, int y_col0, const float *yb,
+                      float *state, long long slot_stride, const int32_t *row_seq, const int32_t *seq_slot,
+                      float *scratch, void *out, int out_dt, int n, int n_seqs, int W, int every_row_starts,
+                      int max_len, cudaStream_t st)
+{
+    if (n <= 0 || n_seqs <= 0)
+        return JB_OK;
+    if (W <= 0 || part <= 0 || W % part || gS <= 0 || S <= 0 || G == nullptr || rb == nullptr || ib == nullptr ||
+        lam == nullptr || u == nullptr || P == nullptr || state == nullptr || out == nullptr || y_col0 < 0 ||
+        ld < y_col0 + W || n_seqs > 65535 || (out_dt != JB_F32 && out_dt != JB_BF16))
+        return JB_EINVAL;
+    LruIn in{G, gS, part, rb, ib, lam, u, P, S, (size_t)stride, ld, y_col0, yb, n, W};
+    unsigned gx = (unsigned)((W + 127) / 128);
+    int piece = jb_lru_piece();
+    bool whole = scratch == nullptr || every_row_starts || max_len < 2 * piece;
+    int pieces = whole ? 1 : (max_len + piece - 1) / piece;
+    if (pieces > 65535)
+        return JB_EINVAL;
+    float *coef = scratch, *AB = whole ? nullptr : scratch + 2ll * n * W, *carry = whole ? nullptr : AB + 2ll * n_seqs * pieces * W;
+    dim3 grid(gx, (unsigned)pieces, (unsigned)n_seqs);
+#define JB_LRU(TO, MODE, U)                                                                                \
+    launch(lru_kernel<TO, MODE, U>, grid, 128, 0, st, in, state, (size_t)slot_stride, row_seq, seq_slot, coef, AB, \
+           (const float *)carry, (TO *)out, every_row_starts, piece)
+    if (whole) {
+        if (every_row_starts) {
+            if (out_dt == JB_F32) JB_LRU(float, 0, 1); else JB_LRU(bf16, 0, 1);
+        } else {
+            if (out_dt == JB_F32) JB_LRU(float, 0, 4); else JB_LRU(bf16, 0, 4);
+        }
+        return launch_status();
+    }
+    if (out_dt == JB_F32) JB_LRU(float, 1, 4); else JB_LRU(bf16, 1, 4);
+    launch(lru_carry_kernel, dim3(gx, (unsigned)n_seqs), 128, 0, st, (const float *)state, (size_t)slot_stride, row_seq,
+           seq_slot, (const float *)AB, carry, n, W, piece, pieces);
+    if (out_dt == JB_F32) JB_LRU(float, 2, 8); else JB_LRU(bf16, 2, 8);
+#undef JB_LRU
+    return launch_status();
+}
 
 // what: 1 = write h, 2 = write the state, 3 = both (see short_conv_kernel for when).
 // state may be null with taps == 1.
@@ -556,20 +803,26 @@ extern "C" int jb_short_conv(const float *x, const float *w, float *state, long 
 }
 
 // u: float32 [S, n, ld]; w: float32 [C, taps]; bias: float32 [C] or null; state: float32
-// [taps - 1, C] per slot (null with taps == 1).  out: [n, out_ld] in out_dt.
+// [taps - 1, C] per slot (null with taps == 1).  out: [n, out_ld] in out_dt.  in_bias: float32 [C]
+// or null; parts (or null): the result once more as [C / part, n, part] in parts_dt.
 extern "C" int jb_causal_conv(const float *u, int S, long long stride, int ld, int col0, const float *w,
                               const float *bias, float *state, long long slot_stride, const int32_t *row_pos,
                               const int32_t *row_seq, const int32_t *seq_slot, void *out, int out_dt, int out_ld,
-                              int n, int C, int taps, int act, int what, cudaStream_t st)
+                              int n, int C, int taps, int act, int what, const float *in_bias, void *parts,
+                              int parts_dt, int part, cudaStream_t st)
 {
     if (n <= 0 || C <= 0 || !(what & 3))
         return JB_OK;
     if (taps < 1 || S <= 0 || ld < col0 + C || col0 < 0 || out_ld < C || u == nullptr || w == nullptr ||
         (taps > 1 && state == nullptr) || ((what & 1) && out == nullptr) || (act != 0 && act != 1))
         return JB_EINVAL;
+    if (parts != nullptr && (part <= 0 || C % part || (parts_dt != JB_F32 && parts_dt != JB_BF16)))
+        return JB_EINVAL;
+    ConvParts cp{parts, parts_dt, part};
     auto al16 = [](const void *p) { return ((uintptr_t)p & 15) == 0; };
     if (S == 1 && taps >= 2 && taps <= 4 && C % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && out_ld % 4 == 0 &&
-        slot_stride % 4 == 0 && al16(u) && al16(bias) && al16(state) && al16(out)) {
+        slot_stride % 4 == 0 && al16(u) && al16(bias) && al16(state) && al16(out) && al16(in_bias) &&
+        (parts == nullptr || (part % 4 == 0 && al16(parts)))) {
         // many rows: eight to a thread; few: one (a decode step's rows are all of other sequences)
         bool many = (size_t)n * (C / 4) >= (size_t)8 * 148 * 1024;
         int rbs = many ? 8 : 1;
@@ -577,7 +830,7 @@ extern "C" int jb_causal_conv(const float *u, int S, long long stride, int ld, i
         unsigned g = (unsigned)((threads + 255) / 256);
 #define JB_CCR(TO, T, RB)                                                                                  \
     launch(causal_conv_rows_kernel<TO, T, RB>, g, 256, 0, st, u, ld, col0, w, bias, state, (size_t)slot_stride, \
-           row_pos, row_seq, seq_slot, (TO *)out, out_ld, n, C, act, what)
+           row_pos, row_seq, seq_slot, (TO *)out, out_ld, n, C, act, what, in_bias, cp)
 #define JB_CCR_T(TO, RB)                                                                                   \
     do {                                                                                                   \
         if (taps == 2) JB_CCR(TO, 2, RB);                                                                  \
@@ -598,10 +851,10 @@ extern "C" int jb_causal_conv(const float *u, int S, long long stride, int ld, i
     unsigned grid = (unsigned)(((size_t)n * C + 255) / 256);
     if (out_dt == JB_F32)
         launch(causal_conv_kernel<float>, grid, 256, 0, st, u, S, (size_t)stride, ld, col0, w, bias, state,
-               (size_t)slot_stride, row_pos, row_seq, seq_slot, (float *)out, out_ld, n, C, taps, act, what);
+               (size_t)slot_stride, row_pos, row_seq, seq_slot, (float *)out, out_ld, n, C, taps, act, what, in_bias, cp);
     else if (out_dt == JB_BF16)
         launch(causal_conv_kernel<bf16>, grid, 256, 0, st, u, S, (size_t)stride, ld, col0, w, bias, state,
-               (size_t)slot_stride, row_pos, row_seq, seq_slot, (bf16 *)out, out_ld, n, C, taps, act, what);
+               (size_t)slot_stride, row_pos, row_seq, seq_slot, (bf16 *)out, out_ld, n, C, taps, act, what, in_bias, cp);
     else
         return JB_EINVAL;
     return launch_status();

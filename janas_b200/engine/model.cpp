@@ -8,6 +8,10 @@ DecoderModel::DecoderModel(const ModelSpec &s, DType dt, Device *d) : spec(s), d
     spec.validate();
     if (dt != F32 && dt != BF16) fail(JB_LLM_EINVAL, "the compute dtype is float32 or bfloat16");
     for (auto &ls : spec.layers) blocks.push_back(build_block(ls, dt, d));
+    for (auto &b : blocks)
+        if (b->streams() != spec.streams)
+            config_error(fmt("a layer's arrangement works on %lld streams, the model's residual stream has %lld "
+                             "(0: it is one)", b->streams(), spec.streams));
     final_norm = build_norm(spec.final_norm, dt, d);
     if (final_norm->size() != spec.hidden_size)
         config_error("the final norm's size is not the model's hidden size");
@@ -224,6 +228,8 @@ Buf DecoderModel::forward(StepContext &ctx, const int32_t *tokens, std::vector<L
     ctx.normed.reset();
     ctx.normed_by = nullptr;
     if (embedding_norm) x = embedding_norm->apply(ctx, x.as<float>(), n, F32, nullptr, nullptr, 0);
+    const int ns = (int)spec.streams;
+    if (ns > 0) x = ops::spread_streams(d, x.as<float>(), ns, n, spec.hidden_size);
     // the embedding output, kept for the entries that add it once more or join it
     Stack again;
     for (auto &e : spec.run_order)
@@ -257,14 +263,19 @@ Buf DecoderModel::forward(StepContext &ctx, const int32_t *tokens, std::vector<L
         b.next_norm = e + 1 < spec.run_order.size() && !spec.run_order[e + 1].add_embedding &&
                               !spec.run_order[e + 1].join_embedding
                           ? blocks[(size_t)spec.run_order[e + 1].layer]->mixer_norm.get() : nullptr;
+        b.next_block = e + 1 < spec.run_order.size() ? blocks[(size_t)spec.run_order[e + 1].layer].get() : nullptr;
         b.forward(ctx, x.as<float>(), pending, caches[e]);
         if (ctx.trace) {
+            Buf sum;
+            ops::StreamRead all_once;
+            if (ns > 0)
+                sum = ops::streams(d, x.as<float>(), ns, n, spec.hidden_size, nullptr, nullptr, &all_once, F32, nullptr, 0, false);
             if (pending) {
                 ops::add_(d, x.as<float>(), n, spec.hidden_size, pending);
                 pending = Stack();
             }
             std::vector<float> host((size_t)n * (size_t)spec.hidden_size);
-            cuda_check(cudaMemcpyAsync(host.data(), x.ptr, host.size() * 4, cudaMemcpyDeviceToHost, d.stream),
+            cuda_check(cudaMemcpyAsync(host.data(), ns > 0 ? sum.ptr : x.ptr, host.size() * 4, cudaMemcpyDeviceToHost, d.stream),
                        "copying the residual stream");
             d.sync();
             ctx.trace->push_back(std::move(host));
@@ -272,8 +283,21 @@ Buf DecoderModel::forward(StepContext &ctx, const int32_t *tokens, std::vector<L
     }
     if (n_want == 0) return Buf();
     bool all = n_want < 0;
-    Buf h = final_norm->apply(ctx, x.as<float>(), n, ctx.dtype, pending ? &pending : nullptr,
+    Buf h;
+    ops::StreamRead last;
+    bool rms = false;
+    if (ns > 0 && final_norm->layer_norm(&last.norm, &rms) && !rms) {
+        // the sum of the streams and the last norm in one pass, of the wanted rows alone
+        h = ops::streams(d, x.as<float>(), ns, n, spec.hidden_size, nullptr, nullptr, &last, ctx.dtype,
+                         all ? nullptr : want_rows, all ? 0 : n_want, ctx.dtype == BF16);
+    } else {
+        if (ns > 0) {
+            last.norm = ops::LnParams();
+            x = ops::streams(d, x.as<float>(), ns, n, spec.hidden_size, nullptr, nullptr, &last, F32, nullptr, 0, false);
+        }
+        h = final_norm->apply(ctx, x.as<float>(), n, ctx.dtype, pending ? &pending : nullptr,
                               all ? nullptr : want_rows, all ? 0 : n_want);
+    }
     Stack lg = ops::linear(d, h.ptr, ctx.dtype, all ? n : n_want, spec.hidden_size, head, true);
     if (spec.logit_scale != 1.0)
         ops::scale_(d, lg.data(), (all ? n : n_want) * spec.vocab_size, (float)spec.logit_scale);

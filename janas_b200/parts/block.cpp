@@ -18,6 +18,11 @@
 //     h = x + conv(x);  x += norm(sublayer(h))          conv(x)_t = sum_j w[:, j] x_{t - taps + 1 + j}
 // for the mixer and then, where the layer has one, for the feed-forward.  The last
 // taps - 1 inputs of either convolution are state of the sequence (float32, per slot).
+//
+// streams: the residual stream is several streams X_1 .. X_s per row (hyper-connections); each
+// sublayer reads a weighted sum of them through its norm and all are mixed as its result joins:
+//     y = ls * sublayer(norm(sum_s in[s] X_s));   X_t <- sum_s mix[s, t] X_s + m out[t] y
+// for the mixer and then, where the layer has one, for the feed-forward, with weights of their own.
 #include "part.h"
 
 namespace jb {
@@ -418,9 +423,136 @@ private:
     DevTensor conv_[2];
 };
 
+// block_params: hidden_size, streams, residual_mult (m, default 1), mixer_streams / ffn_streams: the
+// prefixes (below the layer's) of the weights in [s], out [s] and mix [s, s] (indexed [from, to]),
+// mixer_scale / ffn_scale (optional): the tensor names of the vectors ls [hidden]; fuse (default true):
+// false runs every norm's read as a launch of its own; unused as in sandwich.
+// A sublayer's result joins the streams in the launch that also reads them for the next sublayer (the
+// next layer's first norm included): the streams go through memory once per sublayer.
+class StreamsBlock : public Block {
+public:
+    StreamsBlock(BlockParts p, const LayerSpec &ls, Device *d) : Block(std::move(p)), dev_(d) {
+        if (!mixer_norm || (feed_forward && !ffn_norm)) config_error("streams: every sublayer needs its norm");
+        if (post_mixer_norm || post_ffn_norm) config_error("streams: the arrangement has no norms on results");
+        PartSpec bp{"streams", ls.block_params};
+        hidden_ = bp.get_int("hidden_size", mixer_norm->size());
+        ns_ = bp.get_int("streams");
+        if (ns_ <= 0 || ns_ > ops::max_streams()) config_error(fmt("streams: 1 to %d streams", ops::max_streams()));
+        mult_ = bp.has("residual_mult") ? (float)bp.get_double("residual_mult") : 1.0f;
+        auto word = [&](const char *key, const char *dflt) {
+            return bp.params.get(key).is_string() ? bp.params.get(key).as_string() : std::string(dflt);
+        };
+        n_hc_[0] = word("mixer_streams", "mixer_streams");
+        n_hc_[1] = word("ffn_streams", "ffn_streams");
+        n_ls_[0] = word("mixer_scale", "");
+        n_ls_[1] = word("ffn_scale", "");
+        if (bp.params.get("fuse").is_bool()) fuse_ = bp.params.get("fuse").as_bool();
+        n_sub_ = feed_forward ? 2 : 1;
+        if (!feed_forward)
+            for (auto &v : bp.params.get("unused").items())
+                if (v.is_object() && v.get("name").is_string()) {
+                    std::vector<long long> shape;
+                    for (auto &s : v.get("shape").items()) shape.push_back(s.as_int());
+                    unused_.emplace_back(v.get("name").as_string(), shape);
+                }
+    }
+
+    void tensors(const std::string &prefix, TensorList &out) const override {
+        for (int i = 0; i < n_sub_; i++) {
+            std::string hc = Part::name(prefix, n_hc_[i]);
+            out.emplace_back(Part::name(hc, "in"), TensorSpec{{ns_}, PARAM, false, 0.5f, 0.2f});
+            out.emplace_back(Part::name(hc, "out"), TensorSpec{{ns_}, PARAM, false, 1.0f, 0.2f});
+            out.emplace_back(Part::name(hc, "mix"), TensorSpec{{ns_, ns_}, PARAM, false, 0.25f, 0.1f});
+            if (!n_ls_[i].empty())
+                out.emplace_back(Part::name(prefix, n_ls_[i]), TensorSpec{{hidden_}, PARAM, false, 1.0f, 0.1f});
+        }
+        for (auto &u : unused_)
+            out.emplace_back(Part::name(prefix, u.first), TensorSpec{u.second, PARAM, true});
+    }
+
+    void load(const std::string &prefix, TensorMap &t) override {
+        for (int i = 0; i < n_sub_; i++) {
+            std::string hc = Part::name(prefix, n_hc_[i]);
+            in_[i] = Part::take(t, Part::name(hc, "in"));
+            out_[i] = Part::take(t, Part::name(hc, "out"));
+            mix_[i] = Part::take(t, Part::name(hc, "mix"));
+            if (!n_ls_[i].empty()) scale_[i] = Part::take(t, Part::name(prefix, n_ls_[i]));
+        }
+        for (auto &u : unused_) t.erase(Part::name(prefix, u.first));
+    }
+
+    size_t weight_bytes() const override {
+        size_t total = 0;
+        for (int i = 0; i < 2; i++) total += in_[i].bytes() + out_[i].bytes() + mix_[i].bytes() + scale_[i].bytes();
+        return total;
+    }
+
+    long long streams() const override { return ns_; }
+    const float *first_read() const override { return (const float *)in_[0].ptr; }
+
+    void forward(StepContext &ctx, float *x, Stack &pending, LayerCache &cache) override {
+        if (pending) fail(JB_LLM_EFAIL, "streams: a sum waits for a residual stream that is one stream");
+        Buf h;
+        if (ctx.normed && ctx.normed_by == mixer_norm.get()) h = std::move(ctx.normed);
+        ctx.normed.reset();
+        ctx.normed_by = nullptr;
+        if (!h) h = read(ctx, x, in_[0], mixer_norm.get());
+        Stack y = mixer->forward(ctx, h.ptr, cache);
+        if (feed_forward) {
+            h = write(ctx, x, y, 0, (const float *)in_[1].ptr, ffn_norm.get());
+            if (!h) h = read(ctx, x, in_[1], ffn_norm.get());
+            y = feed_forward->forward(ctx, h.ptr);
+        }
+        const float *next_in = next_block && next_block->streams() == ns_ ? next_block->first_read() : nullptr;
+        ctx.normed = write(ctx, x, y, n_sub_ - 1, next_in, next_in ? const_cast<Norm *>(next_norm) : nullptr);
+        ctx.normed_by = ctx.normed ? next_norm : nullptr;
+    }
+
+private:
+    bool few(const StepContext &ctx) const { return ctx.kind == DECODE && ctx.dtype == BF16; }
+
+    Buf read(StepContext &ctx, float *x, const DevTensor &in, Norm *norm) {
+        ops::StreamRead r;
+        bool rms = false;
+        r.in = (const float *)in.ptr;
+        if (norm->layer_norm(&r.norm, &rms) && !rms)
+            return ops::streams(*dev_, x, (int)ns_, ctx.n_rows, hidden_, nullptr, nullptr, &r, ctx.dtype, nullptr, 0, few(ctx));
+        r.norm = ops::LnParams();
+        Buf u = ops::streams(*dev_, x, (int)ns_, ctx.n_rows, hidden_, nullptr, nullptr, &r, F32, nullptr, 0, false);
+        return norm->apply(ctx, u.as<float>(), ctx.n_rows, ctx.dtype, nullptr, nullptr, 0);
+    }
+
+    // the result of sublayer `which` joins the streams; with a layer norm to come, its read in the same
+    // launch (otherwise an empty handle)
+    Buf write(StepContext &ctx, float *x, Stack &y, int which, const float *next_in, Norm *next) {
+        ops::StreamWrite w;
+        w.ls = scale_[which] ? (const float *)scale_[which].ptr : nullptr;
+        w.out = (const float *)out_[which].ptr;
+        w.mix = (const float *)mix_[which].ptr;
+        w.mult = mult_;
+        ops::StreamRead r;
+        bool rms = false, fused = fuse_ && next && next->layer_norm(&r.norm, &rms) && !rms;
+        r.in = next_in;
+        return ops::streams(*dev_, x, (int)ns_, ctx.n_rows, hidden_, &y, &w, fused ? &r : nullptr, ctx.dtype, nullptr, 0,
+                            few(ctx));
+    }
+
+    Device *dev_;
+    long long hidden_ = 0, ns_ = 1;
+    float mult_ = 1.0f;
+    bool fuse_ = true;
+    int n_sub_ = 1;
+    std::string n_hc_[2], n_ls_[2];
+    DevTensor in_[2], out_[2], mix_[2], scale_[2];
+    std::vector<std::pair<std::string, std::vector<long long>>> unused_;
+};
+
 }  // namespace
 
 void register_builtin_blocks() {
+    register_block("streams", [](BlockParts p, const LayerSpec &ls, DType, Device *d) {
+        return std::unique_ptr<Block>(new StreamsBlock(std::move(p), ls, d));
+    });
     register_block("result_norm", [](BlockParts p, const LayerSpec &ls, DType, Device *) {
         return std::unique_ptr<Block>(new ResultNormBlock(std::move(p), ls));
     });

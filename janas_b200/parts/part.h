@@ -240,6 +240,12 @@ public:
     // compute it together with its own last step and leave the result in
     // ctx.normed.  Set by the model before each forward.
     const Norm *next_norm = nullptr;
+    // The layer that runs next, or null; set by the model as next_norm is.
+    const Block *next_block = nullptr;
+    // How many streams the residual stream must have for this arrangement (0: it is one stream
+    // [n, hidden]), and the weights [streams] on the device with which its first norm reads them.
+    virtual long long streams() const { return 0; }
+    virtual const float *first_read() const { return nullptr; }
     // x: the float32 residual stream [n, hidden], updated in place; pending: a
     // stack of partial sums not yet added to x (empty for none), replaced by what
     // this layer leaves to be added.

@@ -1,5 +1,5 @@
 // Mixers whose memory of the sequence is a state of fixed size (no keys and values):
-// mingru, mamba2 and decay_attention (the last two are described at their classes).
+// mingru, mamba2, decay_attention, mlstm and rglru (the last four are described at their classes).
 //
 // mingru: a gated running value whose gates read the current token alone,
 //
@@ -13,6 +13,7 @@
 // from step to step, so prompts in portions, decoding and batches of unequal rows all
 // run the same kernels (csrc/recurrent.cu).
 #include <algorithm>
+#include <cmath>
 
 #include "part.h"
 
@@ -423,9 +424,285 @@ private:
     long long col0_ = 0;
 };
 
+// Matrix memory with exponential gates, mLSTM ("xLSTM: Extended Long Short-Term Memory"): H heads, D query/key
+// values and Dv values a head, with c(z) = cap tanh(z / cap):
+//
+//   q = Wq h D^(-1/2), k = Wk h, v = Wv h;   i = c(Wi h + bi), f = log sigmoid(c(Wf h + bf))   one each per head
+//   m_t = max(f + m_{t-1}, i), from 0;   a = e^(f + m_{t-1} - m_t), b = e^(i - m_t)
+//   S_t = a S_{t-1} + b k_t v_t^T;   n_t = a n_{t-1} + b k_t
+//   o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + floor)
+//   out = Wo (concat_heads(rms(o)) w * sigmoid(Wg h))
+//
+// q, k, v, the output gate and the two log gates are one product over h; the gates, the state
+// [per head S | n, then all heads' m], the division and the norm are float32 in both compute types.
+//
+// params: hidden_size, heads, head_dim (D), v_head_dim (Dv, default D), gate_cap, eps, floor (default 1e-6),
+// names (optional): q, k, v, g, i, f, bias (a suffix of i and f), o, norm
+class MatrixLSTM : public Mixer {
+public:
+    MatrixLSTM(const PartSpec &s, DType dt, Device *d) : Mixer(s, dt, d) {
+        hidden_ = s.get_int("hidden_size");
+        H_ = s.get_int("heads");
+        D_ = s.get_int("head_dim");
+        Dv_ = s.get_int("v_head_dim", D_);
+        eps_ = (float)s.get_double("eps");
+        cap_ = (float)s.get_double("gate_cap");
+        floor_ = s.has("floor") ? (float)s.get_double("floor") : 1e-6f;
+        if (hidden_ <= 0 || H_ <= 0 || D_ <= 0 || Dv_ <= 0) config_error("mlstm: sizes must be positive");
+        if (D_ > 1024) config_error("mlstm: the recurrence's kernel takes heads of up to 1024 query values");
+        if (!(cap_ > 0.0f)) config_error("mlstm: gate_cap must be positive");
+        const Json &nm = s.params.get("names");
+        auto leaf = [&](const char *key, const char *dflt) {
+            return nm.is_object() && nm.get(key).is_string() ? nm.get(key).as_string() : std::string(dflt);
+        };
+        n_q_ = leaf("q", "q_proj.weight");
+        n_k_ = leaf("k", "k_proj.weight");
+        n_v_ = leaf("v", "v_proj.weight");
+        n_g_ = leaf("g", "g_proj.weight");
+        n_i_ = leaf("i", "i_proj");
+        n_f_ = leaf("f", "f_proj");
+        n_bias_ = leaf("bias", ".bias");
+        n_o_ = leaf("o", "o_proj.weight");
+        n_norm_ = leaf("norm", "norm.weight");
+        i_col_ = 2 * H_ * D_ + 2 * H_ * Dv_;
+    }
+
+    void tensors(const std::string &p, TensorList &out) const override {
+        out.emplace_back(name(p, n_q_), TensorSpec{{H_ * D_, hidden_}, MATRIX, false});
+        out.emplace_back(name(p, n_k_), TensorSpec{{H_ * D_, hidden_}, MATRIX, false});
+        out.emplace_back(name(p, n_v_), TensorSpec{{H_ * Dv_, hidden_}, MATRIX, false});
+        out.emplace_back(name(p, n_g_), TensorSpec{{H_ * Dv_, hidden_}, MATRIX, false});
+        out.emplace_back(name(p, n_i_), TensorSpec{{H_, hidden_}, MATRIX, false});
+        out.emplace_back(name(p, n_f_), TensorSpec{{H_, hidden_}, MATRIX, false});
+        out.emplace_back(name(p, n_i_ + n_bias_), TensorSpec{{H_}, PARAM, false, 0.0f, 0.5f});
+        out.emplace_back(name(p, n_f_ + n_bias_), TensorSpec{{H_}, PARAM, false, 3.0f, 1.0f});
+        out.emplace_back(name(p, n_o_), TensorSpec{{hidden_, H_ * Dv_}, MATRIX, false});
+        out.emplace_back(name(p, n_norm_), TensorSpec{{H_ * Dv_}, PARAM, false, 1.0f, 0.1f});
+    }
+
+    void load(const std::string &p, TensorMap &t) override {
+        std::vector<DevTensor> in;
+        for (const std::string *nm : {&n_q_, &n_k_, &n_v_, &n_g_, &n_i_, &n_f_}) in.push_back(take(t, name(p, *nm)));
+        // rows of sums four to a load
+        long long rows = i_col_ + 2 * H_;
+        if (rows % 8) in.push_back(dev->tensor(in[0].dt, {8 - rows % 8, hidden_}, true));
+        w_in_ = fuse_rows(*dev, in);
+        i_bias_ = take(t, name(p, n_i_ + n_bias_));
+        f_bias_ = take(t, name(p, n_f_ + n_bias_));
+        w_o_ = take(t, name(p, n_o_));
+        norm_ = take(t, name(p, n_norm_));
+    }
+
+    size_t weight_bytes() const override {
+        return w_in_.bytes() + w_o_.bytes() + norm_.bytes() + i_bias_.bytes() + f_bias_.bytes();
+    }
+
+    DevTensor *first_matrix() override { return w_in_ ? &w_in_ : nullptr; }
+    void share_first_product(long long col0) override {
+        shared_ = true;
+        col0_ = col0;
+    }
+
+    StateSpec state_spec() const override { return StateSpec{{H_ * (D_ * Dv_ + D_ + 1)}, F32}; }
+    bool strided_state() const override { return true; }
+    bool graph_safe() const override { return true; }
+
+    Stack forward(StepContext &ctx, const void *h, LayerCache &cache) override {
+        Device &d = *ctx.dev;
+        if (!cache.state || cache.state_spec.bytes() < state_spec().bytes())
+            fail(JB_LLM_EINVAL, "mlstm: the cache holds no state of this mixer's size for the layer");
+        long long n = ctx.n_rows;
+        long long stride = cache.state_stride > 0 ? cache.state_stride : state_spec().shape[0];
+        Stack own;
+        if (!shared_) own = ops::linear(d, h, ctx.dtype, n, hidden_, w_in_);
+        else if (!ctx.shared) fail(JB_LLM_EFAIL, "mlstm: the shared first product is missing");
+        const Stack &P = shared_ ? *ctx.shared : own;
+        const long long c0 = shared_ ? col0_ : 0;
+        ops::GatedMemory m;
+        m.H = (int)H_;
+        m.N = (int)D_;
+        m.P = (int)Dv_;
+        m.qry_col0 = c0;
+        m.key_col0 = c0 + H_ * D_;
+        m.val_col0 = c0 + 2 * H_ * D_;
+        m.gate_col0 = m.val_col0 + H_ * Dv_;
+        m.i_col0 = c0 + i_col_;
+        m.f_col0 = m.i_col0 + H_;
+        m.i_bias = (const float *)i_bias_.ptr;
+        m.f_bias = (const float *)f_bias_.ptr;
+        m.w = (const float *)norm_.ptr;
+        m.cap = cap_;
+        m.q_scale = (float)(1.0 / std::sqrt((double)D_));
+        m.floor = floor_;
+        m.eps = eps_;
+        Buf a = ops::gated_memory(d, P, m, (float *)cache.state, stride, ctx.row_seq, ctx.seq_slot, ctx.n_seqs,
+                                  ctx.kind == DECODE, longest(ctx), ctx.dtype);
+        own = Stack();
+        return ops::linear(d, a.ptr, ctx.dtype, n, H_ * Dv_, w_o_);
+    }
+
+    Json info() const override {
+        Json o = Json::object();
+        o.set("state_floats", state_spec().shape[0]);
+        return o;
+    }
+
+private:
+    long long hidden_, H_, D_, Dv_, i_col_ = 0;
+    float eps_, cap_, floor_;
+    std::string n_q_, n_k_, n_v_, n_g_, n_i_, n_f_, n_bias_, n_o_, n_norm_;
+    DevTensor w_in_, w_o_, norm_, i_bias_, f_bias_;
+    bool shared_ = false;        // the first product's rows went into a pair's shared one
+    long long col0_ = 0;
+};
+
+// A recurrent block around a real-gated linear recurrent unit ("Griffin: Mixing Gated Linear Recurrences with
+// Local Attention for Efficient Language Models"), W channels in `blocks` equal parts:
+//
+//   y = gelu_tanh(Wy h + by);   u = conv(Wx h + bx) + bc        a causal convolution over time per channel
+//   in each part b:  r = sigmoid(Ra_b u_b + ra_b),  i = sigmoid(Ri_b u_b + ri_b)      square matrices [out, in]
+//   log a = -8 r softplus(lam);   S_t = a S_{t-1} + sqrt(1 - a^2) i u;   out = Wo (S * y)
+//
+// The state per sequence: the convolution's last taps - 1 inputs (Wx h + bx), then S, both float32.  The two
+// branches are one product over h, the gates one product per part over u in the compute type; u itself, the
+// gates, decays and the recurrence are float32 in both compute types.
+//
+// params: hidden_size, width (W), blocks (default 1), conv_taps, names (optional): y, x, conv, r, i (the parts'
+// matrices [blocks, W / blocks, W / blocks]), bias (a suffix of all five), lambda, o
+class RealGatedLRU : public Mixer {
+public:
+    RealGatedLRU(const PartSpec &s, DType dt, Device *d) : Mixer(s, dt, d) {
+        hidden_ = s.get_int("hidden_size");
+        W_ = s.get_int("width");
+        blocks_ = s.get_int("blocks", 1);
+        taps_ = (int)s.get_int("conv_taps", 1);
+        if (hidden_ <= 0 || W_ <= 0 || blocks_ <= 0) config_error("rglru: sizes must be positive");
+        if (W_ % blocks_) config_error("rglru: blocks must divide width");
+        if (taps_ < 1) config_error("rglru: conv_taps must be positive");
+        part_ = W_ / blocks_;
+        const Json &nm = s.params.get("names");
+        auto leaf = [&](const char *key, const char *dflt) {
+            return nm.is_object() && nm.get(key).is_string() ? nm.get(key).as_string() : std::string(dflt);
+        };
+        n_y_ = leaf("y", "y_proj");
+        n_x_ = leaf("x", "x_proj");
+        n_conv_ = leaf("conv", "conv1d");
+        n_r_ = leaf("r", "r_gate");
+        n_i_ = leaf("i", "i_gate");
+        n_bias_ = leaf("bias", ".bias");
+        n_lam_ = leaf("lambda", "lambda");
+        n_o_ = leaf("o", "o_proj");
+    }
+
+    void tensors(const std::string &p, TensorList &out) const override {
+        for (const std::string *nm : {&n_y_, &n_x_}) {
+            out.emplace_back(name(p, *nm), TensorSpec{{W_, hidden_}, MATRIX, false});
+            out.emplace_back(name(p, *nm + n_bias_), TensorSpec{{W_}, PARAM, false, 0.0f, 0.02f});
+        }
+        out.emplace_back(name(p, n_conv_), TensorSpec{{W_, taps_}, PARAM, false, 0.25f, 0.25f});
+        out.emplace_back(name(p, n_conv_ + n_bias_), TensorSpec{{W_}, PARAM, false, 0.0f, 0.1f});
+        for (const std::string *nm : {&n_r_, &n_i_}) {
+            out.emplace_back(name(p, *nm), TensorSpec{{blocks_, part_, part_}, MATRIX, false});
+            out.emplace_back(name(p, *nm + n_bias_), TensorSpec{{blocks_, part_}, PARAM, false, 0.0f, 0.5f});
+        }
+        out.emplace_back(name(p, n_lam_), TensorSpec{{W_}, PARAM, false, -4.0f, 1.5f});
+        out.emplace_back(name(p, n_o_), TensorSpec{{hidden_, W_}, MATRIX, false});
+    }
+
+    void load(const std::string &p, TensorMap &t) override {
+        std::vector<DevTensor> in = {take(t, name(p, n_y_)), take(t, name(p, n_x_))};
+        w_in_ = fuse_rows(*dev, in);
+        y_b_ = take(t, name(p, n_y_ + n_bias_));
+        x_b_ = take(t, name(p, n_x_ + n_bias_));
+        conv_w_ = take(t, name(p, n_conv_));
+        conv_b_ = take(t, name(p, n_conv_ + n_bias_));
+        // per part [r's rows | i's rows], all parts one after the other
+        DevTensor r = take(t, name(p, n_r_)), i = take(t, name(p, n_i_));
+        r.shape = i.shape = {blocks_, part_ * part_};
+        std::vector<DevTensor> both = {r, i};
+        r = i = DevTensor();
+        w_gates_ = fuse_cols(*dev, both);
+        w_gates_.shape = {blocks_ * 2 * part_, part_};
+        r_b_ = take(t, name(p, n_r_ + n_bias_));
+        i_b_ = take(t, name(p, n_i_ + n_bias_));
+        lam_ = take(t, name(p, n_lam_));
+        w_o_ = take(t, name(p, n_o_));
+    }
+
+    size_t weight_bytes() const override {
+        return w_in_.bytes() + w_o_.bytes() + w_gates_.bytes() + conv_w_.bytes() + conv_b_.bytes() + y_b_.bytes() +
+               x_b_.bytes() + r_b_.bytes() + i_b_.bytes() + lam_.bytes();
+    }
+
+    DevTensor *first_matrix() override { return w_in_ ? &w_in_ : nullptr; }
+    void share_first_product(long long col0) override {
+        shared_ = true;
+        col0_ = col0;
+    }
+
+    long long conv_state() const { return (long long)(taps_ - 1) * W_; }
+    StateSpec state_spec() const override { return StateSpec{{conv_state() + W_}, F32}; }
+    bool strided_state() const override { return true; }
+    bool graph_safe() const override { return true; }
+
+    Stack forward(StepContext &ctx, const void *h, LayerCache &cache) override {
+        Device &d = *ctx.dev;
+        if (!cache.state || cache.state_spec.bytes() < state_spec().bytes())
+            fail(JB_LLM_EINVAL, "rglru: the cache holds no state of this mixer's size for the layer");
+        long long n = ctx.n_rows;
+        long long stride = cache.state_stride > 0 ? cache.state_stride : state_spec().shape[0];
+        float *st = (float *)cache.state;
+        Stack own;
+        if (!shared_) own = ops::linear(d, h, ctx.dtype, n, hidden_, w_in_);
+        else if (!ctx.shared) fail(JB_LLM_EFAIL, "rglru: the shared first product is missing");
+        const Stack &P = shared_ ? *ctx.shared : own;
+        const long long c0 = shared_ ? col0_ : 0;
+        // u in float32 for the recurrence, and part by part in the compute type for the gates
+        Buf parts;
+        bool two = ctx.kind == EXTEND && taps_ > 1;
+        const float *cw = (const float *)conv_w_.ptr, *cb = (const float *)conv_b_.ptr, *xb = (const float *)x_b_.ptr;
+        Buf u = ops::causal_conv(d, P, c0 + W_, W_, cw, cb, taps_, st, stride, ctx.row_pos, ctx.row_seq, ctx.seq_slot,
+                                 false, F32, true, !two, xb, &parts, ctx.dtype, part_);
+        if (two)
+            ops::causal_conv(d, P, c0 + W_, W_, cw, cb, taps_, st, stride, ctx.row_pos, ctx.row_seq, ctx.seq_slot, false,
+                             F32, false, true, xb);
+        ops::HeadStack G = ops::linear_heads(d, parts.ptr, ctx.dtype, (int)blocks_, n, part_, w_gates_);
+        parts = Buf();
+        ops::LruParams lp;
+        lp.rb = (const float *)r_b_.ptr;
+        lp.ib = (const float *)i_b_.ptr;
+        lp.lam = (const float *)lam_.ptr;
+        lp.yb = (const float *)y_b_.ptr;
+        Buf a = ops::lru(d, G, lp, u.as<float>(), W_, P, c0, st + conv_state(), stride, ctx.row_seq, ctx.seq_slot,
+                         ctx.n_seqs, ctx.kind == DECODE, longest(ctx), ctx.dtype);
+        own = Stack();
+        return ops::linear(d, a.ptr, ctx.dtype, n, W_, w_o_);
+    }
+
+    Json info() const override {
+        Json o = Json::object();
+        o.set("state_floats", state_spec().shape[0]);
+        return o;
+    }
+
+private:
+    long long hidden_, W_, blocks_, part_ = 0;
+    int taps_;
+    std::string n_y_, n_x_, n_conv_, n_r_, n_i_, n_bias_, n_lam_, n_o_;
+    DevTensor w_in_, w_o_, w_gates_, conv_w_, conv_b_, y_b_, x_b_, r_b_, i_b_, lam_;
+    bool shared_ = false;        // the first product's rows went into a pair's shared one
+    long long col0_ = 0;
+};
+
 }  // namespace
 
 void register_recurrent_mixers() {
+    register_part("mixer", "mlstm", [](const PartSpec &s, DType dt, Device *d) {
+        return std::unique_ptr<Part>(new MatrixLSTM(s, dt, d));
+    });
+    register_part("mixer", "rglru", [](const PartSpec &s, DType dt, Device *d) {
+        return std::unique_ptr<Part>(new RealGatedLRU(s, dt, d));
+    });
     register_part("mixer", "mamba2", [](const PartSpec &s, DType dt, Device *d) {
         return std::unique_ptr<Part>(new Mamba2(s, dt, d));
     });

@@ -26,7 +26,7 @@ namespace jb {
 namespace {
 
 // params: rotary_dim, theta, max_positions, scaling (optional): {factor, low, high, original}, or
-// yarn (optional): {factor, original, fast, slow}
+// yarn (optional): {factor, original, fast, slow}, or linear_factor (optional): every frequency is divided by it
 class RopeNeox : public PositionEncoding {
 public:
     RopeNeox(const PartSpec &s, DType dt, Device *d, bool pairs = false) : PositionEncoding(s, dt, d), pairs_(pairs) {
@@ -63,6 +63,13 @@ public:
                 }
                 inv_freq_[(size_t)i] = (float)f;
             }
+        }
+        if (s.has("linear_factor")) {
+            double factor = s.get_double("linear_factor");
+            if (s.has("scaling") || s.has("yarn")) config_error("rope: linear_factor excludes scaling and yarn");
+            if (factor <= 0) config_error("rope: linear_factor must be positive");
+            for (int i = 0; i < half; i++)
+                inv_freq_[(size_t)i] = (float)(std::pow(theta_, -2.0 * (double)i / (double)rotary_dim_) / factor);
         }
         if (s.has("yarn")) {
             // YaRN ("YaRN: Efficient Context Window Extension of Large Language Models", Peng, Quesnelle,

@@ -13,7 +13,8 @@
 // score "chosen_softmax": the choice falls on the largest logits themselves (with router_bias, a
 // vector added to them), and the chosen experts' weights are the softmax over the chosen logits
 // alone, times scale.  With gated, an expert is Wd unit(Wg h, Wu h), the shared expert too (with
-// constants of its own).
+// constants of its own).  weight_on_input: the weight multiplies what the expert reads instead of what it
+// gives: out = sum_{chosen e} Wd_e unit(weight_e Wg_e h, weight_e Wu_e h).
 //
 // All experts' up matrices, the shared expert's and the router's rows are ONE matrix, so
 // one product over h gives every hidden value and the router's logits; the activation
@@ -41,7 +42,8 @@ namespace {
 // {alpha, limit, shift}, the experts' and the shared expert's gated unit, see ops::UnitParams),
 // score ("softmax", the default, "sigmoid": each score the sigmoid of its own logit, or
 // "chosen_softmax"), router_bias (default false: a vector added to the logits), group_best (default 1: a group's score
-// is the sum of this many of its largest choice scores), names (optional): expert (a prefix,
+// is the sum of this many of its largest choice scores), weight_on_input (default false; with gated
+// experts and no identity experts), names (optional): expert (a prefix,
 // the expert's index follows), gate, up, down, router, router_bias, correction, shared
 class RoutedFFN : public FeedForward {
 public:
@@ -75,6 +77,9 @@ public:
         if (hidden_ <= 0 || experts_ < 0 || identity_ < 0 || outs <= 0 || (experts_ > 0 && ff_ <= 0) ||
             shared_ff_ < 0)
             config_error("routed: sizes must be positive");
+        on_input_ = s.has("weight_on_input") && s.params.get("weight_on_input").as_bool();
+        if (on_input_ && (!gated_ || identity_ > 0))
+            config_error("routed: a weight on the input is for gated experts without identity experts");
         if (gated_ && experts_ == 0) config_error("routed: gated needs experts with matrices");
         if (outs > 2048) config_error("routed: the router's kernel takes up to 2048 outputs");
         if (groups_ <= 0 || outs % groups_) config_error("routed: the router's outputs do not form equal groups");
@@ -165,7 +170,8 @@ public:
         Stack out;
         if (act_width_ > 0) {
             Buf act = gated_ ? ops::gated_weighted(d, z, weights.as<float>(), (int)(experts_ + identity_),
-                                                   (int)experts_, ff_, act_, ctx.dtype, shared_ff_, unit_, shared_unit_)
+                                                   (int)experts_, ff_, act_, ctx.dtype, shared_ff_, unit_, shared_unit_,
+                                                   on_input_)
                              : ops::activation_weighted(d, z, act_width_, weights.as<float>(),
                                                         (int)(experts_ + identity_), (int)experts_, ff_, act_,
                                                         ctx.dtype);
@@ -200,7 +206,7 @@ public:
 private:
     long long hidden_, experts_, ff_, identity_, top_, groups_, keep_, shared_ff_;
     long long act_width_ = 0, up_width_ = 0, router_col0_ = 0, group_best_ = 1;
-    bool gated_ = false, bias_ = false;
+    bool gated_ = false, bias_ = false, on_input_ = false;
     int score_ = JB_SCORE_SOFTMAX;
     ops::UnitParams unit_, shared_unit_;
     std::string n_gate_;

@@ -250,6 +250,8 @@ __device__ __forceinline__ void normaliser_rows(const ScanIn &in, const float *f
 // MODE 2: a piece from the state in local[z] (what carry_kernel left there); y is written, and
 //         by a sequence's last piece the slot's state.
 // With pieces, blockIdx.z counts (sequence, piece); pieces that hold no row return.
+// (local is no __restrict__ argument: MODE 2 only reads it, and the compiler might then fetch it ahead
+// of pdl_wait.)
 // NS: the split where it is fixed at compile time (0: nsplit_arg says it).
 // GATED: exponential gates.  The state per head is then [N P | N] with n behind S, all heads' running
 // maxima follow ([H]), and one block more along x walks n.  The running maximum is not written here.
@@ -258,7 +260,7 @@ template <int NR, int TB, int MODE, int NS, bool GATED>
 __global__ void __launch_bounds__(128, NR <= 16 ? 5 : 3)
 matrix_state_scan_kernel(ScanIn in, float *__restrict__ state, size_t slot_stride,
                          const int32_t *__restrict__ row_seq, const int32_t *__restrict__ seq_slot,
-                         float *__restrict__ y, float *__restrict__ local, float *__restrict__ decays, int n,
+                         float *__restrict__ y, float *local, float *decays, int n,
                          int H, int G, int N, int P, int nsplit_arg, int every_row_starts, int piece, int pieces)
 {
     extern __shared__ float4 sm4[];
@@ -519,7 +521,7 @@ matrix_state_scan_kernel(ScanIn in, float *__restrict__ state, size_t slot_strid
 // S <- decays[z] S + local[z], and local[z] is left holding the state its piece starts from
 // (the state after the last piece is written by the second pass).  One thread per state value.
 __global__ void __launch_bounds__(256)
-matrix_state_carry_kernel(float *__restrict__ state, size_t slot_stride, const int32_t *__restrict__ row_seq,
+matrix_state_carry_kernel(const float *state, size_t slot_stride, const int32_t *__restrict__ row_seq,
                           const int32_t *__restrict__ seq_slot, float *__restrict__ local,
                           const float *decays, int n, int H, size_t per_head, int piece, int pieces)
 {
@@ -533,7 +535,7 @@ matrix_state_carry_kernel(float *__restrict__ state, size_t slot_stride, const i
     if (rows <= 0)
         return;
     int used = rows >= 2 * piece ? (rows + piece - 1) / piece : 1;
-    float *st = state + (size_t)seq_slot[seq] * slot_stride + idx;
+    const float *st = state + (size_t)seq_slot[seq] * slot_stride + idx;
     pdl_wait();
     float S = *st;
     // eight pieces' values are fetched together, then walked through in order
@@ -1037,7 +1039,7 @@ static int scan_launch(const ScanIn &in, bool gated, float *state, long long slo
     size_t smem1 = (size_t)TB * (NP + PT + 2) * 4;
     JB_SCAN(1, smem1);
     launch(matrix_state_carry_kernel, dim3((unsigned)(((size_t)H * per_head + 255) / 256), (unsigned)n_seqs), 256, 0, st,
-           state, (size_t)slot_stride, row_seq, seq_slot, local, (const float *)decays, n, H, per_head, piece, pieces);
+           (const float *)state, (size_t)slot_stride, row_seq, seq_slot, local, (const float *)decays, n, H, per_head, piece, pieces);
     JB_SCAN(2, smem);
 #undef JB_SCAN
 #undef JB_SCAN_N

@@ -233,8 +233,8 @@ __device__ __forceinline__ float gated_value(float g, float u, int kind, const G
 // boundaries).
 template <typename TO, int V>
 __global__ void __launch_bounds__(256)
-gated_weighted_kernel(const float *__restrict__ z, int S, size_t stride, int ld,
-                      const float *__restrict__ weights, int w_ld, int n_experts, int ff, int shared_ff,
+gated_weighted_kernel(const float *z, int S, size_t stride, int ld,
+                      const float *weights, int w_ld, int n_experts, int ff, int shared_ff,
                       int kind, GatedUnit unit, GatedUnit shared_unit, TO *__restrict__ out, int width,
                       int on_input)
 {

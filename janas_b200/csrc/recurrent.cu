@@ -204,7 +204,7 @@ __device__ __forceinline__ void store_part4(const ConvParts &q, int n, int r, in
 
 template <typename TO>
 __global__ void __launch_bounds__(256)
-causal_conv_kernel(const float *__restrict__ u, int S, size_t stride, int ld, int col0,
+causal_conv_kernel(const float *u, int S, size_t stride, int ld, int col0,
                    const float *__restrict__ w, const float *__restrict__ bias, float *__restrict__ state,
                    size_t slot_stride, const int32_t *__restrict__ row_pos, const int32_t *__restrict__ row_seq,
                    const int32_t *__restrict__ seq_slot, TO *__restrict__ out, int out_ld, int n, int C, int taps,
@@ -249,7 +249,7 @@ causal_conv_kernel(const float *__restrict__ u, int S, size_t stride, int ld, in
 // in the order of causal_conv_kernel, so a row's bits are the same on either way.
 template <typename TO, int TAPS, int RB>
 __global__ void __launch_bounds__(256)
-causal_conv_rows_kernel(const float *__restrict__ u, int ld, int col0, const float *__restrict__ w,
+causal_conv_rows_kernel(const float *u, int ld, int col0, const float *__restrict__ w,
                         const float *__restrict__ bias, float *__restrict__ state, size_t slot_stride,
                         const int32_t *__restrict__ row_pos, const int32_t *__restrict__ row_seq,
                         const int32_t *__restrict__ seq_slot, TO *__restrict__ out, int out_ld, int n, int C,

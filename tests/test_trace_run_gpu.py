@@ -283,3 +283,54 @@ def test_trace_run_salivik(tmp_path, dtype, tol):
                 break                                   # a tie within rounding: stop comparing
             seq.append(int(lg.argmax()))
         assert len(seq) > 21 and " ".join(map(str, seq[20:])) in r.stdout, r.stdout[-500:]
+
+
+@pytest.mark.parametrize("dtype,tol", [("float32", 5e-5), ("bfloat16", 5e-2)])
+def test_trace_run_dafalix(tmp_path, dtype, tol):
+    """The same program on a model of the Dafalix design: layers that run three times with pages and
+    states of their own in each pass, a window, a batch of unequal requests decoded together,
+    and the command line's generation on the same folder."""
+    import plain_dafalix as pd
+    from dafalix_models import model
+    folder, c, w = model("FA")
+    rng = np.random.default_rng(27)
+    v = c["vocab"]
+    batch = [(tokens(rng, 140, v), 131), (tokens(rng, 3, v), 1), (tokens(rng, 66, v), 64)]
+    steps = trace_batches([batch], want_prompt_all=False)
+    trace = tmp_path / "trace.jsonl"
+    write_trace(trace, steps)
+    out = tmp_path / "out"
+    r = subprocess.run([sys.executable, os.path.join(ROOT, "bin", "trace_run"), "--model", folder,
+                        "--dtype", dtype, "--out", str(out), "--max-tokens", "209"],
+                       stdin=open(trace), capture_output=True, text=True, timeout=900)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert r.stdout.split("\n")[:len(steps)] == [f"done {s['step']}" for s in steps]
+    plain = [pd.forward(c, w, t, None if dtype == "float32" else "bfloat16").numpy() for t, _ in batch]
+    pos = {}
+    for st in steps:
+        n_want = sum(len(e["want"]) for e in st["entries"])
+        got = np.fromfile(out / f"{st['step']}.f32", dtype="<f4").reshape(n_want, v)
+        row = 0
+        for e in st["entries"]:
+            i = int(e["id"][3:])
+            base = pos.get(e["id"], 0)
+            for w_ in e["want"]:
+                assert rel_err(got[row], plain[i][base + w_]) <= tol, (st["step"], e["id"])
+                row += 1
+            pos[e["id"]] = base + len(e["tokens"])
+    if dtype == "float32":
+        # greedy generation through the command line: the plain model's own choices
+        prompt = batch[2][0][:20]
+        r = subprocess.run([sys.executable, os.path.join(ROOT, "bin", "janas-b200"), folder, "--tokens",
+                            " ".join(map(str, prompt)), "--max", "6", "--dtype", "float32"],
+                           capture_output=True, text=True, timeout=900)
+        assert r.returncode == 0, r.stderr[-2000:]
+        import torch
+        seq = list(prompt)
+        for _ in range(6):
+            lg = pd.forward(c, w, seq)[-1]
+            top = torch.topk(lg, 2).values
+            if (top[0] - top[1]) < 1e-4 * lg.abs().max():
+                break                                   # a tie within rounding: stop comparing
+            seq.append(int(lg.argmax()))
+        assert len(seq) > 21 and " ".join(map(str, seq[20:])) in r.stdout, r.stdout[-500:]

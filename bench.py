@@ -12,6 +12,7 @@
     python bench.py --only kefesun [--design-size 4b]      (the Kefesun design beside Dunavik's attention layers)
     python bench.py --only munisun [--design-size 4b]      (the Munisun design beside Kefesun's mixed layers)
     python bench.py --only salivik [--design-size 4b]      (the Salivik design beside Munisun and Dunavik layers)
+    python bench.py --only dafalix [--design-size 4b]      (the Dafalix design beside Munisun layers)
 
 The default run has the layer sizes of Qwen3-4B (36 layers, hidden 2560, 32
 heads, 8 KV heads, head size 128, feed-forward 9728, vocabulary 151936, tied
@@ -648,6 +649,52 @@ def salivik_flops(cfg, tokens):
     return asked + head, run + head
 
 
+def dafalix_cfg(size, n_layers, vocab, mixers="mixed", window=1024):
+    """A Dafalix config.json of the given layer sizes.  mixers: "parallel" (every layer windowed attention
+    beside a real-gated linear recurrent unit as wide as the model, in blocks of 256 channels), "mlstm"
+    (every layer a matrix memory as wide as the model, heads of the size's head size) or "mixed" (the two
+    in turn).  Four streams; every layer's feed-forward is routed and holds as many weights as the dense
+    one of the size: eight experts of an eighth of its width, two per token."""
+    dm, nh, nkv, hd, ff = DESIGN_SIZES[size]
+    moe = {"expert": {"ff": ff // 8}, "kind": "moe", "router": {"experts": 8, "top": 2}}
+    layers = []
+    for i in range(n_layers):
+        if mixers == "mlstm" or (mixers == "mixed" and i % 2 == 1):
+            layers.append({"type": "mlstm", "mlp": moe,
+                           "mixer": {"dim": hd, "gate_cap": 15.0, "heads": dm // hd, "vdim": hd}})
+        else:
+            left = {"dim": hd, "heads": nh, "kv_heads": nkv, "mask": {"size": window}, "scale": hd ** -0.5, "vdim": hd,
+                    "rot": {"base": 500000.0, "dims": hd // 2, "scaling": {"factor": 4.0}}}
+            layers.append({"type": "parallel", "mlp": moe, "mixer": {
+                "left": left, "left_scale": 0.7, "right": {"blocks": dm // 256, "conv": 4, "width": dm}, "right_scale": 0.7}})
+    return {"architecture": "Dafalix", "layers": layers, "norm": {"eps": 1e-5}, "residual_mult": 0.7, "streams": 4,
+            "vocab": vocab, "width": dm}
+
+
+def dafalix_flops(cfg, tokens):
+    """Multiply-adds times two of one prompt of a Dafalix model: (what the design asks for: the chosen
+    experts' products; what the engine runs: every expert's for every token).  Both with the mixers'
+    products, the attention over the keys a row sees, the matrix memories (4 N P per head and token), the
+    gates' block products and the head for one row."""
+    dm, asked, run = cfg["width"], 0.0, 0.0
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        if layer["type"] == "mlstm":
+            qk, vv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            mats, attn = dm * (2 * qk + 2 * vv + 2 * m["heads"]) + vv * dm, 4 * m["heads"] * m["dim"] * m["vdim"] * tokens
+        else:
+            a, r = m["left"], m["right"]
+            H, G, D, Dv, W = a["heads"], a["kv_heads"], a["dim"], a["vdim"], r["width"]
+            mats = dm * (H * D + G * (D + Dv)) + H * Dv * dm + 3 * dm * W + 2 * W * W // r["blocks"]
+            w = (a.get("mask") or {}).get("size") or tokens
+            attn = 2 * H * (D + Dv) * sum(min(t + 1, w) for t in range(tokens))
+        ro, ef = layer["mlp"]["router"], layer["mlp"]["expert"]["ff"]
+        asked += 2 * (mats + dm * ro["experts"] + 3 * dm * ro["top"] * ef) * tokens + attn
+        run += 2 * (mats + dm * ro["experts"] + 3 * dm * ro["experts"] * ef) * tokens + attn
+    head = 2 * dm * cfg["vocab"]
+    return asked + head, run + head
+
+
 def qwen3_cfg(size, n_layers, vocab, max_positions):
     dm, nh, nkv, hd, ff = DESIGN_SIZES[size]
     return dict(QWEN3_4B, num_hidden_layers=n_layers, hidden_size=dm, num_attention_heads=nh,
@@ -739,6 +786,13 @@ def design_compare(args):
                        ("dunavik-latent", dunavik_cfg(size, n_layers, vocab, "latent", args.window))]
             kinds = args.mixers + ",retention" if args.mixers == ap_default_mixers() else args.mixers
             designs += [(f"salivik-{mx}", salivik_cfg(size, n_layers, vocab, mx, args.window)) for mx in kinds.split(",")]
+        if args.only == "dafalix":
+            # beside Munisun's layers: two mixers side by side, recurrences with a vector and with a
+            # matrix as state, gated routed experts
+            designs = [("munisun-mixed", munisun_cfg(size, n_layers, vocab, "mixed")),
+                       ("munisun-parallel2", munisun_cfg(size, n_layers, vocab, "parallel2"))]
+            designs += [(f"dafalix-{mx}", dafalix_cfg(size, n_layers, vocab, mx, args.window))
+                        for mx in args.mixers.replace("attention", "parallel").replace("latent", "mlstm").split(",")]
         for design, cfg in designs:
             rng = np.random.default_rng(0)
             eng = Engine.open_random(cfg, seed=0, dtype=args.dtype, max_tokens=max(room * batch, T + 64),
@@ -751,6 +805,8 @@ def design_compare(args):
                 flops, flops_run = munisun_flops(cfg, T)
             elif design.startswith("salivik"):
                 flops, flops_run = salivik_flops(cfg, T)
+            elif design.startswith("dafalix"):
+                flops, flops_run = dafalix_flops(cfg, T)
             else:
                 flops = (dunavik_flops(cfg, T, args.window) if design.startswith("dunavik")
                          else design_flops(design.split("-")[0], size, n_layers, T, vocab))
@@ -833,7 +889,7 @@ def main():
     ap.add_argument("--share", type=int, default=0,
                     help="--only zuzelorn: also a model whose layers share keys and values in groups of this many")
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "timeline", "prefill-timeline", "generate",
-                                                    "zuzelorn", "dunavik", "kefesun", "munisun", "salivik"],
+                                                    "zuzelorn", "dunavik", "kefesun", "munisun", "salivik", "dafalix"],
                     help="run one part only and print its time (for profiling; no JSON line "
                          "but for generate); prefill-timeline: each kernel's share of one prefill "
                          "step; timeline: when each kernel of one replayed decode "
@@ -851,7 +907,7 @@ def main():
     if args.gpus != 1:
         print("bench.py: this engine runs on one GPU; --gpus must be 1")
         return 2
-    if args.only in ("zuzelorn", "dunavik", "kefesun", "munisun", "salivik"):
+    if args.only in ("zuzelorn", "dunavik", "kefesun", "munisun", "salivik", "dafalix"):
         args.warmup = max(args.warmup, 3)
         return design_compare(args)
     full_layers = MODELS[args.model]["num_hidden_layers"]

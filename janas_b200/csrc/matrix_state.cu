@@ -59,15 +59,24 @@ __device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf
 // log(1 + e^v), the same number as the direct form wherever that does not overflow
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
 
-// row r's log input gate and log forget gate of head h
-__device__ __forceinline__ void log_gates(const LogGates &g, int r, int h, float &i, float &f)
+// row r's sums of the two log gates of head h, and the gates from them
+__device__ __forceinline__ void gate_sums(const LogGates &g, int r, int h, float &zi, float &zf)
 {
     const float *row = g.src + (size_t)r * g.ld + h;
-    float zi = add_partials(g.i_bias[h], row + g.i_col0, g.S, g.stride);
-    float zf = add_partials(g.f_bias[h], row + g.f_col0, g.S, g.stride);
-    i = g.cap * tanhf(zi / g.cap);
-    zf = g.cap * tanhf(zf / g.cap);
+    zi = add_partials(g.i_bias[h], row + g.i_col0, g.S, g.stride);
+    zf = add_partials(g.f_bias[h], row + g.f_col0, g.S, g.stride);
+}
+__device__ __forceinline__ void gates_of(float cap, float zi, float zf, float &i, float &f)
+{
+    i = cap * tanhf(zi / cap);
+    zf = cap * tanhf(zf / cap);
     f = fminf(zf, 0.0f) - log1pf(expf(-fabsf(zf)));
+}
+__device__ __forceinline__ void log_gates(const LogGates &g, int r, int h, float &i, float &f)
+{
+    float zi, zf;
+    gate_sums(g, r, h, zi, zf);
+    gates_of(g.cap, zi, zf, i, f);
 }
 
 // an asynchronous copy of BYTES (4 or 16) from global to shared memory, and the wait for all of a thread's
@@ -96,28 +105,49 @@ __device__ __forceinline__ int first_row_of(const int32_t *__restrict__ row_seq,
 // The gates of a step's rows ahead of a prompt's recurrence: a, b and e^(-m) per row and head, and the
 // slots' running maximum after the step (at m_off + h of a slot's state).  A block per (head,
 // sequence); a thread has consecutive rows, whose maps m -> max(m + F, M) are composed across the
-// block to give every thread the maximum it starts from.
-__global__ void __launch_bounds__(256)
+// block to give every thread the maximum it starts from.  HELD: the most rows a thread keeps the gates
+// of (0: any number, their sums are read and their gates taken twice).
+constexpr int LG_THREADS = 512;
+template <int HELD>
+__global__ void __launch_bounds__(LG_THREADS)
 log_gates_kernel(LogGates g, float *__restrict__ state, size_t slot_stride, size_t m_off,
                  const int32_t *__restrict__ row_seq, const int32_t *__restrict__ seq_slot,
                  float *__restrict__ coef_a, float *__restrict__ coef_b, float *__restrict__ em, int n, int H)
 {
-    __shared__ float wF[8], wM[8], last[256];
+    __shared__ float wF[LG_THREADS / 32], wM[LG_THREADS / 32], last[LG_THREADS];
     pdl_trigger();
     int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     int r0 = first_row_of(row_seq, n, seq), r1 = first_row_of(row_seq, n, seq + 1);
     if (r0 >= r1)
         return;
-    int per = (r1 - r0 + 255) / 256;
+    int per = (r1 - r0 + LG_THREADS - 1) / LG_THREADS;
     int t0 = min(r1, r0 + tid * per), t1 = min(r1, t0 + per);
     float *mp = state + (size_t)seq_slot[seq] * slot_stride + m_off + h;
     pdl_wait();
     float m0 = *mp, F = 0.0f, M = -INFINITY;
-    for (int r = t0; r < t1; r++) {
-        float i, f;
-        log_gates(g, r, h, i, f);
-        F += f;
-        M = fmaxf(M + f, i);
+    constexpr int CAP = HELD > 0 ? HELD : 1;
+    float gi[CAP], gf[CAP];
+    if (HELD > 0) {
+        // (rows past the thread's last repeat it: the loads go out together)
+#pragma unroll
+        for (int k = 0; k < CAP; k++)
+            gate_sums(g, min(t0 + k, r1 - 1), h, gi[k], gf[k]);
+#pragma unroll
+        for (int k = 0; k < CAP; k++)
+            gates_of(g.cap, gi[k], gf[k], gi[k], gf[k]);
+#pragma unroll
+        for (int k = 0; k < CAP; k++)
+            if (t0 + k < t1) {
+                F += gf[k];
+                M = fmaxf(M + gf[k], gi[k]);
+            }
+    } else {
+        for (int r = t0; r < t1; r++) {
+            float i, f;
+            log_gates(g, r, h, i, f);
+            F += f;
+            M = fmaxf(M + f, i);
+        }
     }
 #pragma unroll
     for (int o = 1; o < 32; o *= 2) {
@@ -142,9 +172,7 @@ log_gates_kernel(LogGates g, float *__restrict__ state, size_t slot_stride, size
     // The first row's a is taken from the maximum that the thread before arrived at, not from the
     // composed one, which differs from it in rounding: the products of the a telescope exactly.
     float first_f = 0.0f, first_m = 0.0f;
-    for (int r = t0; r < t1; r++) {
-        float i, f;
-        log_gates(g, r, h, i, f);
+    auto row = [&](int r, float i, float f) {
         float mn = fmaxf(f + m, i);
         if (r == t0) {
             first_f = f;
@@ -155,6 +183,18 @@ log_gates_kernel(LogGates g, float *__restrict__ state, size_t slot_stride, size
         coef_b[(size_t)r * H + h] = expf(i - mn);
         em[(size_t)r * H + h] = expf(-mn);
         m = mn;
+    };
+    if (HELD > 0) {
+#pragma unroll
+        for (int k = 0; k < CAP; k++)
+            if (t0 + k < t1)
+                row(t0 + k, gi[k], gf[k]);
+    } else {
+        for (int r = t0; r < t1; r++) {
+            float i, f;
+            log_gates(g, r, h, i, f);
+            row(r, i, f);
+        }
     }
     last[tid] = m;
     __syncthreads();
@@ -571,18 +611,24 @@ struct PartScale {
     const int32_t *row_seq, *seq_slot;
 };
 
-// the factor on part `part` of row r, and where (null: nowhere) which maximum is to be written after
-// every thread of the part has called this
-__device__ __forceinline__ float part_factor(const PartScale &ps, int r, int part, int parts, float *&mp, float &m)
+// where the running maximum of part `part` of row r stands that is to be written after every thread of
+// the part has called part_factor (null: nowhere); reads the index arrays alone
+__device__ __forceinline__ float *part_maximum(const PartScale &ps, int r, int part)
 {
-    mp = nullptr;
+    if (ps.nq == nullptr || ps.em != nullptr)
+        return nullptr;
+    return ps.state + (size_t)ps.seq_slot[ps.row_seq[r]] * ps.slot_stride + ps.m_off + part;
+}
+
+// the factor on part `part` of row r; with mp the maximum after the row comes back in m
+__device__ __forceinline__ float part_factor(const PartScale &ps, int r, int part, int parts, const float *mp, float &m)
+{
     if (ps.nq == nullptr)
         return 1.0f;
     float e;
     if (ps.em != nullptr) {
         e = ps.em[(size_t)r * parts + part];
     } else {
-        mp = ps.state + (size_t)ps.seq_slot[ps.row_seq[r]] * ps.slot_stride + ps.m_off + part;
         float i, f;
         log_gates(ps.gates, r, part, i, f);
         m = fmaxf(f + *mp, i);
@@ -606,8 +652,9 @@ gated_part_norm_kernel(const float *y, const float *pre, int pre_S, size_t pre_s
     __shared__ float red[32];
     pdl_trigger();
     int r = blockIdx.x, part = blockIdx.y, len = width / parts, c0 = part * len;
+    float *mp = part_maximum(ps, r, part);
     pdl_wait();
-    float ss = 0.0f, m_new = 0.0f, *mp;
+    float ss = 0.0f, m_new = 0.0f;
     const float div = part_factor(ps, r, part, parts, mp, m_new);
     for (int c = c0 + threadIdx.x; c < c0 + len; c += blockDim.x) {
         float v = y[(size_t)r * width + c] * div;
@@ -665,10 +712,11 @@ gated_part_norm_warp_kernel(const float *y, const float *pre, int pre_S, size_t 
         }
         return v;
     };
+    float *mp = part_maximum(ps, (int)r, c0 / len);
     pdl_wait();
     float4 v[U], g[U];
-    float ss = 0.0f, m_new = 0.0f, *mp;
-    const float div = part_factor(ps, (int)r, c0 / len, parts, mp, m_new);
+    float ss = 0.0f, m_new = 0.0f;
+    // y and the second gate are asked for before the factor is worked out
 #pragma unroll
     for (int u = 0; u < U; u++) {
         int c = c0 + 4 * (lane + 32 * u);
@@ -676,9 +724,16 @@ gated_part_norm_warp_kernel(const float *y, const float *pre, int pre_S, size_t 
         if (c >= c0 + len)
             continue;
         v[u] = load4(y + (size_t)r * width + c);
-        v[u] = make_float4(v[u].x * div, v[u].y * div, v[u].z * div, v[u].w * div);
         if (post != nullptr)
             g[u] = sums4(post + (size_t)r * post_ld + post_col0 + c, post_S, post_stride);
+    }
+    const float div = part_factor(ps, (int)r, c0 / len, parts, mp, m_new);
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+        int c = c0 + 4 * (lane + 32 * u);
+        if (c >= c0 + len)
+            continue;
+        v[u] = make_float4(v[u].x * div, v[u].y * div, v[u].z * div, v[u].w * div);
         if (pre != nullptr) {
             float4 t = sums4(pre + (size_t)r * pre_ld + pre_col0 + c, pre_S, pre_stride);
             v[u] = make_float4(v[u].x * silu_f(t.x), v[u].y * silu_f(t.y), v[u].z * silu_f(t.z), v[u].w * silu_f(t.w));
@@ -927,6 +982,30 @@ pair_combine_cluster_kernel(const float *L, int SL, size_t strideL, const float 
     }
 }
 
+// The weighted sum alone, four values a thread; everything on 16-byte boundaries.  The additions run
+// in pair_combine_kernel's order.
+__global__ void __launch_bounds__(256)
+pair_sum_vec_kernel(const float *L, int SL, size_t strideL, const float *R, int SR, size_t strideR, float sl, float sr,
+                    float *__restrict__ out, size_t fours)
+{
+    pdl_trigger();
+    size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= fours)
+        return;
+    auto sums4 = [](const float *p, int S, size_t stride) {
+        float4 v = load4(p);
+        for (int k = 1; k < S; k++) {
+            float4 t = load4(p + (size_t)k * stride);
+            v = make_float4(v.x + t.x, v.y + t.y, v.z + t.z, v.w + t.w);
+        }
+        return v;
+    };
+    pdl_wait();
+    float4 u = sums4(L + 4 * i, SL, strideL), v = sums4(R + 4 * i, SR, strideR);
+    store4(out + 4 * i, make_float4(fmaf(sl, u.x, sr * v.x), fmaf(sl, u.y, sr * v.y), fmaf(sl, u.z, sr * v.z),
+                                    fmaf(sl, u.w, sr * v.w)));
+}
+
 // g[r, j] = gelu_tanh(sum P[r, j]) * table[tokens[r], col0 + j]: a gate computed from the
 // residual stream times the token's own vector for the layer.
 template <typename TT, typename TO>
@@ -1106,8 +1185,16 @@ extern "C" int jb_gated_memory_scan(const float *src, int S, long long stride, i
     if (!every_row_starts) {
         size_t m_off = (size_t)H * ((size_t)N * P + N);
         float *ca = scratch, *cb = scratch + (size_t)n * H;
-        launch(log_gates_kernel, dim3((unsigned)H, (unsigned)n_seqs), 256, 0, st, g, state, (size_t)slot_stride, m_off,
-               row_seq, seq_slot, ca, cb, em, n, H);
+        // (LG_THREADS threads take a sequence's rows; the host may not know how long the longest is)
+        dim3 gg((unsigned)H, (unsigned)n_seqs);
+        int per = ((max_len > 0 ? max_len : n) + LG_THREADS - 1) / LG_THREADS;
+#define JB_LG(HELD)                                                                                             \
+    launch(log_gates_kernel<HELD>, gg, LG_THREADS, 0, st, g, state, (size_t)slot_stride, m_off, row_seq, seq_slot, ca, cb, em, n, H)
+        if (per <= 1) JB_LG(1);
+        else if (per <= 4) JB_LG(4);
+        else if (per <= 8) JB_LG(8);
+        else JB_LG(0);
+#undef JB_LG
         in.coef_a = ca;
         in.coef_b = cb;
         scratch += 2 * (size_t)n * H;
@@ -1246,6 +1333,15 @@ extern "C" int jb_pair_combine(const float *L, int SL, long long strideL, const 
         return JB_OK;
     if (m <= 0 || SL <= 0 || SR <= 0 || L == nullptr || R == nullptr || out == nullptr || (wl == nullptr) != (wr == nullptr))
         return JB_EINVAL;
+    // (a decode step's products leave many partial sums a value: the cluster kernel's threads share them out)
+    if (wl == nullptr && !(few_rows && n <= 32 && m >= 512) && m % 4 == 0 && strideL % 4 == 0 && strideR % 4 == 0 &&
+        (((uintptr_t)L | (uintptr_t)R | (uintptr_t)out) & 15) == 0) {
+        size_t fours = (size_t)n * m / 4;
+        unsigned threads = fours < 148 * 256 ? 64 : 256;       // few rows: more blocks
+        launch(pair_sum_vec_kernel, (unsigned)((fours + threads - 1) / threads), threads, 0, st, L, SL, (size_t)strideL, R, SR,
+               (size_t)strideR, sl, sr, out, fours);
+        return launch_status();
+    }
     if (few_rows && n <= 32 && m >= 512) {
         constexpr int C = 8;
         int cols = (m + C - 1) / C;

@@ -569,17 +569,25 @@ template <bool FAST> __device__ __forceinline__ float gelu_tanh_(float v)
     return 0.5f * v * (1.0f + th);
 }
 
-// a and b = sqrt(1 - a^2) i u of row r's channel ch; c = -8 softplus(lam), all in float32
-__device__ __forceinline__ void lru_coef(const LruIn &in, int r, int ch, float c, float rb, float ib, float &a, float &b)
+// row r's sums of the two gates of channel ch, biases included, and its input u
+__device__ __forceinline__ void lru_sums(const LruIn &in, int r, int ch, float rb, float ib, float &zr, float &zi,
+                                         float &u)
 {
     int blk = ch / in.part, j = ch - blk * in.part;
     const float *g = in.G + ((size_t)blk * in.gS * in.n + r) * 2 * in.part + j;
     size_t gs = (size_t)in.n * 2 * in.part;
-    float rg = sigmoidf_<false>(add_partials(rb, g, in.gS, gs));
-    float ig = sigmoidf_<false>(add_partials(ib, g + in.part, in.gS, gs));
-    float la = c * rg;
-    a = expf(la);
-    b = sqrtf(-expm1f(2.0f * la)) * ig * in.u[(size_t)r * in.W + ch];
+    zr = add_partials(rb, g, in.gS, gs);
+    zi = add_partials(ib, g + in.part, in.gS, gs);
+    u = in.u[(size_t)r * in.W + ch];
+}
+// a and b = sqrt(1 - a^2) i u from them; c = -8 softplus(lam), all in float32.  With e = exp(log a) - 1:
+// a = 1 + e and 1 - a^2 = -e (2 + e), without the loss of a difference from one.
+template <bool FAST>
+__device__ __forceinline__ void lru_coef(float zr, float zi, float u, float c, float &a, float &b)
+{
+    float e = expm1f(c * sigmoidf_<FAST>(zr));
+    a = 1.0f + e;
+    b = sqrtf(-e * (2.0f + e)) * sigmoidf_<FAST>(zi) * u;
 }
 
 // One thread per channel of a sequence's rows, or of a piece of `piece` of them (a sequence with
@@ -591,7 +599,7 @@ __device__ __forceinline__ void lru_coef(const LruIn &in, int r, int ch, float c
 // (What the kernel before this one writes is not a const __restrict__ argument: the compiler may fetch
 // such values through the read-only path ahead of pdl_wait.)
 template <typename TO, int MODE, int U>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, MODE == 0 ? 1 : 10)
 lru_kernel(LruIn in, float *__restrict__ state, size_t slot_stride, const int32_t *__restrict__ row_seq,
            const int32_t *__restrict__ seq_slot, float *__restrict__ coef, float *__restrict__ AB,
            const float *carry, TO *__restrict__ out, int every_row_starts, int piece)
@@ -623,7 +631,7 @@ lru_kernel(LruIn in, float *__restrict__ state, size_t slot_stride, const int32_
     float s = MODE == 0 ? *st : MODE == 1 ? 0.0f : carry[z * in.W + ch];
     float A = 1.0f;
     for (int rr = r0; rr < r1; rr += U) {
-        float a[U], b[U], g[U];
+        float a[U], b[U], g[U], u[U];
 #pragma unroll
         for (int k = 0; k < U; k++) {
             int r = min(rr + k, r1 - 1);
@@ -631,10 +639,15 @@ lru_kernel(LruIn in, float *__restrict__ state, size_t slot_stride, const int32_
                 a[k] = coef[(size_t)r * in.W + ch];
                 b[k] = coef[cw + (size_t)r * in.W + ch];
             } else {
-                lru_coef(in, r, ch, c, rb, ib, a[k], b[k]);
+                lru_sums(in, r, ch, rb, ib, a[k], b[k], u[k]);
             }
             if (MODE != 1)
                 g[k] = add_partials(yb, in.P + (size_t)r * in.ld + in.y_col0 + ch, in.S, in.stride);
+        }
+        if (MODE != 2) {
+#pragma unroll
+            for (int k = 0; k < U; k++)
+                lru_coef<FAST>(a[k], b[k], u[k], c, a[k], b[k]);
         }
 #pragma unroll
         for (int k = 0; k < U; k++)
@@ -742,7 +755,7 @@ extern "C" int jb_lru(const float *G, int gS, int part, const float *rb, const f
     if (out_dt == JB_F32) JB_LRU(float, 1, 4); else JB_LRU(bf16, 1, 4);
     launch(lru_carry_kernel, dim3(gx, (unsigned)n_seqs), 128, 0, st, (const float *)state, (size_t)slot_stride, row_seq,
            seq_slot, (const float *)AB, carry, n, W, piece, pieces);
-    if (out_dt == JB_F32) JB_LRU(float, 2, 8); else JB_LRU(bf16, 2, 8);
+    if (out_dt == JB_F32) JB_LRU(float, 2, 4); else JB_LRU(bf16, 2, 4);
 #undef JB_LRU
     return launch_status();
 }

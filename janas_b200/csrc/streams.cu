@@ -239,6 +239,8 @@ streams_cluster_kernel(float *__restrict__ x, int ns, StreamWrite wr, const int3
         row[c - c0] = u;
         sum += u;
     }
+    if (out == nullptr)
+        return;                             // the write alone: no CTA of the cluster waits for another
     sum = block_sum(sum, red);
     if (threadIdx.x < C)
         cluster_write(&part_sum[rank], threadIdx.x, sum);
@@ -333,7 +335,7 @@ extern "C" int jb_streams(float *x, int ns, const float *y, int S, long long str
     StreamWrite wr{y, S, (size_t)stride, ls, out_w, mix, mult};
     StreamRead rd{in_w, w, b, eps};
     constexpr int CL = 8;
-    if (few_rows && n <= 32 && dm >= 64 * CL && out != nullptr && w != nullptr && out_dt == JB_BF16) {
+    if (few_rows && n <= 32 && dm >= 64 * CL && (out == nullptr || (w != nullptr && out_dt == JB_BF16))) {
         int cols = (dm + CL - 1) / CL;
         unsigned threads = (unsigned)min(512, (cols + 31) / 32 * 32);
 #define JB_STC(NS)                                                                                             \

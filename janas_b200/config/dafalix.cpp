@@ -1,8 +1,8 @@
 // Typed configuration of the Dafalix decoder, read from its config.json.
 //
 // The file names the design ("architecture": "Dafalix"), the sizes (vocab, width, streams), the
-// constants (norm.eps, residual_mult), optionally a loop {start, stop, times} (layers start .. stop-1
-// run `times` times in a row with the same weights and keys, values and states of their own) and a
+// constants (norm.eps, residual_mult), optionally a loop {start, stop, times} (a span of
+// layers that is passed through `times` times; each pass keeps keys, values and states apart) and a
 // list of layers, each with its mixer's type, the mixer's sizes and its feed-forward, or null:
 //
 //   type "parallel": mixer {left {heads, kv_heads, dim, vdim, scale, mask {size}, rot {base, dims,
@@ -17,7 +17,7 @@
 // value i + dims / 2), beside a real-gated linear recurrent unit behind a short convolution; both
 // read the same input and are added with two factors.  "mlstm": a matrix memory with exponential
 // gates, a norm per head and a sigmoid gate.  Experts are SwiGLU without biases; the router's scores
-// are sigmoids, not renormalized, and weigh what the experts read.  The head is the embedding table.
+// are sigmoids, used as they are, and weigh what the experts read.  The head is the embedding table.
 //
 // Tensor names: embed, final.norm, final.norm.b; layer i below "l<i>": norm1, norm1.b, norm2, norm2.b,
 // ls1, ls2, hc1.{in, out, mix}, hc2.{in, out, mix}, mix.left.{q, k, v, o, q.norm, k.norm},

@@ -6,7 +6,7 @@
 // A launch does a write, a read, or a write and the read of what was just written (the next
 // sublayer's), so that the streams go through the chip once per sublayer.  y is a stack of partial
 // sums; ls (a factor per value) may be null; in null: every stream counts once; w null: u itself, in
-// float32.  mix is indexed [from, to].  Everything is computed in float32; mean and variance are two
+// float32.  mix has a row per stream before and a column per stream after.  Everything is computed in float32; mean and variance are two
 // passes over the row, and the order of the additions depends on the row's width alone.
 #include "common.cuh"
 #include "kernels.h"

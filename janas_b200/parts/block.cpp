@@ -424,7 +424,7 @@ private:
 };
 
 // block_params: hidden_size, streams, residual_mult (m, default 1), mixer_streams / ffn_streams: the
-// prefixes (below the layer's) of the weights in [s], out [s] and mix [s, s] (indexed [from, to]),
+// prefixes (below the layer's) of the weights in [s], out [s] and mix [s, s] (row: a stream before, column: a stream after),
 // mixer_scale / ffn_scale (optional): the tensor names of the vectors ls [hidden]; fuse (default true):
 // false runs every norm's read as a launch of its own; unused as in sandwich.
 // A sublayer's result joins the streams in the launch that also reads them for the next sublayer (the

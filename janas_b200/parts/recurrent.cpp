@@ -560,7 +560,7 @@ private:
 // Local Attention for Efficient Language Models"), W channels in `blocks` equal parts:
 //
 //   y = gelu_tanh(Wy h + by);   u = conv(Wx h + bx) + bc        a causal convolution over time per channel
-//   in each part b:  r = sigmoid(Ra_b u_b + ra_b),  i = sigmoid(Ri_b u_b + ri_b)      square matrices [out, in]
+//   in each part b:  r = sigmoid(Ra_b u_b + ra_b),  i = sigmoid(Ri_b u_b + ri_b)
 //   log a = -8 r softplus(lam);   S_t = a S_{t-1} + sqrt(1 - a^2) i u;   out = Wo (S * y)
 //
 // The state per sequence: the convolution's last taps - 1 inputs (Wx h + bx), then S, both float32.  The two

@@ -66,7 +66,7 @@ def read_streams(X: torch.Tensor, w_in: torch.Tensor) -> torch.Tensor:
 
 
 def write_streams(X: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, w_out: torch.Tensor, m: float) -> torch.Tensor:
-    """mix [from, to]; every new stream is made from the old ones"""
+    """a row of mix per stream before, a column per stream after; the old streams alone are read"""
     out = torch.zeros_like(X)
     for t in range(X.shape[1]):
         for s in range(X.shape[1]):
@@ -123,7 +123,7 @@ def attention(h, w, pre, m, eps, rounding=None):
 
 # ------------------------------------------------------- gated linear recurrence
 def causal_conv(u: torch.Tensor, w: torch.Tensor, b: torch.Tensor, before: Optional[torch.Tensor] = None):
-    """u [T, C], w [C, taps] (the last column is the current token's), b [C]; before [taps - 1, C]: the inputs
+    """u [T, C], w [C, taps] (its last column meets the newest input), b [C]; before [taps - 1, C]: the inputs
     ahead of u, zeros when absent"""
     T, taps = u.shape[0], w.shape[1]
     full = torch.cat([torch.zeros(taps - 1, u.shape[1]) if before is None else before, u])
@@ -134,7 +134,7 @@ def causal_conv(u: torch.Tensor, w: torch.Tensor, b: torch.Tensor, before: Optio
 
 
 def block_linear(u: torch.Tensor, w: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
-    """u [T, C] in equal parts, part p times its own square matrix w[p] [out, in], plus b[p]"""
+    """u [T, C] in equal parts, each through its own matrix w[p] and bias b[p]"""
     parts = u.view(u.shape[0], w.shape[0], -1)
     return torch.stack([parts[:, p] @ w[p].T + b[p] for p in range(w.shape[0])], dim=1).reshape(u.shape)
 
